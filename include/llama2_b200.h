@@ -47,8 +47,8 @@ enum l2b_status {
     L2B_ERR_NO_DEVICE = 8
 };
 
-/* GGML tensor types the reference can load (src/load_gguf.jl:26-42,135-154). */
-enum l2b_ggml_type { L2B_TYPE_F32 = 0, L2B_TYPE_Q4_K = 12, L2B_TYPE_Q5_K = 13, L2B_TYPE_Q6_K = 14 };
+/* GGML tensor types the reference can load (src/load_gguf.jl:26-42,135-154), and bf16 for layer-stack models. */
+enum l2b_ggml_type { L2B_TYPE_F32 = 0, L2B_TYPE_Q4_K = 12, L2B_TYPE_Q5_K = 13, L2B_TYPE_Q6_K = 14, L2B_TYPE_BF16 = 30 };
 
 /* Tensor roles = the fields of TransformerWeights / TransformerLayerWeights
  * (src/inference.jl:27-48). */
@@ -122,6 +122,19 @@ int32_t l2b_model_load_gguf(const char* path, int32_t seq_len, int32_t act_plane
  * number of tensors, context length.  Fails with L2B_ERR_BAD_ARG ("Not a GGUF file", :89) on anything else. */
 int32_t l2b_gguf_inspect(const char* path, l2b_config* config_out, int32_t* arch_out, int64_t* n_tensors, int64_t* context_length);
 
+/* ---- layer-stack models (no counterpart in the reference) -------------------------------------------------
+ * Decoders whose config.json lists their layers one by one and names the design under "architecture" (Savozen: latent attention
+ * with a sink and an output gate, dynamic-tanh norms, tanh-gelu feed-forward, per-layer token input, a stretch of layers run
+ * several times).  Every session, batch and sampling entry point below serves them; tensor parallelism does not.
+ *   seq_len       positions a session holds;
+ *   compute_type  L2B_TYPE_BF16: bf16 matrix operands and latent cache, everything else f32; L2B_TYPE_F32: f32 throughout.
+ * l2b_model_load_dir reads DIR/config.json and DIR/model.safetensors.  l2b_model_create_stack builds an empty model from the
+ * text of a config.json; its tensors are then given by their names (bf16; vectors may be f32), and l2b_model_finalize checks
+ * that all are there.  config_out (may be NULL) receives dim, vocab_size, n_layers, seq_len. */
+int32_t l2b_model_load_dir(const char* dir, int32_t seq_len, int32_t compute_type, int32_t device, l2b_config* config_out, l2b_model** model);
+int32_t l2b_model_create_stack(const char* config_json, int32_t seq_len, int32_t compute_type, int32_t device, l2b_config* config_out, l2b_model** model);
+int32_t l2b_model_upload_named(l2b_model* model, const char* name, int32_t type, const void* host_data, const int64_t* shape, int32_t ndim);
+
 /* ---- tokenizer (host only; ids are 0-based here, bos / eos included) ------------------------------------
  * BPETokenizer (src/tokenizer.jl:3-9) from a vocabulary as a file stores it: token i is
  * token_bytes[offsets[i] .. offsets[i+1]); scores may be NULL (all 0); token_types (LLAMA_TOKEN_TYPE, src/load_gguf.jl:44-52)
@@ -194,6 +207,11 @@ int32_t l2b_session_last_phase_ms(l2b_session* session, float* prompt_ms, float*
  * Afterwards the session holds the logits of the last prompt position (l2b_session_logits); *next (may be NULL) is their argmax.
  * Continue with l2b_decode_next(session, chosen_token, pos0 + n, ...). */
 int32_t l2b_prefill(l2b_session* session, const int32_t* tokens, int32_t n, int32_t pos0, int32_t* next);
+/* Feed a portion of a sequence and read logits at chosen places: tokens[0..n-1] at positions pos0 .. pos0+n-1 on top of what the
+ * session holds for positions below pos0; want[0..n_want-1] (ascending, 0..n-1) are the places whose logits go to
+ * host_logits [n_want][vocab_size].  Portions may be cut anywhere (a portion of one token is a decode step). */
+int32_t l2b_session_extend(l2b_session* session, const int32_t* tokens, int32_t n, int32_t pos0, const int32_t* want, int32_t n_want,
+                           float* host_logits);
 /* *min_tokens > 0: runs of at least that many prompt positions that are all followed by a prompt token go through the
  * many-token pass (every matrix product one launch of the tensor-core GEMM, tcgen05 + TMA, 20 tokens per pass over a weight
  * tile; up to 240 tokens per pass over the layers).  0: not available for this model (needs q4_K / q5_K layer matrices, three
@@ -213,7 +231,8 @@ int32_t l2b_session_kernels_per_token(l2b_session* session, int32_t* n);
 /* ---- batched decode (no counterpart in the reference, whose `sample` serves one prompt) ----------------------
  * n_seq independent sequences (2 .. 240), each with its own zeroed KV cache of seq_len positions, advanced one position per
  * call: every matrix is streamed once per 20 sequences by the tensor-core GEMM instead of once per sequence.  Needs q4_K /
- * q5_K layer matrices (the classifier may be q6_K), three activation planes, one GPU; otherwise L2B_ERR_UNSUPPORTED_TYPE.
+ * q5_K layer matrices (the classifier may be q6_K), three activation planes, one GPU, or a layer-stack model; otherwise
+ * L2B_ERR_UNSUPPORTED_TYPE.
  * l2b_batch_decode_next: tokens[i] is fed at position positions[i] of sequence i (transformer!, src/inference.jl:222-315, for
  * each); next_tokens[i] = argmax of its logits (src/inference.jl:360); host_logits (optional) receives [n_seq][vocab_size]. */
 int32_t l2b_batch_create(l2b_model* model, int32_t n_seq, l2b_batch** batch);

@@ -11,7 +11,7 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.environ.get("L2B_LIBRARY") or os.path.join(_HERE, "libllama2_b200.so")
 
 OK, ERR_BAD_ARG, ERR_UNSUPPORTED_TYPE, ERR_CUDA, _ERR_UNUSED, ERR_TIMEOUT, ERR_OOM, ERR_STATE, ERR_NO_DEVICE = range(9)
-TYPE_F32, TYPE_Q4_K, TYPE_Q5_K, TYPE_Q6_K = 0, 12, 13, 14
+TYPE_F32, TYPE_Q4_K, TYPE_Q5_K, TYPE_Q6_K, TYPE_BF16 = 0, 12, 13, 14, 30
 BLOCK_BYTES = {TYPE_Q4_K: 144, TYPE_Q5_K: 176, TYPE_Q6_K: 210}
 (ROLE_TOKEN_EMBEDDING, ROLE_RMS_ATT, ROLE_WQ, ROLE_WK, ROLE_WV, ROLE_WO, ROLE_RMS_FFN, ROLE_W1, ROLE_W2, ROLE_W3,
  ROLE_RMS_FINAL, ROLE_OUTPUT) = range(12)
@@ -76,6 +76,10 @@ _SIGNATURES = {
     "l2b_tokenizer_info": ([_P, C.POINTER(C.c_int32), C.POINTER(C.c_int32), C.POINTER(C.c_int32)], C.c_int32),
     "l2b_tokenizer_token": ([_P, C.c_int32, C.POINTER(_P), C.POINTER(C.c_int64)], C.c_int32),
     "l2b_tokenizer_encode": ([_P, _P, C.c_int64, C.c_int32, _P, C.c_int64, C.POINTER(C.c_int64)], C.c_int32),
+    "l2b_model_load_dir": ([C.c_char_p, C.c_int32, C.c_int32, C.c_int32, _P, C.POINTER(_P)], C.c_int32),
+    "l2b_model_create_stack": ([C.c_char_p, C.c_int32, C.c_int32, C.c_int32, _P, C.POINTER(_P)], C.c_int32),
+    "l2b_model_upload_named": ([_P, C.c_char_p, C.c_int32, _P, _P, C.c_int32], C.c_int32),
+    "l2b_session_extend": ([_P, _P, C.c_int32, C.c_int32, _P, C.c_int32, _P], C.c_int32),
     "l2b_prefill": ([_P, _P, C.c_int32, C.c_int32, C.POINTER(C.c_int32)], C.c_int32),
     "l2b_session_prefill_gemm": ([_P, C.POINTER(C.c_int32)], C.c_int32),
     "l2b_session_prefill_pairs": ([_P, C.POINTER(C.c_int32)], C.c_int32),

@@ -11,6 +11,9 @@
 #include <vector>
 
 #include "gguf_reader.h"
+#include "host_common.h"
+#include "safetensors.h"
+#include "stack.h"
 #include "attention.cuh"
 #include "fused_matvec.cuh"
 #include "sampling.cuh"
@@ -26,28 +29,12 @@ using namespace l2b;
 // ---------------------------------------------------------------------------------------------
 static thread_local std::string g_last_error;
 
-static int32_t fail(int32_t code, const std::string& msg) {
+int32_t fail(int32_t code, const std::string& msg) {
     g_last_error = msg;
     return code;
 }
 // for the other translation units of the library (tokenizer.cpp)
 int32_t l2b_internal_fail(int32_t code, const std::string& msg) { return fail(code, msg); }
-
-#define CU(call)                                                                                         \
-    do {                                                                                                 \
-        cudaError_t e_ = (call);                                                                         \
-        if (e_ != cudaSuccess) {                                                                         \
-            (void)cudaGetLastError();                                                                    \
-            return fail(e_ == cudaErrorMemoryAllocation ? L2B_ERR_OOM : L2B_ERR_CUDA,                    \
-                        std::string(#call) + ": " + cudaGetErrorString(e_) + " (" + __FILE__ + ":" + std::to_string(__LINE__) + ")"); \
-        }                                                                                                \
-    } while (0)
-
-#define L2B_TRY(expr)              \
-    do {                           \
-        int32_t s_ = (expr);       \
-        if (s_ != L2B_OK) return s_; \
-    } while (0)
 
 static int32_t require_device() {
     int n = 0;
@@ -84,7 +71,6 @@ static void free_matrix(DevMatrix& m) {
 // Copy one matrix to the device (repacking q6_K).  `rows` x `in` weights.
 // Rows longer than one stage (in > 4096) are re-ordered into column panels on the device (panelize_kernel) unless
 // `panels` is false (matrices that are read row by row: the embedding table, plain dequantisation).
-static long env_long(const char* name, long dflt);
 // Stage width for a matrix: 16 super-blocks, or 8 where a row is exactly one 16-wide stage and 16-wide ring slots would leave
 // fewer than four slots beside the activation planes (then only one group of consumer warps could work, on a ring three deep;
 // measured on the q6_K classifier 128256 x 4096: 101.7 -> 88.3 us).  Longer rows keep 16: with 8-block stages the q5_K
@@ -164,52 +150,6 @@ static int32_t upload_matrix(DevMatrix& m, int type, const void* host, int64_t i
 // ---------------------------------------------------------------------------------------------
 // kernel launch helpers
 // ---------------------------------------------------------------------------------------------
-struct DeviceInfo {
-    int sms = 148;
-    int max_smem_optin = 227 * 1024;
-};
-
-static int32_t query_device(DeviceInfo& di) {
-    int dev = 0;
-    CU(cudaGetDevice(&dev));
-    CU(cudaDeviceGetAttribute(&di.sms, cudaDevAttrMultiProcessorCount, dev));
-    CU(cudaDeviceGetAttribute(&di.max_smem_optin, cudaDevAttrMaxSharedMemoryPerBlockOptin, dev));
-    return L2B_OK;
-}
-
-// cluster > 1: the grid is launched as thread-block clusters of that many consecutive blocks.
-template <typename Kernel, typename Params>
-static cudaError_t launch_kernel(Kernel k, dim3 grid, dim3 block, size_t smem, cudaStream_t st, bool pdl, const Params& prm, int cluster = 1) {
-    cudaLaunchConfig_t cfg;
-    memset(&cfg, 0, sizeof(cfg));
-    cfg.gridDim = grid;
-    cfg.blockDim = block;
-    cfg.dynamicSmemBytes = smem;
-    cfg.stream = st;
-    cudaLaunchAttribute attr[2];
-    int n = 0;
-    if (pdl) {
-        attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-        attr[n].val.programmaticStreamSerializationAllowed = 1;
-        ++n;
-    }
-    if (cluster > 1) {
-        attr[n].id = cudaLaunchAttributeClusterDimension;
-        attr[n].val.clusterDim.x = (unsigned)cluster;
-        attr[n].val.clusterDim.y = 1;
-        attr[n].val.clusterDim.z = 1;
-        ++n;
-    }
-    cfg.attrs = attr;
-    cfg.numAttrs = n;
-    return cudaLaunchKernelEx(&cfg, k, prm);
-}
-
-static long env_long(const char* name, long dflt) {
-    const char* v = getenv(name);
-    return v && *v ? atol(v) : dflt;
-}
-
 // A fused matrix-vector launch, fully planned on the host.
 struct MvLaunch {
     MvParams p;
@@ -422,22 +362,6 @@ static int choose_gq(int n_heads, int n_kv) {
 }
 
 // ---- tensor-core GEMM (kq_gemm.cuh): host side ----------------------------------------------------------
-// cuTensorMapEncodeTiled comes from the driver; the library links the runtime only, so the entry point is looked up.
-typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
-                                  const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-static EncodeTiledFn encode_tiled_fn() {
-    static EncodeTiledFn fn = [] {
-        void* f = nullptr;
-        cudaDriverEntryPointQueryResult qr;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &f, cudaEnableDefault, &qr) != cudaSuccess || qr != cudaDriverEntryPointSuccess) {
-            (void)cudaGetLastError();
-            f = nullptr;
-        }
-        return (EncodeTiledFn)f;
-    }();
-    return fn;
-}
-
 static bool gemm_supported(const DevMatrix& w) { return (w.type == T_Q4_K || w.type == T_Q5_K) && w.out >= 1; }
 
 // The matrix as a 3-D byte tensor [panels][rows][panel row bytes]; box = one super-block of 128 rows.
@@ -546,6 +470,7 @@ struct l2b_model {
     std::vector<LayerW> layers;
     bool finalized = false;
     int planes = 3;
+    StackModel* stack = nullptr;  // a layer-stack model (stack.h): its weights; the fields above that describe llama weights stay empty
     // tensor parallelism: this process holds rank `rank` of `tp` shards.  Heads are split by kv group, the ffn by
     // hidden units; wo and w2 are split along their INPUT (block columns), so their outputs are partial sums.
     int tp = 1, rank = 0;
@@ -556,6 +481,7 @@ struct l2b_model {
 
 struct l2b_session {
     l2b_model* model = nullptr;
+    StackSession* stack = nullptr;  // layer-stack models: caches and activations
     cudaStream_t stream = nullptr;
     bool own_stream = false;
     DeviceInfo di;
@@ -595,6 +521,9 @@ struct l2b_session {
     size_t tp_bytes = 0;
     unsigned* tp_epoch = nullptr;  // tokens completed (device word)
     uint8_t* peer_mem[MV_MAX_TP] = {nullptr};  // [r]: rank r's tp_mem as seen from this process ([rank] = own)
+    // logits of chosen rows of a many-token pass (l2b_session_extend): row numbers and results, allocated on first use
+    int* want_index = nullptr;
+    float* want_logits = nullptr;
     // many-token prompt pass through the tensor-core GEMM (kq_gemm.cuh): buffers for PF_MAX_TOK tokens, allocated on first use
     bool pf_checked = false, pf_ok = false;
     GemmBufs pf;
@@ -688,6 +617,7 @@ static int32_t upload_vector(float*& dst, const void* host, int64_t n) {
 extern "C" int32_t l2b_model_upload_tensor(l2b_model* m, int32_t role, int32_t layer, int32_t type, const void* host, int64_t in_dim, int64_t out_dim) {
     if (!m || !host) return fail(L2B_ERR_BAD_ARG, "null argument");
     if (m->finalized) return fail(L2B_ERR_STATE, "model already finalized");
+    if (m->stack) return fail(L2B_ERR_STATE, "a layer-stack model takes its tensors by name (l2b_model_upload_named)");
     CU(cudaSetDevice(m->device));
     const l2b_config& c = m->cfg;
     const int hs = c.dim / c.n_heads, kv_dim = hs * c.n_kv_heads;
@@ -757,6 +687,11 @@ extern "C" int32_t l2b_model_upload_tensor(l2b_model* m, int32_t role, int32_t l
 
 extern "C" int32_t l2b_model_finalize(l2b_model* m) {
     if (!m) return fail(L2B_ERR_BAD_ARG, "null model");
+    if (m->stack) {
+        L2B_TRY(stack_model_finalize(m->stack));
+        m->finalized = true;
+        return L2B_OK;
+    }
     if (!m->tok_emb.present() || !m->output.present() || !m->rms_final) return fail(L2B_ERR_STATE, "token embedding, output weight or final norm missing");
     for (int l = 0; l < m->cfg.n_layers; ++l) {
         const LayerW& w = m->layers[l];
@@ -775,6 +710,7 @@ extern "C" int32_t l2b_model_finalize(l2b_model* m) {
 extern "C" int32_t l2b_model_destroy(l2b_model* m) {
     if (!m) return L2B_OK;
     cudaSetDevice(m->device);
+    stack_model_free(m->stack);
     free_matrix(m->tok_emb);
     free_matrix(m->output);
     if (m->rms_final) cudaFree(m->rms_final);
@@ -790,6 +726,10 @@ extern "C" int32_t l2b_model_destroy(l2b_model* m) {
 
 extern "C" int32_t l2b_model_weight_bytes(const l2b_model* m, int64_t* bytes) {
     if (!m || !bytes) return fail(L2B_ERR_BAD_ARG, "null argument");
+    if (m->stack) {
+        *bytes = stack_model_bytes_per_token(m->stack);
+        return L2B_OK;
+    }
     int64_t b = m->output.file_bytes + (int64_t)m->cfg.dim * 4;  // output matrix + final norm gain
     b += m->tok_emb.file_bytes / m->cfg.vocab_size;               // one embedding row
     for (const auto& w : m->layers)
@@ -935,10 +875,87 @@ extern "C" int32_t l2b_model_load_gguf(const char* path, int32_t seq_len, int32_
 }
 
 // ---------------------------------------------------------------------------------------------
+// layer-stack models: config.json + model.safetensors (stack.h)
+// ---------------------------------------------------------------------------------------------
+extern "C" int32_t l2b_model_create_stack(const char* config_json, int32_t seq_len, int32_t compute_type, int32_t device, l2b_config* config_out, l2b_model** out) {
+    if (!config_json || !out) return fail(L2B_ERR_BAD_ARG, "null argument");
+    *out = nullptr;
+    if (seq_len <= 0) return fail(L2B_ERR_BAD_ARG, "seq_len must be positive");
+    if (compute_type != L2B_TYPE_BF16 && compute_type != L2B_TYPE_F32) return fail(L2B_ERR_UNSUPPORTED_TYPE, "layer-stack models compute in bf16 or f32");
+    l2b_model* m = new l2b_model();
+    auto run = [&]() -> int32_t {
+        StackConfig check;  // a configuration error is reported whether or not there is a device
+        std::string err;
+        if (!parse_stack_config(config_json, strlen(config_json), check, err)) return fail(L2B_ERR_BAD_ARG, err);
+        L2B_TRY(require_device());
+        if (device >= 0) CU(cudaSetDevice(device));
+        CU(cudaGetDevice(&m->device));
+        L2B_TRY(stack_model_create(config_json, strlen(config_json), compute_type == L2B_TYPE_F32, &m->stack));
+        l2b_config& c = m->cfg;
+        memset(&c, 0, sizeof(c));
+        c.dim = check.width; c.vocab_size = check.vocab; c.n_layers = (int32_t)check.layers.size(); c.seq_len = seq_len;
+        c.hidden_dim = check.layers[0].ff; c.n_heads = c.n_kv_heads = check.layers[0].mix.heads;
+        c.rope_freq_base = (float)check.layers[0].mix.rot.base;
+        c.device = device; c.tp_size = 1;
+        return L2B_OK;
+    };
+    const int32_t st = run();
+    if (st != L2B_OK) {
+        l2b_model_destroy(m);
+        return st;
+    }
+    if (config_out) *config_out = m->cfg;
+    *out = m;
+    return L2B_OK;
+}
+
+extern "C" int32_t l2b_model_upload_named(l2b_model* m, const char* name, int32_t type, const void* host, const int64_t* shape, int32_t ndim) {
+    if (!m || !name || !host || (ndim > 0 && !shape) || ndim < 0) return fail(L2B_ERR_BAD_ARG, "null argument");
+    if (!m->stack) return fail(L2B_ERR_STATE, "this model takes its tensors by role (l2b_model_upload_tensor)");
+    if (m->finalized) return fail(L2B_ERR_STATE, "model already finalized");
+    CU(cudaSetDevice(m->device));
+    return stack_model_upload(m->stack, name, type, host, shape, ndim);
+}
+
+extern "C" int32_t l2b_model_load_dir(const char* dir, int32_t seq_len, int32_t compute_type, int32_t device, l2b_config* config_out, l2b_model** out) {
+    if (!dir || !out) return fail(L2B_ERR_BAD_ARG, "null argument");
+    *out = nullptr;
+    const std::string base = std::string(dir) + "/";
+    std::string json;
+    FILE* fp = fopen((base + "config.json").c_str(), "rb");
+    if (!fp) return fail(L2B_ERR_BAD_ARG, "cannot open " + base + "config.json");
+    char buf[4096];
+    for (size_t n; (n = fread(buf, 1, sizeof(buf), fp)) > 0;) json.append(buf, n);
+    fclose(fp);
+    l2b_model* m = nullptr;
+    L2B_TRY(l2b_model_create_stack(json.c_str(), seq_len, compute_type, device, config_out, &m));
+    auto run = [&]() -> int32_t {
+        SafeTensorsFile f;
+        if (!f.open(base + "model.safetensors")) return fail(L2B_ERR_BAD_ARG, f.error());
+        for (const auto& e : f.tensors()) {
+            if (!stack_model_has(m->stack, e.first)) continue;  // nothing of the design reads it
+            const int type = e.second.dtype == "BF16" ? L2B_TYPE_BF16 : e.second.dtype == "F32" ? L2B_TYPE_F32 : -1;
+            L2B_TRY(l2b_model_upload_named(m, e.first.c_str(), type, e.second.data, e.second.shape.data(), (int32_t)e.second.shape.size()));
+        }
+        return l2b_model_finalize(m);
+    };
+    const int32_t st = run();
+    if (st != L2B_OK) {
+        l2b_model_destroy(m);
+        return st;
+    }
+    *out = m;
+    return L2B_OK;
+}
+
+// ---------------------------------------------------------------------------------------------
 // session
 // ---------------------------------------------------------------------------------------------
 static void session_free(l2b_session* s) {
     if (!s) return;
+    stack_session_free(s->stack);
+    if (s->want_index) cudaFree(s->want_index);
+    if (s->want_logits) cudaFree(s->want_logits);
     if (s->graph) cudaGraphExecDestroy(s->graph);
     if (s->graph2) cudaGraphExecDestroy(s->graph2);
     void* bufs[] = {s->x, s->q, s->att, s->tickets, s->hb, s->logits, s->kc, s->vc, s->part_m, s->part_l, s->part_acc, s->amax_val, s->amax_idx,
@@ -970,15 +987,34 @@ static void session_free(l2b_session* s) {
 struct l2b_session;
 static cudaError_t cudaLaunchKernelEx_embed(const l2b_model* m, l2b_session* s, int blocks, int threads, int second);
 
+// Next token (inference.jl:354-368) and advance, from the logits and `nparts` per-block maxima.
+static int32_t enqueue_finalize(l2b_session* s, int nparts) {
+    FinalizeParams f;
+    memset(&f, 0, sizeof(f));
+    f.logits = s->logits; f.vocab = s->model->cfg.vocab_size;
+    f.amax_val = s->amax_val; f.amax_idx = s->amax_idx; f.nparts = nparts;
+    f.ctl = s->ctl; f.prompt = s->prompt; f.out_tokens = s->out_tokens; f.advance = 1; f.next_token = s->next_token;
+    f.tp_epoch = s->tp_epoch;
+    f.status = s->status;
+    CU(launch_kernel(finalize_token_kernel, dim3(1), dim3(FIN_THREADS), 0, s->stream, true, f));
+    return L2B_OK;
+}
+
 // Enqueue every kernel of one token on the session stream (this is what the graph captures).
 // nb = 2: a pass over TWO consecutive prompt positions (pos, pos + 1), both of which are followed by a prompt token:
 // every matrix is streamed once for both, no logits are computed and nothing is sampled.
 static int32_t enqueue_token(l2b_session* s, int* nlaunch, int nb = 1) {
     const l2b_model* m = s->model;
     const l2b_config& c = m->cfg;
+    int count = 0, last_grid = 0;
+    if (m->stack) {  // layer-stack models: their own kernels up to the logits, then the same choice of the next token
+        L2B_TRY(stack_enqueue_token(s->stack, &s->ctl->token, &s->ctl->pos, s->logits, s->amax_val, s->amax_idx, s->stream, &count, &last_grid));
+        L2B_TRY(enqueue_finalize(s, last_grid));
+        if (nlaunch) *nlaunch = count + 1;
+        return L2B_OK;
+    }
     const int hs = c.dim / c.n_heads;
     const size_t kvl = kv_layer_elems(m);
-    int count = 0, last_grid = 0;
     bool first = true;
     auto mv = [&](MvLaunch& L) -> int32_t {
         L.planes = m->planes;
@@ -1169,18 +1205,8 @@ static int32_t enqueue_token(l2b_session* s, int* nlaunch, int nb = 1) {
         L2B_TRY(mv(L));
         norm_done();
     }
-    // --- next token (inference.jl:354-368) and advance
-    {
-        FinalizeParams f;
-        memset(&f, 0, sizeof(f));
-        f.logits = s->logits; f.vocab = c.vocab_size;
-        f.amax_val = s->amax_val; f.amax_idx = s->amax_idx; f.nparts = last_grid;
-        f.ctl = s->ctl; f.prompt = s->prompt; f.out_tokens = s->out_tokens; f.advance = 1; f.next_token = s->next_token;
-        f.tp_epoch = s->tp_epoch;
-        f.status = s->status;
-        CU(launch_kernel(finalize_token_kernel, dim3(1), dim3(FIN_THREADS), 0, s->stream, true, f));
-        ++count;
-    }
+    L2B_TRY(enqueue_finalize(s, last_grid));
+    ++count;
     if (nlaunch) *nlaunch = count;
     return L2B_OK;
 }
@@ -1236,6 +1262,7 @@ static int32_t build_token_kernel(l2b_session* s) {
     const l2b_model* m = s->model;
     const l2b_config& c = m->cfg;
     s->tk = false;
+    if (m->stack) return L2B_OK;
     // Opt-in (L2B_TOKEN_KERNEL=1): measured on a B200 the single launch is not faster than the chain of launches yet (the
     // consumer warps, not the hand-over between kernels, bound the token), so the chain stays the default.
     if (m->tp != 1 || env_long("L2B_TOKEN_KERNEL", 0) == 0) return L2B_OK;
@@ -1478,7 +1505,7 @@ static int32_t capture_token_graph(l2b_session* s) {
     }
     }
     // Second graph: two prompt positions per pass.  Needs k-quant matrices throughout, three planes, one GPU.
-    if (s->model->tp == 1 && s->model->planes == 3 && s->all_kquant && !s->trace && env_long("L2B_PREFILL_PAIRS", 1) != 0) {
+    if (!s->model->stack && s->model->tp == 1 && s->model->planes == 3 && s->all_kquant && !s->trace && env_long("L2B_PREFILL_PAIRS", 1) != 0) {
         cudaGraph_t g2 = nullptr;
         int n2 = 0;
         CU(cudaStreamBeginCapture(s->stream, cudaStreamCaptureModeThreadLocal));
@@ -1500,6 +1527,8 @@ static int32_t capture_token_graph(l2b_session* s) {
     return L2B_OK;
 }
 
+constexpr int STACK_PASS_ROWS = 2048;  // rows of a many-token pass of a layer-stack model
+
 extern "C" int32_t l2b_session_create(l2b_model* m, void* stream, l2b_session** out) {
     if (!m || !out) return fail(L2B_ERR_BAD_ARG, "null argument");
     *out = nullptr;
@@ -1507,7 +1536,7 @@ extern "C" int32_t l2b_session_create(l2b_model* m, void* stream, l2b_session** 
     CU(cudaSetDevice(m->device));
     L2B_TRY(check_kernel_attrs());
     const l2b_config& c = m->cfg;
-    const int hs = c.dim / c.n_heads;
+    const int hs = m->stack ? 0 : c.dim / c.n_heads;
     l2b_session* s = new l2b_session();
     s->model = m;
     int32_t st = L2B_OK;
@@ -1521,6 +1550,30 @@ extern "C" int32_t l2b_session_create(l2b_model* m, void* stream, l2b_session** 
         else {
             CU(cudaStreamCreateWithFlags(&s->stream, cudaStreamNonBlocking));
             s->own_stream = true;
+        }
+        // loop state, logits and what the choice of the next token needs: every model
+        CU(cudaMalloc(&s->logits, (size_t)c.vocab_size * 4));
+        CU(cudaMalloc(&s->amax_val, (size_t)s->di.sms * 4));
+        CU(cudaMalloc(&s->amax_idx, (size_t)s->di.sms * 4));
+        CU(cudaMalloc(&s->ctl, sizeof(Control)));
+        CU(cudaMalloc(&s->next_token, 8));  // next token and status word side by side: one copy brings both back
+        s->status = s->next_token + 1;
+        CU(cudaMalloc(&s->prompt, (size_t)c.seq_len * 4));
+        CU(cudaMalloc(&s->out_tokens, (size_t)c.seq_len * 4));
+        CU(cudaMallocHost(&s->h_ctl, sizeof(Control)));
+        CU(cudaMallocHost(&s->h_small, 16));
+        CU(cudaEventCreate(&s->ev0));
+        CU(cudaEventCreate(&s->ev1));
+        CU(cudaEventCreate(&s->ev_mid));
+        CU(cudaMemsetAsync(s->status, 0, 4, s->stream));
+        CU(cudaMemsetAsync(s->ctl, 0, sizeof(Control), s->stream));
+        CU(cudaMemsetAsync(s->prompt, 0, (size_t)c.seq_len * 4, s->stream));
+        if (m->stack) {
+            StackSessionInfo info;
+            info.seq_len = c.seq_len;
+            info.max_rows = std::min(c.seq_len, STACK_PASS_ROWS);
+            L2B_TRY(stack_session_create(m->stack, info, s->di, s->stream, &s->stack));
+            return capture_token_graph(s);
         }
         s->gq = choose_gq(m->l_heads, m->l_kv);
         // blocks per head group in the attention launches: whole clusters for the decode kernel (L2B_ATTN_SPLITS is rounded up)
@@ -1540,31 +1593,15 @@ extern "C" int32_t l2b_session_create(l2b_model* m, void* stream, l2b_session** 
         CU(cudaMalloc(&s->att, (size_t)m->l_qdim() * 4 * 2));
         CU(cudaMalloc(&s->tickets, (size_t)c.n_heads * 4 * 2));
         CU(cudaMalloc(&s->hb, (size_t)m->l_hidden * 4 * 2));
-        CU(cudaMalloc(&s->logits, (size_t)c.vocab_size * 4));
         CU(cudaMalloc(&s->kc, kvl * c.n_layers * 4));
         CU(cudaMalloc(&s->vc, kvl * c.n_layers * 4));
         // (room for 32 splits, the most any launch uses: the token kernel chooses its own split count)
         CU(cudaMalloc(&s->part_m, (size_t)m->l_heads * 32 * 4 * 2));
         CU(cudaMalloc(&s->part_l, (size_t)m->l_heads * 32 * 4 * 2));
         CU(cudaMalloc(&s->part_acc, (size_t)m->l_heads * 32 * hs * 4 * 2));
-        CU(cudaMalloc(&s->amax_val, (size_t)s->di.sms * 4));
-        CU(cudaMalloc(&s->amax_idx, (size_t)s->di.sms * 4));
-        CU(cudaMalloc(&s->ctl, sizeof(Control)));
-        CU(cudaMalloc(&s->next_token, 8));  // next token and status word side by side: one copy brings both back
-        s->status = s->next_token + 1;
-        CU(cudaMalloc(&s->prompt, (size_t)c.seq_len * 4));
-        CU(cudaMalloc(&s->out_tokens, (size_t)c.seq_len * 4));
-        CU(cudaMallocHost(&s->h_ctl, sizeof(Control)));
-        CU(cudaMallocHost(&s->h_small, 16));
-        CU(cudaEventCreate(&s->ev0));
-        CU(cudaEventCreate(&s->ev1));
-        CU(cudaEventCreate(&s->ev_mid));
         CU(cudaMemsetAsync(s->kc, 0, kvl * c.n_layers * 4, s->stream));
         CU(cudaMemsetAsync(s->vc, 0, kvl * c.n_layers * 4, s->stream));
-        CU(cudaMemsetAsync(s->status, 0, 4, s->stream));
         CU(cudaMemsetAsync(s->tickets, 0, (size_t)c.n_heads * 4 * 2, s->stream));
-        CU(cudaMemsetAsync(s->ctl, 0, sizeof(Control), s->stream));
-        CU(cudaMemsetAsync(s->prompt, 0, (size_t)c.seq_len * 4, s->stream));
         std::vector<float> cs;
         rope_table_host(cs, c.seq_len, hs, c.rope_freq_base);
         CU(cudaMalloc(&s->rope_cs, cs.size() * 4));
@@ -1605,6 +1642,11 @@ extern "C" int32_t l2b_session_create(l2b_model* m, void* stream, l2b_session** 
 extern "C" int32_t l2b_session_reset(l2b_session* s) {
     if (!s) return fail(L2B_ERR_BAD_ARG, "null session");
     CU(cudaSetDevice(s->model->device));
+    if (s->stack) {
+        L2B_TRY(stack_session_reset(s->stack, s->stream));
+        CU(cudaStreamSynchronize(s->stream));
+        return L2B_OK;
+    }
     const size_t bytes = kv_layer_elems(s->model) * s->model->cfg.n_layers * 4;
     CU(cudaMemsetAsync(s->kc, 0, bytes, s->stream));
     CU(cudaMemsetAsync(s->vc, 0, bytes, s->stream));
@@ -1709,6 +1751,7 @@ static int32_t run_one(l2b_session* s, int token, int pos, float temperature, do
 // Needs q4_K / q5_K layer matrices, three activation planes, one GPU; otherwise the caller uses the decode passes.
 constexpr int PF_MAX_TOK = 240;
 constexpr int PF_MIN_TOK = 12;
+constexpr int STACK_MIN_ROWS = 2;  // layer-stack models
 
 // Every layer for n tokens whose residual-stream rows are in B.x.  One sequence: token t sits at position pos0 + t and the
 // layer's caches are kc / vc + l * layer_stride.  Batched decode (pos_list non-null): token t is the next position pos_list[t]
@@ -1785,6 +1828,7 @@ static bool alloc_gemm_bufs(const l2b_model* m, GemmBufs& B, size_t T) {
 }
 
 static bool prefill_gemm_eligible(l2b_session* s) {
+    if (s->stack) return true;
     if (s->pf_checked) return s->pf_ok;
     s->pf_checked = true;
     // (a pass that cannot get its buffers leaves prompts to the decode passes)
@@ -1792,11 +1836,21 @@ static bool prefill_gemm_eligible(l2b_session* s) {
     return s->pf_ok;
 }
 
+// Shortest run of forced positions that goes through a many-token pass.
+static int min_pass_tokens(const l2b_session* s) { return s->stack ? STACK_MIN_ROWS : PF_MIN_TOK; }
+
 // Positions pos0 .. pos0 + n - 1 of the prompt already in s->prompt (device), 2 <= n <= PF_MAX_TOK; all enqueued on the session stream.
 static int32_t enqueue_prefill_gemm(l2b_session* s, int pos0, int n) {
     const l2b_model* m = s->model;
     const l2b_config& c = m->cfg;
     cudaStream_t st = s->stream;
+    if (s->stack) {
+        L2B_TRY(stack_enqueue_rows(s->stack, s->prompt + pos0, n, pos0, nullptr, s->status, st, &s->last_launches));
+        fill_forced_kernel<<<1, 256, 0, st>>>(s->prompt, s->out_tokens, pos0, n);
+        CU(cudaGetLastError());
+        ++s->last_launches;
+        return L2B_OK;
+    }
     embed_rows_kernel<<<dim3(std::max(1, std::min(16, c.dim / 256)), n), 256, 0, st>>>(m->tok_emb.type, m->tok_emb.data, m->tok_emb.d6, s->prompt + pos0, c.dim,
                                                                                       c.vocab_size, s->pf.x);
     CU(cudaGetLastError());
@@ -1811,9 +1865,9 @@ static int32_t enqueue_prefill_gemm(l2b_session* s, int pos0, int n) {
 // token is host_tokens[to - base].  Many-token passes where possible, the decode graphs for the rest.
 static int32_t enqueue_forced_positions(l2b_session* s, int from, int to, const int32_t* host_prompt_at_from) {
     int i = from;
-    if (to - from >= PF_MIN_TOK && prefill_gemm_eligible(s)) {
+    if (to - from >= min_pass_tokens(s) && prefill_gemm_eligible(s)) {
         while (i < to) {
-            const int n = std::min(PF_MAX_TOK, to - i);
+            const int n = std::min(s->stack ? stack_session_max_rows(s->stack) : PF_MAX_TOK, to - i);
             L2B_TRY(enqueue_prefill_gemm(s, i, n));
             i += n;
         }
@@ -1953,10 +2007,67 @@ extern "C" int32_t l2b_prefill(l2b_session* s, const int32_t* tokens, int32_t n,
     return check_status_word(s);
 }
 
+// Feed a portion of n tokens at positions pos0 .. and return the logits at n_want places among them (ascending).  Layer-stack
+// models: one many-token pass (a single token: the captured one-position graph, as in generation), then the classifier on the
+// wanted rows.  Other models: the prompt passes of l2b_prefill up to each wanted place, whose position takes the graph.
+extern "C" int32_t l2b_session_extend(l2b_session* s, const int32_t* tokens, int32_t n, int32_t pos0, const int32_t* want, int32_t n_want, float* host_logits) {
+    if (!s || !tokens || n_want < 0 || (n_want > 0 && (!want || !host_logits))) return fail(L2B_ERR_BAD_ARG, "null argument");
+    const l2b_config& c = s->model->cfg;
+    if (n < 1 || pos0 < 0 || (int64_t)pos0 + n > c.seq_len) return fail(L2B_ERR_BAD_ARG, "positions pos0 .. pos0+n-1 must lie in 0..seq_len-1");
+    for (int i = 0; i < n; ++i)
+        if (tokens[i] < 0 || tokens[i] >= c.vocab_size) return fail(L2B_ERR_BAD_ARG, "token id out of range");
+    for (int i = 0; i < n_want; ++i)
+        if (want[i] < (i ? want[i - 1] + 1 : 0) || want[i] >= n) return fail(L2B_ERR_BAD_ARG, "wanted places must ascend and lie in 0..n-1");
+    const size_t row = (size_t)c.vocab_size;
+    if (!s->stack || n == 1) {
+        int done = 0;
+        for (int i = 0; i <= n_want; ++i) {
+            const int upto = i < n_want ? want[i] + 1 : n;
+            if (upto == done) break;
+            L2B_TRY(l2b_prefill(s, tokens + done, upto - done, pos0 + done, nullptr));
+            if (i < n_want) L2B_TRY(l2b_session_logits(s, host_logits + i * row));
+            done = upto;
+        }
+        return L2B_OK;
+    }
+    CU(cudaSetDevice(s->model->device));
+    constexpr int WANT_ROWS = 128;  // rows per classifier pass
+    const int max_rows = stack_session_max_rows(s->stack);
+    if (n_want > 0 && !s->want_index) {
+        CU(cudaMalloc(&s->want_index, (size_t)WANT_ROWS * 4));
+        CU(cudaMalloc(&s->want_logits, (size_t)WANT_ROWS * row * 4));
+    }
+    s->last_launches = 0;
+    CU(cudaEventRecord(s->ev0, s->stream));
+    CU(cudaMemcpyAsync(s->prompt + pos0, tokens, (size_t)n * 4, cudaMemcpyHostToDevice, s->stream));
+    int w = 0;
+    for (int i = 0; i < n; i += max_rows) {
+        const int k = std::min(max_rows, n - i);
+        L2B_TRY(stack_enqueue_rows(s->stack, s->prompt + pos0 + i, k, pos0 + i, nullptr, s->status, s->stream, &s->last_launches));
+        while (w < n_want && want[w] < i + k) {
+            int idx[WANT_ROWS], nw = 0;
+            while (nw < WANT_ROWS && w + nw < n_want && want[w + nw] < i + k) {
+                idx[nw] = want[w + nw] - i;
+                ++nw;
+            }
+            CU(cudaMemcpyAsync(s->want_index, idx, (size_t)nw * 4, cudaMemcpyHostToDevice, s->stream));
+            L2B_TRY(stack_enqueue_logits(s->stack, s->want_index, nw, s->want_logits, s->status, s->stream, &s->last_launches));
+            CU(cudaMemcpyAsync(host_logits + w * row, s->want_logits, (size_t)nw * row * 4, cudaMemcpyDeviceToHost, s->stream));
+            CU(cudaStreamSynchronize(s->stream));
+            w += nw;
+        }
+    }
+    CU(cudaMemcpyAsync(&s->h_small[1], s->status, 4, cudaMemcpyDeviceToHost, s->stream));
+    CU(cudaEventRecord(s->ev1, s->stream));
+    CU(cudaStreamSynchronize(s->stream));
+    CU(cudaEventElapsedTime(&s->last_ms, s->ev0, s->ev1));
+    return check_status_word(s);
+}
+
 extern "C" int32_t l2b_session_prefill_gemm(l2b_session* s, int32_t* min_tokens) {
     if (!s || !min_tokens) return fail(L2B_ERR_BAD_ARG, "null argument");
     CU(cudaSetDevice(s->model->device));
-    *min_tokens = prefill_gemm_eligible(s) ? PF_MIN_TOK : 0;
+    *min_tokens = prefill_gemm_eligible(s) ? min_pass_tokens(s) : 0;
     return L2B_OK;
 }
 
@@ -2028,9 +2139,9 @@ extern "C" int32_t l2b_session_read(l2b_session* s, int32_t which, float* host_o
     const float* src = nullptr;
     int64_t len = 0;
     switch (which) {
-        case 0: src = s->x; len = c.dim; break;
-        case 2: src = s->q; len = c.dim; break;
-        case 5: src = s->hb; len = c.hidden_dim; break;
+        case 0: src = s->stack ? stack_session_residual(s->stack) : s->x; len = c.dim; break;
+        case 2: if (s->stack) return fail(L2B_ERR_BAD_ARG, "not kept by layer-stack models"); src = s->q; len = c.dim; break;
+        case 5: if (s->stack) return fail(L2B_ERR_BAD_ARG, "not kept by layer-stack models"); src = s->hb; len = c.hidden_dim; break;
         case 6: src = s->logits; len = c.vocab_size; break;
         default: return fail(L2B_ERR_BAD_ARG, "unknown buffer id");
     }
@@ -2069,6 +2180,7 @@ extern "C" int32_t l2b_session_kernels_per_token(l2b_session* s, int32_t* n) {
 // ---------------------------------------------------------------------------------------------
 struct l2b_batch {
     l2b_model* model = nullptr;
+    StackSession* stack = nullptr;       // layer-stack models: caches of all sequences and activations
     int n_seq = 0;
     cudaStream_t stream = nullptr;
     DeviceInfo di;
@@ -2083,6 +2195,7 @@ struct l2b_batch {
 
 static void batch_free(l2b_batch* b) {
     if (!b) return;
+    stack_session_free(b->stack);
     free_gemm_bufs(b->B);
     void* bufs[] = {b->kc, b->vc, b->rope_cs, b->logits, b->tokens, b->pos, b->next, b->status};
     for (void* p : bufs)
@@ -2099,23 +2212,16 @@ extern "C" int32_t l2b_batch_create(l2b_model* m, int32_t n_seq, l2b_batch** out
     if (n_seq < 2 || n_seq > PF_MAX_TOK) return fail(L2B_ERR_BAD_ARG, "a batch holds 2 .. " + std::to_string(PF_MAX_TOK) + " sequences");
     CU(cudaSetDevice(m->device));
     L2B_TRY(check_kernel_attrs());
-    if (!gemm_layers_supported(m))
+    if (!m->stack && !gemm_layers_supported(m))
         return fail(L2B_ERR_UNSUPPORTED_TYPE, "batched decode needs q4_K / q5_K layer matrices, three activation planes and one GPU");
     const l2b_config& c = m->cfg;
-    const int hs = c.dim / c.n_heads;
+    const int hs = m->stack ? 0 : c.dim / c.n_heads;
     l2b_batch* b = new l2b_batch();
     b->model = m;
     b->n_seq = n_seq;
     auto run = [&]() -> int32_t {
         L2B_TRY(query_device(b->di));
         CU(cudaStreamCreateWithFlags(&b->stream, cudaStreamNonBlocking));
-        b->gq = choose_gq(c.n_heads, c.n_kv_heads);
-        if (!alloc_gemm_bufs(m, b->B, (size_t)n_seq)) return fail(L2B_ERR_OOM, "out of device memory for the batch buffers");
-        const size_t cache = kv_layer_elems(m) * c.n_layers * (size_t)n_seq * 4;
-        CU(cudaMalloc(&b->kc, cache));
-        CU(cudaMalloc(&b->vc, cache));
-        CU(cudaMemsetAsync(b->kc, 0, cache, b->stream));
-        CU(cudaMemsetAsync(b->vc, 0, cache, b->stream));
         CU(cudaMalloc(&b->logits, (size_t)n_seq * c.vocab_size * 4));
         CU(cudaMalloc(&b->tokens, (size_t)n_seq * 4));
         CU(cudaMalloc(&b->pos, (size_t)n_seq * 4));
@@ -2123,6 +2229,22 @@ extern "C" int32_t l2b_batch_create(l2b_model* m, int32_t n_seq, l2b_batch** out
         CU(cudaMalloc(&b->status, 4));
         CU(cudaMemsetAsync(b->status, 0, 4, b->stream));
         CU(cudaMallocHost(&b->h_io, (size_t)(3 * n_seq + 1) * 4));
+        if (m->stack) {
+            StackSessionInfo info;
+            info.seq_len = c.seq_len;
+            info.n_seq = info.max_rows = n_seq;
+            info.decode = false;
+            L2B_TRY(stack_session_create(m->stack, info, b->di, b->stream, &b->stack));
+            CU(cudaStreamSynchronize(b->stream));
+            return L2B_OK;
+        }
+        b->gq = choose_gq(c.n_heads, c.n_kv_heads);
+        if (!alloc_gemm_bufs(m, b->B, (size_t)n_seq)) return fail(L2B_ERR_OOM, "out of device memory for the batch buffers");
+        const size_t cache = kv_layer_elems(m) * c.n_layers * (size_t)n_seq * 4;
+        CU(cudaMalloc(&b->kc, cache));
+        CU(cudaMalloc(&b->vc, cache));
+        CU(cudaMemsetAsync(b->kc, 0, cache, b->stream));
+        CU(cudaMemsetAsync(b->vc, 0, cache, b->stream));
         std::vector<float> cs;
         rope_table_host(cs, c.seq_len, hs, c.rope_freq_base);
         CU(cudaMalloc(&b->rope_cs, cs.size() * 4));
@@ -2150,6 +2272,11 @@ extern "C" int32_t l2b_batch_destroy(l2b_batch* b) {
 extern "C" int32_t l2b_batch_reset(l2b_batch* b) {
     if (!b) return fail(L2B_ERR_BAD_ARG, "null batch");
     CU(cudaSetDevice(b->model->device));
+    if (b->stack) {
+        L2B_TRY(stack_session_reset(b->stack, b->stream));
+        CU(cudaStreamSynchronize(b->stream));
+        return L2B_OK;
+    }
     const size_t cache = kv_layer_elems(b->model) * b->model->cfg.n_layers * (size_t)b->n_seq * 4;
     CU(cudaMemsetAsync(b->kc, 0, cache, b->stream));
     CU(cudaMemsetAsync(b->vc, 0, cache, b->stream));
@@ -2157,21 +2284,11 @@ extern "C" int32_t l2b_batch_reset(l2b_batch* b) {
     return L2B_OK;
 }
 
-extern "C" int32_t l2b_batch_decode_next(l2b_batch* b, const int32_t* tokens, const int32_t* positions, int32_t* next_tokens, float* host_logits) {
-    if (!b || !tokens || !positions || !next_tokens) return fail(L2B_ERR_BAD_ARG, "null argument");
+// Every sequence's token through the llama layers and the classifier: b->tokens, b->pos -> b->logits.
+static int32_t enqueue_batch_llama(l2b_batch* b, cudaStream_t st) {
     const l2b_model* m = b->model;
     const l2b_config& c = m->cfg;
     const int n = b->n_seq;
-    for (int i = 0; i < n; ++i) {
-        if (tokens[i] < 0 || tokens[i] >= c.vocab_size) return fail(L2B_ERR_BAD_ARG, "token id out of range");
-        if (positions[i] < 0 || positions[i] >= c.seq_len) return fail(L2B_ERR_BAD_ARG, "position out of range (seq_len)");
-    }
-    CU(cudaSetDevice(m->device));
-    cudaStream_t st = b->stream;
-    memcpy(b->h_io, tokens, (size_t)n * 4);
-    memcpy(b->h_io + n, positions, (size_t)n * 4);
-    CU(cudaMemcpyAsync(b->tokens, b->h_io, (size_t)n * 4, cudaMemcpyHostToDevice, st));
-    CU(cudaMemcpyAsync(b->pos, b->h_io + n, (size_t)n * 4, cudaMemcpyHostToDevice, st));
     embed_rows_kernel<<<dim3(std::max(1, std::min(16, c.dim / 256)), n), 256, 0, st>>>(m->tok_emb.type, m->tok_emb.data, m->tok_emb.d6, b->tokens, c.dim,
                                                                                       c.vocab_size, b->B.x);
     CU(cudaGetLastError());
@@ -2196,6 +2313,30 @@ extern "C" int32_t l2b_batch_decode_next(l2b_batch* b, const int32_t* tokens, co
             L2B_TRY(plan_matvec(L, b->di));
             CU(launch_matvec(L, st, false));
         }
+    }
+    return L2B_OK;
+}
+
+extern "C" int32_t l2b_batch_decode_next(l2b_batch* b, const int32_t* tokens, const int32_t* positions, int32_t* next_tokens, float* host_logits) {
+    if (!b || !tokens || !positions || !next_tokens) return fail(L2B_ERR_BAD_ARG, "null argument");
+    const l2b_model* m = b->model;
+    const l2b_config& c = m->cfg;
+    const int n = b->n_seq;
+    for (int i = 0; i < n; ++i) {
+        if (tokens[i] < 0 || tokens[i] >= c.vocab_size) return fail(L2B_ERR_BAD_ARG, "token id out of range");
+        if (positions[i] < 0 || positions[i] >= c.seq_len) return fail(L2B_ERR_BAD_ARG, "position out of range (seq_len)");
+    }
+    CU(cudaSetDevice(m->device));
+    cudaStream_t st = b->stream;
+    memcpy(b->h_io, tokens, (size_t)n * 4);
+    memcpy(b->h_io + n, positions, (size_t)n * 4);
+    CU(cudaMemcpyAsync(b->tokens, b->h_io, (size_t)n * 4, cudaMemcpyHostToDevice, st));
+    CU(cudaMemcpyAsync(b->pos, b->h_io + n, (size_t)n * 4, cudaMemcpyHostToDevice, st));
+    if (b->stack) {
+        L2B_TRY(stack_enqueue_rows(b->stack, b->tokens, n, 0, b->pos, b->status, st, nullptr));
+        L2B_TRY(stack_enqueue_logits(b->stack, nullptr, n, b->logits, b->status, st, nullptr));
+    } else {
+        L2B_TRY(enqueue_batch_llama(b, st));
     }
     argmax_rows_kernel<<<n, 1024, 0, st>>>(b->logits, c.vocab_size, b->next, b->status);
     CU(cudaGetLastError());

@@ -267,29 +267,6 @@ constexpr int ATTN_CL = 8;  // blocks per cluster (the portable maximum)
 constexpr int ATTN_DW = 8;  // warps per block
 constexpr int ATTN_CLUSTER_POS = ATTN_CL * ATTN_DW * ATTN_UNROLL;  // positions a cluster takes in one batch per warp
 
-__device__ __forceinline__ void cluster_sync_all() {
-    asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
-}
-__device__ __forceinline__ uint32_t cluster_map(const void* smem_ptr, uint32_t rank) {  // the same variable in block `rank` of the cluster
-    uint32_t r;
-    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(smem_u32(smem_ptr)), "r"(rank));
-    return r;
-}
-__device__ __forceinline__ void st_cluster_f32(uint32_t addr, float v) { asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(addr), "f"(v) : "memory"); }
-__device__ __forceinline__ void st_cluster_f32x4(uint32_t addr, float4 v) {
-    asm volatile("st.shared::cluster.v4.f32 [%0], {%1, %2, %3, %4};" ::"r"(addr), "f"(v.x), "f"(v.y), "f"(v.z), "f"(v.w) : "memory");
-}
-__device__ __forceinline__ float ld_cluster_f32(uint32_t addr) {
-    float v;
-    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr) : "memory");
-    return v;
-}
-__device__ __forceinline__ float4 ld_cluster_f32x4(uint32_t addr) {
-    float4 v;
-    asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(addr) : "memory");
-    return v;
-}
-
 // PDL = false: launched without a programmatic dependency (no previous kernel to wait for).
 template <int GQ, bool PDL>
 __device__ __forceinline__ void attention_decode_body(const AttnParams& p) {

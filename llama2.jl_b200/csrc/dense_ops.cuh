@@ -1,0 +1,139 @@
+// Arithmetic shared by the kernels of the layer-stack models (stack.cu): 8 stored values at a time as f32, activations, rotary
+// pairs, and the epilogues of the dense matrix products.
+#pragma once
+#include <cuda_bf16.h>
+
+#include "common.cuh"
+
+namespace l2b {
+
+typedef __nv_bfloat16 bf16;
+
+// eight consecutive values (16-byte aligned bf16, 32-byte aligned f32) as f32
+struct Vec8 {
+    float v[8];
+};
+__device__ __forceinline__ Vec8 unpack8(uint4 r) {
+    Vec8 o;
+    const uint32_t w[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        o.v[2 * i] = __uint_as_float(w[i] << 16);
+        o.v[2 * i + 1] = __uint_as_float(w[i] & 0xFFFF0000u);
+    }
+    return o;
+}
+template <typename T>
+struct Raw8;  // the same eight values as loaded, before conversion
+template <>
+struct Raw8<bf16> {
+    uint4 r;
+    __device__ __forceinline__ void zero() { r = make_uint4(0u, 0u, 0u, 0u); }
+    __device__ __forceinline__ void load(const bf16* p) { r = __ldcg(reinterpret_cast<const uint4*>(p)); }
+    __device__ __forceinline__ Vec8 get() const { return unpack8(r); }
+};
+template <>
+struct Raw8<float> {
+    float4 a, b;
+    __device__ __forceinline__ void zero() { a = b = make_float4(0.f, 0.f, 0.f, 0.f); }
+    __device__ __forceinline__ void load(const float* p) {
+        a = __ldcg(reinterpret_cast<const float4*>(p));
+        b = __ldcg(reinterpret_cast<const float4*>(p) + 1);
+    }
+    __device__ __forceinline__ Vec8 get() const {
+        Vec8 o;
+        o.v[0] = a.x; o.v[1] = a.y; o.v[2] = a.z; o.v[3] = a.w;
+        o.v[4] = b.x; o.v[5] = b.y; o.v[6] = b.z; o.v[7] = b.w;
+        return o;
+    }
+};
+
+__device__ __forceinline__ void put(float* p, float v) { *p = v; }
+__device__ __forceinline__ void put(bf16* p, float v) { *p = __float2bfloat16_rn(v); }
+__device__ __forceinline__ float as_stored(const float*, float v) { return v; }  // the value a store of that type keeps
+__device__ __forceinline__ float as_stored(const bf16*, float v) { return __bfloat162float(__float2bfloat16_rn(v)); }
+
+__device__ __forceinline__ float gelu_tanh(float z) {
+    const float t = tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z));  // sqrt(2 / pi)
+    return 0.5f * z * (1.f + t);
+}
+__device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float dynamic_tanh(float x, float alpha, float w, float b) { return fmaf(tanhf(alpha * x), w, b); }
+
+// element d of a vector whose first rdims elements are interleaved rotary pairs; get(i) reads element i, cs = this position's row
+template <class Get>
+__device__ __forceinline__ float rotary_element(int d, int rdims, const float2* cs, Get get) {
+    if (d >= rdims) return get(d);
+    const float2 t = __ldg(cs + (d >> 1));
+    return (d & 1) ? get(d) * t.x + get(d - 1) * t.y : get(d) * t.x - get(d + 1) * t.y;
+}
+
+// What happens to a result of a dense product W x before it is stored.
+enum : int {
+    DE_STORE = 0,     // y[t][f] f32
+    DE_RESIDUAL = 1,  // y[t][f] += f32
+    DE_GEGLU = 2,     // act[t][f] = gelu_tanh(gate) * up (two weight rows per result)
+    DE_SIDE = 3,      // act[t][f] = gelu_tanh(v) * e, e = element e_off + f of the token's row of an embedding table
+    DE_LOGITS = 4,    // as DE_STORE, and the block's first maximum
+    DE_STORE_ACT = 5, // act[t][f]
+    DE_STORE_T = 6    // act[f][t] (transposed)
+};
+struct DenseEpilogue {
+    int kind;
+    float* y;
+    void* act;
+    int ld;               // elements between rows of y / act
+    const bf16* etab;     // DE_SIDE
+    int e_ld, e_off;
+    const int* tokens;    // DE_SIDE: token of result row t
+    int vocab;            // DE_SIDE: rows of the table (an id outside it contributes zero)
+};
+__device__ __forceinline__ float side_value(const DenseEpilogue& e, int t, int f) {
+    const int tok = __ldcg(e.tokens + t);
+    return tok >= 0 && tok < e.vocab ? __bfloat162float(e.etab[(size_t)tok * e.e_ld + e.e_off + f]) : 0.f;
+}
+template <typename AT>
+__device__ __forceinline__ void dense_epilogue(const DenseEpilogue& e, int t, int f, float v, float v2) {
+    const size_t o = (size_t)t * e.ld + f;
+    AT* act = static_cast<AT*>(e.act);
+    switch (e.kind) {
+        case DE_STORE: case DE_LOGITS: e.y[o] = v; break;
+        case DE_RESIDUAL: e.y[o] += v; break;
+        case DE_GEGLU: put(act + o, gelu_tanh(v) * v2); break;
+        case DE_SIDE: put(act + o, gelu_tanh(v) * side_value(e, t, f)); break;
+        case DE_STORE_ACT: put(act + o, v); break;
+        case DE_STORE_T: put(act + (size_t)f * e.ld + t, v); break;
+    }
+}
+
+// Pending changes of the residual stream that the next reader applies: x' = x + y / rms(y) * side_w + step.
+struct ResidualUpdate {
+    const float* y;       // output of the per-layer token input, before its norm (null: none)
+    const float* side_w;  // that norm's weight
+    float eps;
+    const float* step;    // vector added at the beginning of a loop pass (null: none)
+};
+// The norm in front of a dense product.
+struct NormParams {
+    int kind;             // 0: none; 1: dynamic tanh
+    float alpha;
+    const float* w;
+    const float* b;
+};
+__device__ __forceinline__ float apply_norm(const NormParams& n, float x, int i) {
+    return n.kind ? dynamic_tanh(x, n.alpha, __ldg(n.w + i), __ldg(n.b + i)) : x;
+}
+
+// Sum over the threads of a block of NW warps; every thread gets it.  s holds NW floats and may be reused after the next barrier.
+template <int NW>
+__device__ __forceinline__ float block_sum_all(float v, float* s) {
+    v = warp_sum(v);
+    if ((threadIdx.x & 31) == 0) s[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float t = 0.f;
+#pragma unroll
+    for (int i = 0; i < NW; ++i) t += s[i];
+    return t;
+}
+
+}  // namespace l2b

@@ -8,6 +8,7 @@ reference is 1-based Julia).  Weight matrices are given as the reference stores 
 matrices are `QuantMatrix` (raw super-block bytes, out rows of in/256 blocks).
 """
 import ctypes as C
+import json
 import random
 import sys
 import time
@@ -95,11 +96,63 @@ class TransformerWeights:
     output_weight: Matrix
 
 
+@dataclass
+class StackConfig:
+    """A layer-stack model's configuration: the parsed config.json (`raw`; "architecture" names the design), the positions a
+    session holds, and what it computes in ("bfloat16" or "float32")."""
+    raw: dict
+    seq_len: int
+    compute: str = "bfloat16"
+
+    @property
+    def architecture(self):
+        return self.raw["architecture"]
+
+    @property
+    def vocab_size(self):
+        return self.raw["vocab"]
+
+    @property
+    def dim(self):
+        return self.raw["width"]
+
+    @property
+    def n_layers(self):
+        return len(self.raw["layers"])
+
+    def compute_type(self):
+        return compute_type(self.compute)
+
+    def __str__(self):
+        return f"StackConfig(\n  architecture   = {self.architecture},\n  seq_len        = {self.seq_len},\n  compute        = {self.compute},\n)"
+
+
+def compute_type(name: str) -> int:
+    try:
+        return {"bfloat16": L.TYPE_BF16, "float32": L.TYPE_F32}[name]
+    except KeyError:
+        raise ValueError(f"compute type {name!r}: layer-stack models compute in 'bfloat16' or 'float32'") from None
+
+
+class StackWeights(dict):
+    """A layer-stack model's weights by tensor name: uint16 arrays are bf16 bit patterns, float32 arrays are rounded to bf16
+    (nearest even) when they are matrices and kept as they are when they are vectors."""
+
+
+def bf16_bits(a: np.ndarray) -> np.ndarray:
+    """float32 -> bf16 bit patterns, round to nearest even (finite values)."""
+    u = np.ascontiguousarray(a, dtype=np.float32).view(np.uint32)
+    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
+
+
 class _DeviceModel:
     """Owns an l2b_model and one l2b_session (RunState)."""
 
     def __init__(self, config: ModelConfig, weights: TransformerWeights, act_planes=0, device=-1, stream=None, tp_size=1, tp_rank=0):
         lib = L.lib()
+        if isinstance(config, StackConfig):
+            self._init_stack(config, weights, device, stream, tp_size)
+            return
         cfg = L.Config(dim=config.dim, hidden_dim=config.hidden_dim, n_layers=config.n_layers, n_heads=config.n_heads,
                        n_kv_heads=config.n_kv_heads, vocab_size=config.vocab_size, seq_len=config.seq_len,
                        rope_freq_base=float(config.rope_freq_base), rope_is_neox=int(bool(config.rope_is_neox)),
@@ -129,6 +182,39 @@ class _DeviceModel:
         except Exception:
             self.close()
             raise
+
+    def _init_stack(self, config: StackConfig, weights: StackWeights, device, stream, tp_size):
+        if tp_size != 1:
+            raise L.L2BError(L.ERR_UNSUPPORTED_TYPE, "layer-stack models run on one GPU")
+        lib = L.lib()
+        self.model, self.session = C.c_void_p(), C.c_void_p()
+        L.check(lib.l2b_model_create_stack(json.dumps(config.raw).encode(), config.seq_len, config.compute_type(), device, None, C.byref(self.model)))
+        try:
+            for name, a in weights.items():
+                a = np.asarray(a)
+                data = np.ascontiguousarray(a) if a.dtype == np.uint16 else bf16_bits(a) if a.ndim == 2 else np.ascontiguousarray(a, dtype=np.float32)
+                kind = L.TYPE_BF16 if data.dtype == np.uint16 else L.TYPE_F32
+                shape = (C.c_int64 * max(a.ndim, 1))(*a.shape)
+                L.check(lib.l2b_model_upload_named(self.model, name.encode(), kind, L.ptr(data), shape, a.ndim))
+            L.check(lib.l2b_model_finalize(self.model))
+            L.check(lib.l2b_session_create(self.model, stream, C.byref(self.session)))
+        except Exception:
+            self.close()
+            raise
+
+    @classmethod
+    def from_dir(cls, path: str, config: StackConfig, device=-1, stream=None):
+        """config.json and model.safetensors read by the library itself (l2b_model_load_dir)."""
+        lib = L.lib()
+        self = cls.__new__(cls)
+        self.model, self.session = C.c_void_p(), C.c_void_p()
+        L.check(lib.l2b_model_load_dir(path.encode(), config.seq_len, config.compute_type(), device, None, C.byref(self.model)))
+        try:
+            L.check(lib.l2b_session_create(self.model, stream, C.byref(self.session)))
+        except Exception:
+            self.close()
+            raise
+        return self
 
     @classmethod
     def from_gguf(cls, path: str, seq_len: int, act_planes=0, device=-1, stream=None, tp_size=1, tp_rank=0):
@@ -235,11 +321,15 @@ class RunState:
     """src/inference.jl:72-100: the per-call state.  Here it is a handle on the device session;
     creating one zeroes the KV cache exactly like `RunState(config)`."""
 
-    def __init__(self, model: LanguageModel):
+    def __init__(self, model: LanguageModel, session=None):
+        """`session`: a session handle of the caller's instead of the model's own."""
         self.model = model
-        self.session = model.device_model().session
-        L.check(L.lib().l2b_session_reset(self.session))
+        self.session = model.device_model().session if session is None else session
+        self.reset()
         self.logits = np.zeros(model.config.vocab_size, dtype=np.float32)
+
+    def reset(self):
+        L.check(L.lib().l2b_session_reset(self.session))
 
 
 class BatchRunState:
@@ -313,6 +403,16 @@ def prefill(s: RunState, tokens, pos0: int = 0) -> int:
     L.check(L.lib().l2b_prefill(s.session, L.ptr(t), t.size, int(pos0), C.byref(nxt)))
     L.check(L.lib().l2b_session_logits(s.session, L.ptr(s.logits)))
     return nxt.value
+
+
+def extend(s: RunState, tokens, pos0: int, want=()) -> np.ndarray:
+    """A portion of a sequence on top of what the state holds: tokens at positions pos0.., logits [len(want), vocab] at the places
+    `want` (ascending, counted within the portion)."""
+    t = np.ascontiguousarray(tokens, dtype=np.int32)
+    w = np.ascontiguousarray(want, dtype=np.int32)
+    out = np.zeros((w.size, s.model.config.vocab_size), dtype=np.float32)
+    L.check(L.lib().l2b_session_extend(s.session, L.ptr(t), t.size, int(pos0), L.ptr(w), w.size, L.ptr(out)))
+    return out
 
 
 def generate(model: LanguageModel, prompt_tokens, n_positions: int, temperature: float = 0.0, seed: int = 0):
