@@ -3,7 +3,7 @@ counter-based generators of the test-support library (libl2b_synth.so, include/l
 import numpy as np
 
 from . import _lib as L
-from .model import ModelConfig, QuantMatrix, TransformerLayerWeights, TransformerWeights
+from .model import ModelConfig, QuantMatrix, StackWeights, TransformerLayerWeights, TransformerWeights
 
 Q4, Q5, Q6, F32 = L.TYPE_Q4_K, L.TYPE_Q5_K, L.TYPE_Q6_K, L.TYPE_F32
 
@@ -86,3 +86,73 @@ def scaled(spec, n_layers=None, vocab_size=None, seq_len=None):
 def prompt_tokens(spec, seed):
     c = spec["config"]
     return tokens(spec["n_prompt"], seed ^ 0xABCDEF, 3, c.vocab_size)
+
+
+# ---- layer-stack models ------------------------------------------------------------------------------------
+def _savozen(width, ff, heads, dim, rot, vdim, rank, side, layers, vocab):
+    mix = dict(heads=heads, dim=dim, rot_dim=rot, vdim=vdim, kv_rank=rank, scale=(dim + rot) ** -0.5, rot=dict(base=500000.0, dims=rot))
+    return dict(architecture="Savozen", embedding=dict(scale=1.0), norm=dict(eps=1e-5), vocab=vocab, width=width, token_side=dict(dim=side),
+                layers=[dict(type="latent_attention", mixer=mix, mlp=dict(kind="dense", ff=ff)) for _ in range(layers)])
+
+
+# Layers of the size of a real model's, and the llama shape of equal width, feed-forward and head count that they are measured beside.
+SAVOZEN_SIZES = {
+    "2k": dict(raw=_savozen(2048, 8192, 16, 128, 64, 128, 512, 128, 8, 32768), llama=ModelConfig(2048, 8192, 8, 16, 16, 32768, 2048, 500000.0, False)),
+    "4k": dict(raw=_savozen(4096, 14336, 32, 128, 64, 128, 512, 256, 8, 32768), llama=ModelConfig(4096, 14336, 8, 32, 8, 32768, 2048, 500000.0, False)),
+}
+
+
+def bf16_matrix(out_dim, in_dim, seed):
+    """Random bf16 bit patterns with magnitudes around 1/64 (two octaves, both signs)."""
+    bits = np.random.default_rng(seed).integers(0, 65536, size=(out_dim, in_dim), dtype=np.uint16)
+    return (bits & np.uint16(0x80FF)) | np.uint16(0x3C00)
+
+
+def savozen_weights(raw, seed):
+    """Weights of a Savozen configuration by tensor name; layers of one size share their host arrays (every layer has its own device
+    copy)."""
+    D, V, shared = raw["width"], raw["vocab"], {}
+
+    def mat(key, out, inn):
+        if (key, out, inn) not in shared:
+            shared[(key, out, inn)] = bf16_matrix(out, inn, seed + len(shared))
+        return shared[(key, out, inn)]
+    w = StackWeights(embed=mat("embed", V, D), head=mat("head", V, D))
+
+    def norm(name):
+        w[name] = np.ones(D, np.float32)
+        w[name + ".b"] = np.zeros(D, np.float32)
+        w[name + ".alpha"] = np.float32(0.5)
+    norm("final.norm")
+    if raw.get("loop"):
+        w["loop.step"] = normal_f32(raw["loop"]["times"] * D, seed, 0.1).reshape(-1, D)
+    side = raw["token_side"]["dim"] if raw.get("token_side") else 0
+    if side:
+        w["side.embed"] = mat("side.embed", V, side * len(raw["layers"]))
+    for i, l in enumerate(raw["layers"]):
+        p, m = f"l{i}.", l["mixer"]
+        H, d, r, dv, R = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+        norm(p + "norm1")
+        for name, out, inn in (("q", H * (d + r), D), ("dkv", R + r, D), ("uk", H * d, R), ("uv", H * dv, R), ("g", H * dv, D), ("o", D, H * dv)):
+            w[p + "mix." + name] = mat(name, out, inn)
+        w[p + "mix.dkv.norm"] = np.ones(R, np.float32)
+        w[p + "mix.sink"] = np.zeros(H, np.float32)
+        if l["mlp"]:
+            norm(p + "norm2")
+            ff = l["mlp"]["ff"]
+            w[p + "mlp.gate"], w[p + "mlp.up"], w[p + "mlp.down"] = mat("gate", ff, D), mat("up", ff, D), mat("down", D, ff)
+        if side:
+            w[p + "side.gate"], w[p + "side.proj"], w[p + "side.norm"] = mat("sgate", side, D), mat("sproj", D, side), np.full(D, 0.5, np.float32)
+    return w
+
+
+def savozen_flops_per_token(raw, npos):
+    """Multiply-adds x 2 of one prompt token's matrix products, and of its attention over npos positions (expanded form)."""
+    D, side = raw["width"], raw["token_side"]["dim"] if raw.get("token_side") else 0
+    dense = att = 0
+    for l in raw["layers"]:
+        m = l["mixer"]
+        H, d, r, dv, R = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+        dense += D * (H * (d + r) + R + r + H * dv) + H * (d + dv) * R + H * dv * D + 3 * D * (l["mlp"]["ff"] if l["mlp"] else 0) + 2 * D * side
+        att += H * npos * (d + r + dv)
+    return 2 * dense, 2 * att

@@ -1,6 +1,9 @@
 """Plain restatement of the Savozen design for the tests: numpy, float64, one function per mechanism, no cache (every call
 sees whole sequences).  It shares no code with the library; weights are a dict name -> float array, the configuration is the
-parsed config.json."""
+parsed config.json.
+
+`operand` is applied to what enters a matrix product or the cache.  The identity gives the exact result; rounding to bf16 gives
+what a 16-bit computation of the same design may lose."""
 import math
 
 import numpy as np
@@ -40,31 +43,35 @@ def sink_softmax(scores, sink):
     return e / (e.sum(-1, keepdims=True) + np.exp(sink[:, None, None] - m))
 
 
-def latent_attention(h, w, m, eps, positions=None):
+def exact(x):
+    return x
+
+
+def latent_attention(h, w, m, eps, positions=None, operand=exact):
     """h [tokens, width]; w: this mixer's tensors by their short names; m: the mixer's sizes."""
     T = h.shape[0]
     H, d, r, dv, R = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
     pos = np.arange(T, dtype=np.float64) if positions is None else positions
     q = (h @ w["q"].T).reshape(T, H, d + r).transpose(1, 0, 2)
-    q_plain = q[..., :d]
-    q_rot = rotate_interleaved(q[..., d:], pos, m["rot"]["base"], m["rot"]["dims"])
+    q_plain = operand(q[..., :d])
+    q_rot = operand(rotate_interleaved(q[..., d:], pos, m["rot"]["base"], m["rot"]["dims"]))
     down = h @ w["dkv"].T
-    c = rms_norm(down[:, :R], w["dkv.norm"], eps)
-    k_rot = rotate_interleaved(down[:, R:], pos, m["rot"]["base"], m["rot"]["dims"])
-    k = (c @ w["uk"].T).reshape(T, H, d).transpose(1, 0, 2)
-    v = (c @ w["uv"].T).reshape(T, H, dv).transpose(1, 0, 2)
+    c = operand(rms_norm(down[:, :R], w["dkv.norm"], eps))
+    k_rot = operand(rotate_interleaved(down[:, R:], pos, m["rot"]["base"], m["rot"]["dims"]))
+    k = operand(c @ w["uk"].T).reshape(T, H, d).transpose(1, 0, 2)
+    v = operand(c @ w["uv"].T).reshape(T, H, dv).transpose(1, 0, 2)
     s = (q_plain @ k.transpose(0, 2, 1) + q_rot @ k_rot.T[None]) * m["scale"]
     s = np.where(np.tril(np.ones((T, T), bool))[None], s, -np.inf)
-    o = (sink_softmax(s, w["sink"]) @ v).transpose(1, 0, 2).reshape(T, H * dv)
-    return (o * sigmoid(h @ w["g"].T)) @ w["o"].T
+    o = (operand(sink_softmax(s, w["sink"])) @ v).transpose(1, 0, 2).reshape(T, H * dv)
+    return operand(o * sigmoid(h @ w["g"].T)) @ w["o"].T
 
 
-def gated_mlp(h, gate, up, down):
-    return (gelu_tanh(h @ gate.T) * (h @ up.T)) @ down.T
+def gated_mlp(h, gate, up, down, operand=exact):
+    return operand(gelu_tanh(h @ gate.T) * (h @ up.T)) @ down.T
 
 
-def token_side(x, e, gate, proj, norm, eps):
-    y = (gelu_tanh(x @ gate.T) * e) @ proj.T
+def token_side(x, e, gate, proj, norm, eps, operand=exact):
+    y = operand(gelu_tanh(operand(x) @ gate.T) * e) @ proj.T
     return x + rms_norm(y, norm, eps)
 
 
@@ -81,14 +88,14 @@ def layer_runs(cfg):
     return runs + [(i, None) for i in range(b, n)]
 
 
-def forward(cfg, weights, tokens, residuals=None):
+def forward(cfg, weights, tokens, residuals=None, operand=exact):
     """Logits [tokens, vocab]; residuals (a list, optional) receives the residual stream after every layer run."""
     W = {k: np.asarray(v, np.float64) for k, v in weights.items()}
     tokens = np.asarray(tokens)
     eps = cfg["norm"]["eps"]
 
     def norm(name, x):
-        return dynamic_tanh(x, W[name + ".alpha"], W[name], W[name + ".b"])
+        return operand(dynamic_tanh(x, W[name + ".alpha"], W[name], W[name + ".b"]))
     x = W["embed"][tokens] * cfg["embedding"]["scale"]
     side = cfg.get("token_side")
     for i, t in layer_runs(cfg):
@@ -96,12 +103,12 @@ def forward(cfg, weights, tokens, residuals=None):
             x = x + W["loop.step"][t]
         p = f"l{i}."
         mix = {k[len(p) + 4:]: v for k, v in W.items() if k.startswith(p + "mix.")}
-        x = x + latent_attention(norm(p + "norm1", x), mix, cfg["layers"][i]["mixer"], eps)
+        x = x + latent_attention(norm(p + "norm1", x), mix, cfg["layers"][i]["mixer"], eps, operand=operand)
         if cfg["layers"][i].get("mlp"):
-            x = x + gated_mlp(norm(p + "norm2", x), W[p + "mlp.gate"], W[p + "mlp.up"], W[p + "mlp.down"])
+            x = x + gated_mlp(norm(p + "norm2", x), W[p + "mlp.gate"], W[p + "mlp.up"], W[p + "mlp.down"], operand)
         if side:
             e = W["side.embed"][tokens][:, i * side["dim"]:(i + 1) * side["dim"]]
-            x = token_side(x, e, W[p + "side.gate"], W[p + "side.proj"], W[p + "side.norm"], eps)
+            x = token_side(x, e, W[p + "side.gate"], W[p + "side.proj"], W[p + "side.norm"], eps, operand)
         if residuals is not None:
             residuals.append(x)
     return norm("final.norm", x) @ W["head"].T
