@@ -1008,7 +1008,7 @@ static int32_t enqueue_token(l2b_session* s, int* nlaunch, int nb = 1) {
     const l2b_config& c = m->cfg;
     int count = 0, last_grid = 0;
     if (m->stack) {  // layer-stack models: their own kernels up to the logits, then the same choice of the next token
-        L2B_TRY(stack_enqueue_token(s->stack, &s->ctl->token, &s->ctl->pos, s->logits, s->amax_val, s->amax_idx, s->stream, &count, &last_grid));
+        L2B_TRY(stack_enqueue_token(s->stack, &s->ctl->token, &s->ctl->pos, s->logits, s->amax_val, s->amax_idx, s->status, s->stream, &count, &last_grid));
         L2B_TRY(enqueue_finalize(s, last_grid));
         if (nlaunch) *nlaunch = count + 1;
         return L2B_OK;

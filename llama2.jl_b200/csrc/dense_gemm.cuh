@@ -2,12 +2,14 @@
 //   bf16_gemm_kernel  bf16 activations on the 5th-generation tensor cores (tcgen05 + TMA + tensor memory);
 //   f32_gemm_kernel   f32 activations on the CUDA cores in f32 (the 32-bit mode: bf16 weights are exact in f32).
 //
-// bf16_gemm_kernel: one block = 128 weight rows x BN tokens, times NA weight tiles that share the token tile (NA = 2: the next 128
+// bf16_gemm_kernel: a tile = 128 weight rows x BN tokens, times NA weight tiles that share the token tile (NA = 2: the next 128
 // rows, or the same rows of a second matrix, so that gate and up of a feed-forward unit meet in one thread).  Weight rows
 // are the M dimension: a thread of the epilogue owns one row, and consecutive lanes store consecutive results of a token.
+// Persistent: one block per SM walks tiles (token tiles innermost, so that a weight tile is read from L2 after its first use), with
+// two sets of NA x BN accumulator columns in tensor memory, so that a tile's epilogue runs beside the next tile's products.
 //   warp 0     producer: TMA tiled copies of 64-value wide operand tiles (128-byte swizzle) into a ring of stages
-//   warp 1     MMA issue: four K = 16 steps per stage and weight tile into NA x BN columns of tensor memory
-//   warps 2-5  epilogue: tcgen05.ld, then what follows the product (dense_epilogue)
+//   warp 1     MMA issue: four K = 16 steps per stage and weight tile
+//   warps 2-5  epilogue: tcgen05.ld, then what follows the product
 // Every mbarrier wait is bounded; a wait that runs out sets the status word, and the block still frees its tensor memory.
 #pragma once
 #include "dense_ops.cuh"
@@ -22,30 +24,86 @@ struct GemmDenseParams {
     int n_tok;
     int k;
     int row2;      // distance of the second weight tile's rows (128: next rows; 0: the same rows of the second matrix)
+    int mtiles, ntiles;
     int stages;
     DenseEpilogue epi;
     int* status;
 };
 __host__ __device__ constexpr int bg_stage_bytes(int BN, int NA) { return (NA * 128 + BN) * BG_KB * 2; }
 
+// 32 consecutive tokens (n of them exist) of one result row.  What has to be read is read for all of them first.
+template <int KIND>
+__device__ __forceinline__ void epilogue_tokens(const DenseEpilogue& e, int t0, int n, int f, const float (&v)[32], const float (&v2)[32]) {
+    bf16* const act = static_cast<bf16*>(e.act);
+    if (KIND == DE_RESIDUAL) {
+        float r[32];
+#pragma unroll
+        for (int k = 0; k < 32; ++k) r[k] = e.y[(size_t)(t0 + min(k, n - 1)) * e.ld + f];
+#pragma unroll
+        for (int k = 0; k < 32; ++k)
+            if (k < n) e.y[(size_t)(t0 + k) * e.ld + f] = r[k] + v[k];
+    } else if (KIND == DE_SIDE) {
+        float r[32];
+#pragma unroll
+        for (int k = 0; k < 32; ++k) r[k] = side_value(e, t0 + min(k, n - 1), f);
+#pragma unroll
+        for (int k = 0; k < 32; ++k)
+            if (k < n) put(act + (size_t)(t0 + k) * e.ld + f, gelu_tanh(v[k]) * r[k]);
+    } else if (KIND == DE_STORE_T && n == 32 && (e.ld & 7) == 0) {  // a thread's 32 tokens are contiguous
+        uint4* dst = reinterpret_cast<uint4*>(act + (size_t)f * e.ld + t0);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            uint32_t w[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const __nv_bfloat162 pk = __floats2bfloat162_rn(v[8 * k + 2 * i], v[8 * k + 2 * i + 1]);
+                w[i] = *reinterpret_cast<const uint32_t*>(&pk);
+            }
+            dst[k] = make_uint4(w[0], w[1], w[2], w[3]);
+        }
+    } else {
+#pragma unroll
+        for (int k = 0; k < 32; ++k) {
+            if (k >= n) continue;
+            if (KIND == DE_STORE) e.y[(size_t)(t0 + k) * e.ld + f] = v[k];
+            if (KIND == DE_GEGLU) put(act + (size_t)(t0 + k) * e.ld + f, gelu_tanh(v[k]) * v2[k]);
+            if (KIND == DE_STORE_ACT) put(act + (size_t)(t0 + k) * e.ld + f, v[k]);
+            if (KIND == DE_STORE_T) put(act + (size_t)f * e.ld + t0 + k, v[k]);
+        }
+    }
+}
+__device__ __forceinline__ void epilogue_tokens(const DenseEpilogue& e, int t0, int n, int f, const float (&v)[32], const float (&v2)[32]) {
+    switch (e.kind) {
+        case DE_RESIDUAL: epilogue_tokens<DE_RESIDUAL>(e, t0, n, f, v, v2); break;
+        case DE_GEGLU: epilogue_tokens<DE_GEGLU>(e, t0, n, f, v, v2); break;
+        case DE_SIDE: epilogue_tokens<DE_SIDE>(e, t0, n, f, v, v2); break;
+        case DE_STORE_ACT: epilogue_tokens<DE_STORE_ACT>(e, t0, n, f, v, v2); break;
+        case DE_STORE_T: epilogue_tokens<DE_STORE_T>(e, t0, n, f, v, v2); break;
+        default: epilogue_tokens<DE_STORE>(e, t0, n, f, v, v2); break;
+    }
+}
+
 template <int BN, int NA>
 __global__ void __launch_bounds__(BG_THREADS) bf16_gemm_kernel(const __grid_constant__ GemmDenseParams p, const __grid_constant__ CUtensorMap map_a,
                                                                const __grid_constant__ CUtensorMap map_a2, const __grid_constant__ CUtensorMap map_b) {
     extern __shared__ __align__(1024) uint8_t bg_raw[];
-    __shared__ __align__(8) uint64_t s_full[BG_MAX_STAGES], s_free[BG_MAX_STAGES], s_done;
+    __shared__ __align__(8) uint64_t s_full[BG_MAX_STAGES], s_free[BG_MAX_STAGES], s_acc[2], s_acc_free[2];
     __shared__ uint32_t s_tmem;
     uint8_t* smem = bg_raw + ((1024u - (smem_u32(bg_raw) & 1023u)) & 1023u);
-    constexpr int COLS = NA * BN < 32 ? 32 : NA * BN;
+    constexpr int COLS = 2 * NA * BN;  // 64 .. 512, a power of two
     constexpr int STAGE = bg_stage_bytes(BN, NA);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int row0 = (int)blockIdx.x * (p.row2 ? 128 * NA : 128), tok0 = (int)blockIdx.y * BN;
-    const int nk = (p.k + BG_KB - 1) / BG_KB;
+    const int tile_rows = p.row2 ? 128 * NA : 128;
+    const int nk = (p.k + BG_KB - 1) / BG_KB, tiles = p.mtiles * p.ntiles;
     if (threadIdx.x == 0) {
         for (int i = 0; i < p.stages; ++i) {
             mbar_init(s_full + i, 1);
             mbar_init(s_free + i, 1);
         }
-        mbar_init(&s_done, 1);
+        for (int i = 0; i < 2; ++i) {
+            mbar_init(s_acc + i, 1);
+            mbar_init(s_acc_free + i, 4);
+        }
         fence_barrier_init();
         fence_proxy_async();
     }
@@ -58,17 +116,21 @@ __global__ void __launch_bounds__(BG_THREADS) bf16_gemm_kernel(const __grid_cons
     if (warp == 0) {
         if (lane == 0) {
             bool ok = true;
-            for (int j = 0; j < nk && ok; ++j) {
-                const int s = j % p.stages, use = j / p.stages;
-                if (use > 0 && !mbar_wait_bounded(s_free + s, (uint32_t)((use - 1) & 1))) {
-                    ok = false;
-                    break;
+            int s = 0, use = 0;
+            for (int tile = (int)blockIdx.x; tile < tiles && ok; tile += (int)gridDim.x) {
+                const int row0 = tile / p.ntiles * tile_rows, tok0 = tile % p.ntiles * BN;
+                for (int j = 0; j < nk; ++j) {
+                    if (use > 0 && !mbar_wait_bounded(s_free + s, (uint32_t)((use - 1) & 1))) {
+                        ok = false;
+                        break;
+                    }
+                    uint8_t* st = smem + (size_t)s * STAGE;
+                    mbar_arrive_expect_tx(s_full + s, (uint32_t)STAGE);
+                    tma_load_2d(st, &map_a, j * BG_KB, row0, s_full + s);
+                    if (NA == 2) tma_load_2d(st + 128 * BG_KB * 2, &map_a2, j * BG_KB, row0 + p.row2, s_full + s);
+                    tma_load_2d(st + NA * 128 * BG_KB * 2, &map_b, j * BG_KB, tok0, s_full + s);
+                    if (++s == p.stages) s = 0, ++use;
                 }
-                uint8_t* st = smem + (size_t)s * STAGE;
-                mbar_arrive_expect_tx(s_full + s, (uint32_t)STAGE);
-                tma_load_2d(st, &map_a, j * BG_KB, row0, s_full + s);
-                if (NA == 2) tma_load_2d(st + 128 * BG_KB * 2, &map_a2, j * BG_KB, row0 + p.row2, s_full + s);
-                tma_load_2d(st + NA * 128 * BG_KB * 2, &map_b, j * BG_KB, tok0, s_full + s);
             }
             if (!ok) {
                 atomicExch(p.status, DEV_ERR_TMA_TIMEOUT);
@@ -79,69 +141,66 @@ __global__ void __launch_bounds__(BG_THREADS) bf16_gemm_kernel(const __grid_cons
         if (lane == 0) {
             constexpr uint32_t idesc = umma_idesc_bf16(128, BN);
             bool ok = true;
-            for (int j = 0; j < nk; ++j) {
-                const int s = j % p.stages;
-                if (!mbar_wait_bounded(s_full + s, (uint32_t)((j / p.stages) & 1))) {
+            int s = 0, n = 0;
+            uint32_t par = 0;
+            for (int tile = (int)blockIdx.x; tile < tiles && ok; tile += (int)gridDim.x, ++n) {
+                const int buf = n & 1;
+                if (n >= 2 && !mbar_wait_bounded(s_acc_free + buf, (uint32_t)(((n - 2) >> 1) & 1))) {
                     ok = false;
                     break;
                 }
                 tc_fence_after();
-                const uint8_t* st = smem + (size_t)s * STAGE;
-                const uint8_t* bt = st + NA * 128 * BG_KB * 2;
+                for (int j = 0; j < nk; ++j) {
+                    if (!mbar_wait_bounded(s_full + s, par)) {
+                        ok = false;
+                        break;
+                    }
+                    tc_fence_after();
+                    const uint8_t* st = smem + (size_t)s * STAGE;
+                    const uint8_t* bt = st + NA * 128 * BG_KB * 2;
 #pragma unroll
-                for (int kk = 0; kk < BG_KB / 16; ++kk)
+                    for (int kk = 0; kk < BG_KB / 16; ++kk)
 #pragma unroll
-                    for (int a = 0; a < NA; ++a)
-                        umma_bf16(tmem + (uint32_t)(a * BN), umma_desc_sw128(st + a * 128 * BG_KB * 2, kk * 32), umma_desc_sw128(bt, kk * 32), idesc,
-                                  (j | kk) ? 1u : 0u);
-                umma_commit(s_free + s);
+                        for (int a = 0; a < NA; ++a)
+                            umma_bf16(tmem + (uint32_t)((buf * NA + a) * BN), umma_desc_sw128(st + a * 128 * BG_KB * 2, kk * 32), umma_desc_sw128(bt, kk * 32), idesc,
+                                      (j | kk) ? 1u : 0u);
+                    umma_commit(s_free + s);
+                    if (++s == p.stages) s = 0, par ^= 1u;
+                }
+                if (ok) umma_commit(s_acc + buf);
             }
-            if (ok) umma_commit(&s_done);
-            else atomicExch(p.status, DEV_ERR_TMA_TIMEOUT);
+            if (!ok) atomicExch(p.status, DEV_ERR_TMA_TIMEOUT);
         }
     } else {
         const int qd = warp & 3;
         const int r = 32 * qd + lane;
-        const bool ok = __all_sync(0xffffffffu, mbar_wait_bounded(&s_done, 0u));
-        if (!ok) {
-            if (lane == 0) atomicExch(p.status, DEV_ERR_TMA_TIMEOUT);
-        } else {
+        const bool dual = NA == 2 && p.row2 == 0;
+        int n = 0;
+        bool ok = true;
+        for (int tile = (int)blockIdx.x; tile < tiles; tile += (int)gridDim.x, ++n) {
+            const int buf = n & 1, f = tile / p.ntiles * tile_rows + r, tok0 = tile % p.ntiles * BN;
+            if (!__all_sync(0xffffffffu, mbar_wait_bounded(s_acc + buf, (uint32_t)((n >> 1) & 1)))) {
+                ok = false;
+                break;
+            }
             tc_fence_after();
-            const uint32_t ta = tmem + ((uint32_t)(32 * qd) << 16);
-            const bool dual = NA == 2 && p.row2 == 0;
+            const uint32_t ta = tmem + ((uint32_t)(32 * qd) << 16) + (uint32_t)(buf * NA * BN);
 #pragma unroll 1
             for (int c = 0; c < BN; c += 32) {
-                if (tok0 + c >= p.n_tok) break;
+                const int left = min(32, p.n_tok - tok0 - c);
+                if (left <= 0) break;
                 __syncwarp();
                 float v[32], v2[32];
                 tmem_ld32f(ta + (uint32_t)c, v);
                 if (NA == 2) tmem_ld32f(ta + (uint32_t)(BN + c), v2);
-                const int n = min(32, p.n_tok - tok0 - c);
-                if (p.epi.kind == DE_STORE_T && n == 32 && (p.epi.ld & 7) == 0) {  // a thread's 32 tokens are contiguous
-#pragma unroll
-                    for (int a = 0; a < NA; ++a) {
-                        const int f = row0 + a * 128 + r;
-                        if (f >= p.rows) continue;
-                        bf16* dst = static_cast<bf16*>(p.epi.act) + (size_t)f * p.epi.ld + tok0 + c;
-#pragma unroll
-                        for (int k = 0; k < 32; k += 2) {
-                            const float x0 = a ? v2[k] : v[k], x1 = a ? v2[k + 1] : v[k + 1];
-                            *reinterpret_cast<__nv_bfloat162*>(dst + k) = __floats2bfloat162_rn(x0, x1);
-                        }
-                    }
-                    continue;
-                }
-                const int f = row0 + r;
-#pragma unroll
-                for (int k = 0; k < 32; ++k)
-                    if (k < n && f < p.rows) dense_epilogue<bf16>(p.epi, tok0 + c + k, f, v[k], NA == 2 ? v2[k] : 0.f);
-                if (NA == 2 && !dual) {
-#pragma unroll
-                    for (int k = 0; k < 32; ++k)
-                        if (k < n && f + 128 < p.rows) dense_epilogue<bf16>(p.epi, tok0 + c + k, f + 128, v2[k], 0.f);
-                }
+                if (f < p.rows) epilogue_tokens(p.epi, tok0 + c, left, f, v, v2);
+                if (NA == 2 && !dual && f + 128 < p.rows) epilogue_tokens(p.epi, tok0 + c, left, f + 128, v2, v2);
             }
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(s_acc_free + buf);
         }
+        if (!ok && lane == 0) atomicExch(p.status, DEV_ERR_TMA_TIMEOUT);
     }
     // every path ends here; the tensor memory is freed by the warp that allocated it
     tc_fence_before();

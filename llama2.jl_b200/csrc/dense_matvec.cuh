@@ -1,22 +1,27 @@
 // Matrix-vector product of the decode path of layer-stack models: bf16 weights, f32 activations and accumulation.  The counterpart
 // of fused_matvec_kernel for matrices stored in bf16.
 //
-// One block per SM, 16 warps, every block a contiguous range of rows.
-//   before the wait on the previous kernel (programmatic dependent launch): the block's rows are prefetched into L2 with a few
-//       bulk prefetches and every warp loads its first step of weights into registers -- weights are constants;
+// One block per SM, 8 consumer warps and a producer warp, every block a contiguous range of rows.
+//   producer : a stage is 4 * gs rows x cs 256-value chunks (16 KiB at most); stages come into a ring with bulk asynchronous copies
+//       (one copy of adjacent whole rows, or one per row when rows are longer than a stage).  Weights are constants, so
+//       the ring is filled, and the rows behind it are prefetched into L2, BEFORE the wait on the previous kernel
+//       (programmatic dependent launch).  The block is small enough in shared memory for the next kernel's block to do the same
+//       beside it;
 //   prologue : the input vector goes to shared memory as f32, after the pending changes of the residual stream (the normalised
 //       per-layer token input, the step vector of a loop pass) and the norm; block 0 writes the changed residual stream back
 //       to its other buffer, because the other blocks still read this one;
-//   weights  : a warp takes items of 4 rows x a range of 256-value chunks, the next step's loads in flight during the arithmetic;
-//       four row sums are reduced over the lanes together (6 shuffles);
-//   epilogue : the range sums of a row are added in a fixed order by one thread: store | residual add | gelu(gate) * up (rows
+//   weights  : a consumer warp works on 4 rows x 1 chunk of every stage and adds over the stages of its rows in registers; four row
+//       sums are then reduced over the lanes together;
+//   epilogue : the chunk sums of a row are added in a fixed order by one thread: store | residual add | gelu(gate) * up (rows
 //       2u and 2u+1 of an interleaved matrix) | gelu * token embedding | logits with the block's first maximum.
+// Every mbarrier wait is bounded, as everywhere in the library.
 #pragma once
 #include "dense_ops.cuh"
 
 namespace l2b {
 
-constexpr int DMV_WARPS = 16, DMV_THREADS = DMV_WARPS * 32, DMV_ROWS = 4;
+constexpr int DMV_WARPS = 8, DMV_CONSUMERS = DMV_WARPS * 32, DMV_THREADS = DMV_CONSUMERS + 32, DMV_ROWS = 4;
+constexpr int DMV_STAGE = DMV_WARPS * DMV_ROWS * 512, DMV_STAGES = 4;
 
 struct DmvParams {
     const bf16* w;          // [rows][kp], kp a multiple of 8
@@ -24,8 +29,8 @@ struct DmvParams {
     int unit;               // rows per result: 1, or 2 (interleaved gate / up)
     int per_lo, per_rem;    // results of block b: per_lo + (b < per_rem), contiguous
     int nchunk;             // 256-value chunks per row
-    int nslice, cps;        // a row is summed in nslice ranges of cps chunks
-    int prefetch;           // bytes of the block's rows to prefetch into L2
+    int gs, cs, nseg;       // a stage: 4 * gs rows x cs chunks (gs * cs <= 8); nseg stages per row group, gs = 1 when nseg > 1
+    int prefetch;           // bytes of the block's rows to have in flight before the wait, ring included
     const float* x;         // input vector [k]
     ResidualUpdate upd;
     float* x_out;           // block 0 writes the updated vector here (null: no update)
@@ -33,144 +38,177 @@ struct DmvParams {
     DenseEpilogue epi;      // t = 0
     float* amax_val;        // DE_LOGITS: per block
     int* amax_idx;
+    int* status;
 };
 inline size_t dmv_smem_bytes(const DmvParams& p) {
-    const int rows = p.unit * (p.per_lo + (p.per_rem ? 1 : 0));
-    return ((size_t)p.nchunk * 256 + (size_t)((rows + DMV_ROWS - 1) / DMV_ROWS * DMV_ROWS) * p.nslice) * 4;
+    const int rows = p.unit * (p.per_lo + (p.per_rem ? 1 : 0)), per_stage = DMV_ROWS * p.gs;
+    return (size_t)DMV_STAGES * DMV_STAGE + ((size_t)p.nchunk * 256 + (size_t)((rows + per_stage - 1) / per_stage * per_stage) * p.cs) * 4;
 }
 
 __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __grid_constant__ DmvParams p) {
-    extern __shared__ __align__(16) float dmv_smem[];
+    extern __shared__ __align__(128) uint8_t dmv_smem[];
+    __shared__ __align__(8) uint64_t s_full[DMV_STAGES], s_empty[DMV_STAGES];
     __shared__ float s_red[DMV_WARPS];
     __shared__ int s_idx[DMV_WARPS];
-    float* const xf = dmv_smem;
-    float* const part = dmv_smem + p.nchunk * 256;
+    float* const xf = reinterpret_cast<float*>(dmv_smem + DMV_STAGES * DMV_STAGE);
+    float* const part = xf + p.nchunk * 256;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     pdl_launch_dependents();
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < DMV_STAGES; ++i) {
+            mbar_init(s_full + i, 1);
+            mbar_init(s_empty + i, DMV_WARPS);
+        }
+        fence_barrier_init();
+        fence_proxy_async();
+    }
+    __syncthreads();
     const int b = (int)blockIdx.x;
     const int u0 = b * p.per_lo + min(b, p.per_rem), nu = p.per_lo + (b < p.per_rem ? 1 : 0);
     const int nr = nu * p.unit;
     const bf16* const wb = p.w + (size_t)u0 * p.unit * p.kp;
+    const int per_stage = DMV_ROWS * p.gs, nstage = (nr + per_stage - 1) / per_stage * p.nseg;
+    const int seg_vals = p.cs * 256, pitch = p.nseg == 1 ? p.kp : seg_vals;  // values between the rows of a stage
+    bool dead = false;
 
-    if (warp == DMV_WARPS - 1) {
-        const size_t total = min((size_t)p.prefetch, (size_t)nr * p.kp * 2);
-        for (size_t o = (size_t)lane * 4096; o < total; o += 32 * 4096)
-            asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(reinterpret_cast<const char*>(wb) + o), "r"((uint32_t)min((size_t)4096, total - o)) : "memory");
-    }
-    const int nitems = (nr + DMV_ROWS - 1) / DMV_ROWS * p.nslice;
-    int it = warp, g = 0, c = 0, c1 = 0;
-    uint4 nxt[DMV_ROWS];
-    auto begin_item = [&]() {
-        g = it / p.nslice;
-        c = (it - g * p.nslice) * p.cps;
-        c1 = min(p.nchunk, c + p.cps);
-    };
-    auto load = [&]() {
-        const int e = c * 256 + lane * 8;
-        const bf16* src = wb + (size_t)g * DMV_ROWS * p.kp + e;
-        const int lim = nr - 1 - g * DMV_ROWS;
-#pragma unroll
-        for (int i = 0; i < DMV_ROWS; ++i) {
-            nxt[i] = make_uint4(0u, 0u, 0u, 0u);
-            if (e < p.kp) nxt[i] = __ldg(reinterpret_cast<const uint4*>(src + (size_t)min(i, lim) * p.kp));
+    if (warp == DMV_WARPS) {
+        const uint64_t policy = policy_evict_first();
+        int row = 0, seg = 0;
+        for (int j = 0; j < nstage; ++j) {
+            const int s = j % DMV_STAGES, use = j / DMV_STAGES;
+            if (use > 0 && !mbar_wait_bounded(s_empty + s, (uint32_t)((use - 1) & 1))) {
+                dead = true;
+                break;
+            }
+            __syncwarp();
+            const int rows = min(per_stage, nr - row), vals = p.nseg == 1 ? p.kp : min(seg_vals, p.kp - seg * seg_vals);
+            uint8_t* const dst = dmv_smem + s * DMV_STAGE;
+            if (lane == 0) mbar_arrive_expect_tx(s_full + s, (uint32_t)(rows * vals * 2));
+            __syncwarp();
+            const bf16* const src = wb + (size_t)row * p.kp + seg * seg_vals;
+            if (p.nseg == 1) {
+                if (lane == 0) bulk_g2s(dst, src, (uint32_t)(rows * vals * 2), s_full + s, policy);
+            } else if (lane < rows) {
+                bulk_g2s(dst + lane * seg_vals * 2, src + (size_t)lane * p.kp, (uint32_t)(vals * 2), s_full + s, policy);
+            }
+            if (++seg == p.nseg) {
+                seg = 0;
+                row += per_stage;
+            }
+            if (j == min(DMV_STAGES, nstage) - 1) {  // the ring is full: what follows it, into L2
+                const size_t total = min((size_t)p.prefetch, (size_t)nr * p.kp * 2);
+                for (size_t o = (size_t)row * p.kp * 2 + (size_t)lane * 4096; o < total; o += 32 * 4096)
+                    asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(reinterpret_cast<const char*>(wb) + o), "r"((uint32_t)min((size_t)4096, total - o))
+                                 : "memory");
+            }
         }
-    };
-    bool have = it < nitems;
-    if (have) {
-        begin_item();
-        load();
+        if (dead) {
+            if (lane == 0) atomicExch(p.status, DEV_ERR_TMA_TIMEOUT);
+            for (int i = 0; i < 2000; ++i) __nanosleep(1000);  // copies in flight land within microseconds
+        }
+        __syncthreads();
+        if (p.epi.kind == DE_LOGITS) __syncthreads();
+        return;
     }
 
     pdl_wait();
     {
-        constexpr int U = 4;
+        constexpr int U = 8;
         const int k = p.k, kc = p.nchunk * 256;
         float scale = 0.f;
         if (p.upd.y) {
             float ss = 0.f;
-            for (int i0 = threadIdx.x; i0 < k; i0 += U * DMV_THREADS) {
+            for (int i0 = threadIdx.x; i0 < k; i0 += U * DMV_CONSUMERS) {
                 float v[U];
 #pragma unroll
-                for (int u = 0; u < U; ++u) v[u] = i0 + u * DMV_THREADS < k ? __ldcg(p.upd.y + i0 + u * DMV_THREADS) : 0.f;
+                for (int u = 0; u < U; ++u) v[u] = i0 + u * DMV_CONSUMERS < k ? __ldcg(p.upd.y + i0 + u * DMV_CONSUMERS) : 0.f;
 #pragma unroll
                 for (int u = 0; u < U; ++u) {
                     ss = fmaf(v[u], v[u], ss);
-                    if (i0 + u * DMV_THREADS < k) xf[i0 + u * DMV_THREADS] = v[u];
+                    if (i0 + u * DMV_CONSUMERS < k) xf[lane_major(i0 + u * DMV_CONSUMERS)] = v[u];
                 }
             }
             scale = 1.f / sqrtf(block_sum_all<DMV_WARPS>(ss, s_red) / (float)k + p.upd.eps);
         }
-        for (int i0 = threadIdx.x; i0 < kc; i0 += U * DMV_THREADS) {
+        for (int i0 = threadIdx.x; i0 < kc; i0 += U * DMV_CONSUMERS) {
             float v[U];
 #pragma unroll
-            for (int u = 0; u < U; ++u) v[u] = i0 + u * DMV_THREADS < k ? __ldcg(p.x + i0 + u * DMV_THREADS) : 0.f;
+            for (int u = 0; u < U; ++u) v[u] = i0 + u * DMV_CONSUMERS < k ? __ldcg(p.x + i0 + u * DMV_CONSUMERS) : 0.f;
 #pragma unroll
             for (int u = 0; u < U; ++u) {
-                const int i = i0 + u * DMV_THREADS;
+                const int i = i0 + u * DMV_CONSUMERS, at = lane_major(i);
                 if (i < k) {
                     float t = v[u];
-                    if (p.upd.y) t = fmaf(xf[i] * scale, __ldg(p.upd.side_w + i), t);
+                    if (p.upd.y) t = fmaf(xf[at] * scale, __ldg(p.upd.side_w + i), t);
                     if (p.upd.step) t += __ldg(p.upd.step + i);
                     if (p.x_out && b == 0) p.x_out[i] = t;
-                    xf[i] = apply_norm(p.norm, t, i);
+                    xf[at] = apply_norm(p.norm, t, i);
                 } else if (i < kc) {
-                    xf[i] = 0.f;
+                    xf[at] = 0.f;
                 }
             }
         }
     }
-    __syncthreads();
+    partial_sync(DMV_CONSUMERS);
 
-    float acc[DMV_ROWS];
+    {
+        const int ug = warp / p.cs, uc = warp - ug * p.cs;  // this warp's row group and chunk of a stage
+        const bool mine = ug < p.gs;
+        int row = ug * DMV_ROWS, seg = 0, s = 0;
+        uint32_t par = 0;
+        f32x2 acc[DMV_ROWS];
 #pragma unroll
-    for (int i = 0; i < DMV_ROWS; ++i) acc[i] = 0.f;
-    while (have) {
-        uint4 cur[DMV_ROWS];
+        for (int i = 0; i < DMV_ROWS; ++i) acc[i] = 0ull;
+        for (int j = 0; j < nstage; ++j) {
+            if (!dead && !mbar_wait_bounded(s_full + s, par)) dead = true;
+            const int c = seg * p.cs + uc, e = uc * 256 + lane * 8;
+            if (mine && !dead && c * 256 + lane * 8 < p.kp && row < nr) {
+                const uint8_t* src = dmv_smem + s * DMV_STAGE + ((size_t)ug * DMV_ROWS * pitch + e) * 2;
+                uint4 w[DMV_ROWS];
 #pragma unroll
-        for (int i = 0; i < DMV_ROWS; ++i) cur[i] = nxt[i];
-        const int ccur = c, itcur = it, gcur = g;
-        const bool last = c + 1 == c1;
-        if (last) {
-            it += DMV_WARPS;
-            have = it < nitems;
-            if (have) begin_item();
-        } else {
-            ++c;
+                for (int i = 0; i < DMV_ROWS; ++i) w[i] = *reinterpret_cast<const uint4*>(src + (size_t)i * pitch * 2);
+                const Pairs8 x = read_lane_major(xf, c, lane);
+#pragma unroll
+                for (int i = 0; i < DMV_ROWS; ++i) {
+                    acc[i] = fma2(widen2(w[i].x), x.p[0], acc[i]);
+                    acc[i] = fma2(widen2(w[i].y), x.p[1], acc[i]);
+                    acc[i] = fma2(widen2(w[i].z), x.p[2], acc[i]);
+                    acc[i] = fma2(widen2(w[i].w), x.p[3], acc[i]);
+                }
+            }
+            __syncwarp();
+            if (lane == 0) mbar_arrive(s_empty + s);
+            if (++s == DMV_STAGES) s = 0, par ^= 1u;
+            if (++seg == p.nseg) {
+                seg = 0;
+                if (mine) {  // (uniform over the warp) four sums over the lanes at once: lanes 8q .. 8q+7 end up with row q
+                    float a[DMV_ROWS];
+#pragma unroll
+                    for (int i = 0; i < DMV_ROWS; ++i) a[i] = sum2(acc[i]), acc[i] = 0ull;
+                    const bool hi = lane & 16, mid = lane & 8;
+                    float v0 = (hi ? a[2] : a[0]) + __shfl_xor_sync(0xffffffffu, hi ? a[0] : a[2], 16);
+                    float v1 = (hi ? a[3] : a[1]) + __shfl_xor_sync(0xffffffffu, hi ? a[1] : a[3], 16);
+                    float v = (mid ? v1 : v0) + __shfl_xor_sync(0xffffffffu, mid ? v0 : v1, 8);
+                    v += __shfl_xor_sync(0xffffffffu, v, 4);
+                    v += __shfl_xor_sync(0xffffffffu, v, 2);
+                    v += __shfl_xor_sync(0xffffffffu, v, 1);
+                    if ((lane & 7) == 0) part[(row + (lane >> 3)) * p.cs + uc] = v;
+                }
+                row += per_stage;
+            }
         }
-        if (have) load();
-        const float4 xa = *reinterpret_cast<const float4*>(xf + ccur * 256 + lane * 8), xb = *reinterpret_cast<const float4*>(xf + ccur * 256 + lane * 8 + 4);
-#pragma unroll
-        for (int i = 0; i < DMV_ROWS; ++i) {
-            const Vec8 w = unpack8(cur[i]);
-            float a = acc[i];
-            a = fmaf(w.v[0], xa.x, a); a = fmaf(w.v[1], xa.y, a); a = fmaf(w.v[2], xa.z, a); a = fmaf(w.v[3], xa.w, a);
-            a = fmaf(w.v[4], xb.x, a); a = fmaf(w.v[5], xb.y, a); a = fmaf(w.v[6], xb.z, a); a = fmaf(w.v[7], xb.w, a);
-            acc[i] = a;
-        }
-        if (last) {
-            // four sums over the lanes at once: lanes 8q .. 8q+7 end up with row q
-            const bool hi = lane & 16, mid = lane & 8;
-            float v0 = (hi ? acc[2] : acc[0]) + __shfl_xor_sync(0xffffffffu, hi ? acc[0] : acc[2], 16);
-            float v1 = (hi ? acc[3] : acc[1]) + __shfl_xor_sync(0xffffffffu, hi ? acc[1] : acc[3], 16);
-            float v = (mid ? v1 : v0) + __shfl_xor_sync(0xffffffffu, mid ? v0 : v1, 8);
-            v += __shfl_xor_sync(0xffffffffu, v, 4);
-            v += __shfl_xor_sync(0xffffffffu, v, 2);
-            v += __shfl_xor_sync(0xffffffffu, v, 1);
-            if ((lane & 7) == 0) part[(gcur * DMV_ROWS + (lane >> 3)) * p.nslice + (itcur - gcur * p.nslice)] = v;
-#pragma unroll
-            for (int i = 0; i < DMV_ROWS; ++i) acc[i] = 0.f;
-        }
+        if (dead && lane == 0) atomicExch(p.status, DEV_ERR_TMA_TIMEOUT);
     }
     __syncthreads();
 
     float best = -INFINITY;
     int best_i = 0x7fffffff;
-    for (int u = threadIdx.x; u < nu; u += DMV_THREADS) {
+    for (int u = threadIdx.x; u < nu; u += DMV_CONSUMERS) {
         float v = 0.f, v2 = 0.f;
-        const float* pr = part + u * p.unit * p.nslice;
-        for (int s = 0; s < p.nslice; ++s) v += pr[s];
+        const float* pr = part + u * p.unit * p.cs;
+        for (int s = 0; s < p.cs; ++s) v += pr[s];
         if (p.unit == 2)
-            for (int s = 0; s < p.nslice; ++s) v2 += pr[p.nslice + s];
+            for (int s = 0; s < p.cs; ++s) v2 += pr[p.cs + s];
         dense_epilogue<float>(p.epi, 0, u0 + u, v, v2);
         if (v > best) {
             best = v;

@@ -9,6 +9,75 @@ namespace l2b {
 
 typedef __nv_bfloat16 bf16;
 
+// Two f32 values in one register pair: one instruction does both multiply-adds, each rounded as fmaf rounds.
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2(float lo, float hi) {
+    f32x2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+__device__ __forceinline__ void unpack2(f32x2 v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+    f32x2 r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+    f32x2 r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+__device__ __forceinline__ float sum2(f32x2 v) {
+    float lo, hi;
+    unpack2(v, lo, hi);
+    return lo + hi;
+}
+// two stored bf16 (one word) as two f32
+__device__ __forceinline__ f32x2 widen2(uint32_t w) { return pack2(__uint_as_float(w << 16), __uint_as_float(w & 0xFFFF0000u)); }
+
+// An f32 vector that warps read 8 consecutive values per lane (value e = 256 c + 8 lane + j) lies in shared memory as two float4
+// halves per 256 values, so that the 16-byte reads of a warp are free of bank conflicts.
+__device__ __forceinline__ int lane_major(int e) { return (e & ~255) + ((e >> 2) & 1) * 128 + ((e >> 3) & 31) * 4 + (e & 3); }
+struct Pairs8 {
+    f32x2 p[4];
+};
+__device__ __forceinline__ Pairs8 read_lane_major(const float* x, int c, int lane) {
+    const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(x + c * 256 + lane * 4), b = *reinterpret_cast<const ulonglong2*>(x + c * 256 + 128 + lane * 4);
+    Pairs8 o;
+    o.p[0] = a.x; o.p[1] = a.y; o.p[2] = b.x; o.p[3] = b.y;
+    return o;
+}
+
+// N sums over the lanes of a warp at once; every lane gets all of them.  While more than one value is left, a step exchanges half of
+// the values across a lane bit and halves their number; the remaining bits are reduced as usual.
+template <int N>
+__device__ __forceinline__ void warp_sums(float (&v)[N]) {
+    static_assert(N == 1 || N == 2 || N == 4 || N == 8, "number of sums");
+    const int lane = threadIdx.x & 31;
+    float t[N];
+#pragma unroll
+    for (int i = 0; i < N; ++i) t[i] = v[i];
+    int o = 16;
+#pragma unroll
+    for (int n = N; n > 1; n >>= 1, o >>= 1) {
+        const bool up = lane & o;
+#pragma unroll
+        for (int i = 0; i < n / 2; ++i) {
+            const float keep = up ? t[i + n / 2] : t[i], send = up ? t[i] : t[i + n / 2];
+            t[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+        }
+    }
+#pragma unroll
+    for (; o > 0; o >>= 1) t[0] += __shfl_xor_sync(0xffffffffu, t[0], o);
+#pragma unroll
+    for (int i = 0; i < N; ++i) {  // value i sits in the lanes whose upper bits spell i
+        int src = 0, bit = 16;
+#pragma unroll
+        for (int n = N; n > 1; n >>= 1, bit >>= 1) src += (i & (n / 2)) ? bit : 0;
+        v[i] = N > 1 ? __shfl_sync(0xffffffffu, t[0], src) : t[0];
+    }
+}
+
 // eight consecutive values (16-byte aligned bf16, 32-byte aligned f32) as f32
 struct Vec8 {
     float v[8];
@@ -31,6 +100,12 @@ struct Raw8<bf16> {
     __device__ __forceinline__ void zero() { r = make_uint4(0u, 0u, 0u, 0u); }
     __device__ __forceinline__ void load(const bf16* p) { r = __ldcg(reinterpret_cast<const uint4*>(p)); }
     __device__ __forceinline__ Vec8 get() const { return unpack8(r); }
+    __device__ __forceinline__ void read(const void* smem) { r = *static_cast<const uint4*>(smem); }
+    __device__ __forceinline__ Pairs8 pairs() const {
+        Pairs8 o;
+        o.p[0] = widen2(r.x); o.p[1] = widen2(r.y); o.p[2] = widen2(r.z); o.p[3] = widen2(r.w);
+        return o;
+    }
 };
 template <>
 struct Raw8<float> {
@@ -44,6 +119,15 @@ struct Raw8<float> {
         Vec8 o;
         o.v[0] = a.x; o.v[1] = a.y; o.v[2] = a.z; o.v[3] = a.w;
         o.v[4] = b.x; o.v[5] = b.y; o.v[6] = b.z; o.v[7] = b.w;
+        return o;
+    }
+    __device__ __forceinline__ void read(const void* smem) {
+        a = static_cast<const float4*>(smem)[0];
+        b = static_cast<const float4*>(smem)[1];
+    }
+    __device__ __forceinline__ Pairs8 pairs() const {
+        Pairs8 o;
+        o.p[0] = pack2(a.x, a.y); o.p[1] = pack2(a.z, a.w); o.p[2] = pack2(b.x, b.y); o.p[3] = pack2(b.z, b.w);
         return o;
     }
 };
@@ -89,8 +173,10 @@ struct DenseEpilogue {
     int vocab;            // DE_SIDE: rows of the table (an id outside it contributes zero)
 };
 __device__ __forceinline__ float side_value(const DenseEpilogue& e, int t, int f) {
-    const int tok = __ldcg(e.tokens + t);
-    return tok >= 0 && tok < e.vocab ? __bfloat162float(e.etab[(size_t)tok * e.e_ld + e.e_off + f]) : 0.f;
+    const int tok = __ldg(e.tokens + t);
+    const bool valid = tok >= 0 && tok < e.vocab;  // (the load does not depend on it: several are in flight together)
+    const float v = __bfloat162float(e.etab[(size_t)(valid ? tok : 0) * e.e_ld + e.e_off + f]);
+    return valid ? v : 0.f;
 }
 template <typename AT>
 __device__ __forceinline__ void dense_epilogue(const DenseEpilogue& e, int t, int f, float v, float v2) {
@@ -124,12 +210,15 @@ __device__ __forceinline__ float apply_norm(const NormParams& n, float x, int i)
     return n.kind ? dynamic_tanh(x, n.alpha, __ldg(n.w + i), __ldg(n.b + i)) : x;
 }
 
-// Sum over the threads of a block of NW warps; every thread gets it.  s holds NW floats and may be reused after the next barrier.
+// Barrier over the first `threads` threads of the block.
+__device__ __forceinline__ void partial_sync(int threads) { asm volatile("bar.sync 1, %0;" ::"r"(threads) : "memory"); }
+
+// Sum over the first NW warps of a block; each of their threads gets it.  s holds NW floats and may be reused after the next barrier.
 template <int NW>
 __device__ __forceinline__ float block_sum_all(float v, float* s) {
     v = warp_sum(v);
     if ((threadIdx.x & 31) == 0) s[threadIdx.x >> 5] = v;
-    __syncthreads();
+    partial_sync(NW * 32);
     float t = 0.f;
 #pragma unroll
     for (int i = 0; i < NW; ++i) t += s[i];

@@ -167,14 +167,19 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prefill_kernel(const __grid
             __syncwarp();
             if (lane == 0) mbar_arrive(s_sfree + b);
             const int lim = qpos - j * LP_TILE;  // keys 0 .. lim of the tile are seen
-            float mx = -INFINITY;
+            if (j * LP_TILE + LP_TILE - 1 > p.pos0 + q0) {  // (the last tiles only)
+#pragma unroll
+                for (int c = 0; c < 4; ++c)
+#pragma unroll
+                    for (int k = 0; k < 32; ++k)
+                        if (32 * c + k > lim) s[c][k] = -INFINITY;
+            }
+            float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
             for (int c = 0; c < 4; ++c)
 #pragma unroll
-                for (int k = 0; k < 32; ++k) {
-                    s[c][k] = 32 * c + k <= lim ? s[c][k] * p.scale2 : -INFINITY;
-                    mx = fmaxf(mx, s[c][k]);
-                }
+                for (int k = 0; k < 32; ++k) m4[k & 3] = fmaxf(m4[k & 3], s[c][k]);
+            const float mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3])) * p.scale2;  // (scale2 > 0)
             if (j > 0 && !__all_sync(0xffffffffu, mbar_wait_bounded(&s_o, (uint32_t)((j - 1) & 1)))) {  // P and O are free
                 ok = false;
                 break;
@@ -195,6 +200,7 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prefill_kernel(const __grid
                     tmem_st32f(tmem_o + lane_off + (uint32_t)c, o);
                 }
             }
+            float l4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
             for (int c = 0; c < 4; ++c)
 #pragma unroll
@@ -202,14 +208,15 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prefill_kernel(const __grid
                     uint32_t w[4];
 #pragma unroll
                     for (int k = 0; k < 4; ++k) {
-                        const float e0 = exp2f(s[c][8 * g + 2 * k] - m), e1 = exp2f(s[c][8 * g + 2 * k + 1] - m);
-                        l += e0 + e1;
+                        const float e0 = exp2f(fmaf(s[c][8 * g + 2 * k], p.scale2, -m)), e1 = exp2f(fmaf(s[c][8 * g + 2 * k + 1], p.scale2, -m));
+                        l4[k] += e0 + e1;
                         const __nv_bfloat162 pk = __floats2bfloat162_rn(e0, e1);
                         w[k] = *reinterpret_cast<const uint32_t*>(&pk);
                     }
                     const int chunk = 4 * (c & 1) + g;
                     *reinterpret_cast<uint4*>(smem + L.p + (c >> 1) * LP_SUB + r * 128 + ((chunk ^ (r & 7)) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);
                 }
+            l += (l4[0] + l4[1]) + (l4[2] + l4[3]);
             fence_proxy_async();
             tc_fence_before();
             __syncwarp();
@@ -221,18 +228,26 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prefill_kernel(const __grid
         } else {
             tc_fence_after();
             const float inv = 1.f / (l + exp2f(__ldg(p.sink + h) * 1.4426950408889634f - m));  // the sink: a term of the denominator only
-            const float* gate = p.gate + (size_t)qi * p.ld + h * p.vdim;
             bf16* out = p.out + (size_t)qi * p.ldo + h * p.vdim;
             const bool wide = ((p.vdim | p.ldo) & 7) == 0;
+            // gates of this warp's 32 queries, 32 values at a time, through the shared memory that held P (its last product is done)
+            float* const sg = reinterpret_cast<float*>(smem + L.p) + qd * (32 * 33);
 #pragma unroll 1
             for (int c = 0; c < p.vdim; c += 32) {
                 float o[32];
                 __syncwarp();
+#pragma unroll
+                for (int i = 0; i < 32; ++i) {
+                    const int t = q0 + 32 * qd + i;
+                    o[i] = t < p.n && c + lane < p.vdim ? __ldg(p.gate + (size_t)t * p.ld + h * p.vdim + c + lane) : 0.f;
+                }
+#pragma unroll
+                for (int i = 0; i < 32; ++i) sg[i * 33 + lane] = o[i];
+                __syncwarp();
                 tmem_ld32f(tmem_o + lane_off + (uint32_t)c, o);
                 const int nv = qi < p.n ? p.vdim - c : 0;  // values of this query to store
 #pragma unroll
-                for (int k = 0; k < 32; ++k)
-                    if (k < nv) o[k] *= inv * sigmoid(__ldg(gate + c + k));
+                for (int k = 0; k < 32; ++k) o[k] *= inv * sigmoid(sg[lane * 33 + k]);
                 if (wide) {
 #pragma unroll
                     for (int g = 0; g < 4; ++g)
@@ -259,17 +274,26 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prefill_kernel(const __grid
 }
 
 // Query operand of the kernel above: [row][head][dq] = unrotated part rounded up to 16 (zeros), rotated part rounded up to 16.
-__global__ void __launch_bounds__(256) latent_queries_kernel(const float* __restrict__ qdg, int ld, const float2* __restrict__ rope, int pos0, LatentShape s, int dq,
+// Grid (rows, heads); a thread makes two values.
+__global__ void __launch_bounds__(128) latent_queries_kernel(const float* __restrict__ qdg, int ld, const float2* __restrict__ rope, int pos0, LatentShape s, int dq,
                                                             bf16* __restrict__ out) {
-    const int row = (int)blockIdx.x;
+    const int row = (int)blockIdx.x, h = (int)blockIdx.y;
     const float2* cs = rope + (size_t)(pos0 + row) * (s.rdims >> 1);
-    for (int i = threadIdx.x; i < s.heads * dq; i += 256) {
-        const int h = i / dq, d = i - h * dq;
-        const float* q = qdg + (size_t)row * ld + h * (s.dim + s.rot);
-        float v = 0.f;
-        if (d < s.dp) v = d < s.dim ? q[d] : 0.f;
-        else if (d - s.dp < s.rot) v = rotary_element(d - s.dp, s.rdims, cs, [&](int j) { return q[s.dim + j]; });
-        put(out + (size_t)row * s.heads * dq + i, v);
+    const float* q = qdg + (size_t)row * ld + h * (s.dim + s.rot);
+    bf16* dst = out + ((size_t)row * s.heads + h) * dq;
+    for (int d = 2 * threadIdx.x; d < dq; d += 256) {
+        float v0 = 0.f, v1 = 0.f;
+        if (d < s.dp) {
+            v0 = d < s.dim ? q[d] : 0.f;
+            v1 = d + 1 < s.dim ? q[d + 1] : 0.f;
+        } else {
+            const int r = d - s.dp;  // even: a whole pair, or two unrotated values
+            if (r < s.rot) {
+                v0 = rotary_element(r, s.rdims, cs, [&](int j) { return q[s.dim + j]; });
+                v1 = rotary_element(r + 1, s.rdims, cs, [&](int j) { return q[s.dim + j]; });
+            }
+        }
+        *reinterpret_cast<__nv_bfloat162*>(dst + d) = __floats2bfloat162_rn(v0, v1);
     }
 }
 

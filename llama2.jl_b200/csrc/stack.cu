@@ -309,9 +309,12 @@ static int32_t set_stack_kernel_attrs() {
         set((const void*)bf16_gemm_kernel<64, 1>); set((const void*)bf16_gemm_kernel<64, 2>);
         set((const void*)bf16_gemm_kernel<128, 1>); set((const void*)bf16_gemm_kernel<128, 2>);
 #define L2B_SET_LA(NI)                                                    \
-    set((const void*)latent_attention_kernel<bf16, float, NI>);           \
-    set((const void*)latent_attention_kernel<bf16, bf16, NI>);            \
-    set((const void*)latent_attention_kernel<float, float, NI>);
+    set((const void*)latent_attention_kernel<bf16, float, NI, 1>);        \
+    set((const void*)latent_attention_kernel<bf16, float, NI, 2>);        \
+    set((const void*)latent_attention_kernel<bf16, bf16, NI, 1>);         \
+    set((const void*)latent_attention_kernel<bf16, bf16, NI, 2>);         \
+    set((const void*)latent_attention_kernel<float, float, NI, 1>);       \
+    set((const void*)latent_attention_kernel<float, float, NI, 2>);
         L2B_SET_LA(1) L2B_SET_LA(2) L2B_SET_LA(3) L2B_SET_LA(4)
 #undef L2B_SET_LA
     });
@@ -418,36 +421,43 @@ static LatentAttnParams latent_params(const StackSession* s, int run, const floa
     a.cache = s->cache[run];
     return a;
 }
-template <typename CT, typename OT>
-static cudaError_t launch_latent_attention(const LatentAttnParams& a, int rows, bool pdl, cudaStream_t st) {
-    const dim3 grid(a.s.heads * a.cl, rows), block(LA_THREADS);
-    const size_t smem = (size_t)la_smem_layout(a.s).total * 4;
+// Heads and blocks per cluster: two heads where one head per cluster of the portable size would need more than one block per SM, then
+// as many blocks as fill the GPU once (decode) or a few times (many rows).
+template <typename CT, typename OT, int GH>
+static cudaError_t launch_latent_attention_gh(const LatentAttnParams& a, int rows, bool pdl, cudaStream_t st) {
+    const dim3 grid(a.s.heads / GH * a.cl, rows), block(LA_THREADS);
+    const size_t smem = (size_t)la_smem_layout(a.s, GH, la_stage_rows<CT>() * a.s.row * (int)sizeof(CT) / 4, a.stages).total * 4;
     switch ((a.s.row + 255) / 256) {
-        case 1: return launch_kernel(latent_attention_kernel<CT, OT, 1>, grid, block, smem, st, pdl, a, a.cl);
-        case 2: return launch_kernel(latent_attention_kernel<CT, OT, 2>, grid, block, smem, st, pdl, a, a.cl);
-        case 3: return launch_kernel(latent_attention_kernel<CT, OT, 3>, grid, block, smem, st, pdl, a, a.cl);
-        default: return launch_kernel(latent_attention_kernel<CT, OT, 4>, grid, block, smem, st, pdl, a, a.cl);
+        case 1: return launch_kernel(latent_attention_kernel<CT, OT, 1, GH>, grid, block, smem, st, pdl, a, a.cl);
+        case 2: return launch_kernel(latent_attention_kernel<CT, OT, 2, GH>, grid, block, smem, st, pdl, a, a.cl);
+        case 3: return launch_kernel(latent_attention_kernel<CT, OT, 3, GH>, grid, block, smem, st, pdl, a, a.cl);
+        default: return launch_kernel(latent_attention_kernel<CT, OT, 4, GH>, grid, block, smem, st, pdl, a, a.cl);
     }
 }
-// Blocks per (row, head): as many as fill the GPU about twice, at most a portable cluster.
-static int latent_cluster(long pairs, const DeviceInfo& di) {
-    int cl = LA_MAX_CL;
-    while (cl > 1 && pairs * cl > 2L * di.sms) cl >>= 1;
-    return cl;
+template <typename CT, typename OT>
+static cudaError_t launch_latent_attention(LatentAttnParams a, int rows, bool pdl, const DeviceInfo& di, cudaStream_t st) {
+    const int gh = (long)a.s.heads * rows * LA_MAX_CL > di.sms && a.s.heads % 2 == 0 ? 2 : 1;
+    const long groups = (long)a.s.heads / gh * rows;
+    a.cl = LA_MAX_CL;
+    while (a.cl > 1 && groups * a.cl > (a.fused ? di.sms : 2L * di.sms)) a.cl >>= 1;
+    a.stages = a.fused ? LA_MAX_STAGES : 2;
+    const int stage_floats = la_stage_rows<CT>() * a.s.row * (int)sizeof(CT) / 4;
+    while (a.stages > 1 && la_smem_layout(a.s, gh, stage_floats, a.stages).total * 4 > di.max_smem_optin - 2048) --a.stages;
+    return gh == 2 ? launch_latent_attention_gh<CT, OT, 2>(a, rows, pdl, st) : launch_latent_attention_gh<CT, OT, 1>(a, rows, pdl, st);
 }
 
 // ---- one position ------------------------------------------------------------------------------
-static int32_t launch_dense_matvec(const StackSession* s, const StackMatrix& w, DmvParams& p, cudaStream_t st, int* nblocks = nullptr) {
+static int32_t launch_dense_matvec(const StackSession* s, const StackMatrix& w, DmvParams& p, int* status, cudaStream_t st, int* nblocks = nullptr) {
+    p.status = status;
     p.w = w.w; p.kp = w.kp; p.k = w.k; p.unit = w.pair;
     const int results = w.results(), grid = std::min(s->di.sms, results);
     p.per_lo = results / grid;
     p.per_rem = results % grid;
     p.nchunk = (w.k + 255) / 256;
-    const int rows = (p.per_lo + (p.per_rem ? 1 : 0)) * w.pair, groups = (rows + DMV_ROWS - 1) / DMV_ROWS;
-    const int want = std::max(1, (3 * DMV_WARPS + groups - 1) / groups);  // about three items per warp
-    p.nslice = std::min(p.nchunk, want);
-    p.cps = (p.nchunk + p.nslice - 1) / p.nslice;
-    p.nslice = (p.nchunk + p.cps - 1) / p.cps;
+    p.nseg = (p.nchunk + DMV_WARPS - 1) / DMV_WARPS;
+    p.cs = (p.nchunk + p.nseg - 1) / p.nseg;
+    p.nseg = (p.nchunk + p.cs - 1) / p.cs;
+    p.gs = p.nseg == 1 ? DMV_WARPS / p.cs : 1;
     p.prefetch = 256 * 1024;
     const size_t smem = dmv_smem_bytes(p);
     if (smem > (size_t)s->di.max_smem_optin - 1024) return fail(L2B_ERR_BAD_ARG, "input vector too long for shared memory");
@@ -456,8 +466,8 @@ static int32_t launch_dense_matvec(const StackSession* s, const StackMatrix& w, 
     return L2B_OK;
 }
 
-int32_t stack_enqueue_token(StackSession* s, const int* token, const int* pos, float* logits, float* amax_val, int* amax_idx, cudaStream_t st, int* nlaunch,
-                            int* nparts) {
+int32_t stack_enqueue_token(StackSession* s, const int* token, const int* pos, float* logits, float* amax_val, int* amax_idx, int* status, cudaStream_t st,
+                            int* nlaunch, int* nparts) {
     const StackModel* m = s->m;
     const StackConfig& c = m->cfg;
     int count = 0, cur = 0;
@@ -492,7 +502,7 @@ int32_t stack_enqueue_token(StackSession* s, const int* token, const int* pos, f
         p.epi.y = out;
         p.epi.act = out;
         ++count;
-        return launch_dense_matvec(s, w, p, st, nb);
+        return launch_dense_matvec(s, w, p, status, st, nb);
     };
     DmvParams p;
     for (size_t r = 0; r < m->runs.size(); ++r) {
@@ -507,8 +517,8 @@ int32_t stack_enqueue_token(StackSession* s, const int* token, const int* pos, f
             a.out = s->att1;
             a.ldo = w.o.k;
             a.fused = 1;
-            a.cl = latent_cluster(w.shape.heads, s->di);
-            CU(m->f32 ? (launch_latent_attention<float, float>(a, 1, true, st)) : (launch_latent_attention<bf16, float>(a, 1, true, st)));
+            a.status = status;
+            CU(m->f32 ? (launch_latent_attention<float, float>(a, 1, true, s->di, st)) : (launch_latent_attention<bf16, float>(a, 1, true, s->di, st)));
             ++count;
         }
         from_vector(p, s->att1);
@@ -574,15 +584,17 @@ static int32_t launch_gemm(const StackSession* s, const StackMatrix& w, const vo
     memset(&g, 0, sizeof(g));
     g.rows = rows; g.n_tok = n; g.k = w.k; g.epi = epi; g.status = status;
     g.row2 = w.pair == 2 || na == 1 ? 0 : 128;
-    const int nk = (w.k + BG_KB - 1) / BG_KB, stage = bg_stage_bytes(bn, na);
-    g.stages = std::max(1, std::min(std::min(BG_MAX_STAGES, nk), (s->di.max_smem_optin - 4096) / stage));
+    const int stage = bg_stage_bytes(bn, na);
+    g.stages = std::min(BG_MAX_STAGES, (s->di.max_smem_optin - 4096) / stage);
     CUtensorMap ma, ma2, mb;
     L2B_TRY(bf16_map(ma, w.w, w.k, rows, (int64_t)w.stride(), 128));
     ma2 = ma;
     if (w.pair == 2) L2B_TRY(bf16_map(ma2, w.second(), w.k, rows, (int64_t)w.stride(), 128));
     L2B_TRY(bf16_map(mb, static_cast<const bf16*>(x), w.k, n, ldx, bn));
     const int per = w.pair == 2 ? 128 : 128 * na;
-    const dim3 grid((rows + per - 1) / per, (n + bn - 1) / bn), block(BG_THREADS);
+    g.mtiles = (rows + per - 1) / per;
+    g.ntiles = (n + bn - 1) / bn;
+    const dim3 grid((unsigned)std::min<long>((long)g.mtiles * g.ntiles, s->di.sms)), block(BG_THREADS);
     const size_t smem = (size_t)g.stages * stage + 1024;
     auto go = [&](auto k) { return launch_kernel_args(k, grid, block, smem, st, false, 1, g, ma, ma2, mb); };
     cudaError_t e;
@@ -593,8 +605,9 @@ static int32_t launch_gemm(const StackSession* s, const StackMatrix& w, const vo
 }
 
 static int32_t launch_residual_rows(const StackSession* s, const RowsParams& r, int n, cudaStream_t st) {
-    if (s->m->f32) residual_rows_kernel<float><<<n, 256, 0, st>>>(r);
-    else residual_rows_kernel<bf16><<<n, 256, 0, st>>>(r);
+    const bool wide = r.width % 4 == 0;
+    if (s->m->f32) wide ? residual_rows_kernel<float, 4><<<n, 256, 0, st>>>(r) : residual_rows_kernel<float, 1><<<n, 256, 0, st>>>(r);
+    else wide ? residual_rows_kernel<bf16, 4><<<n, 256, 0, st>>>(r) : residual_rows_kernel<bf16, 1><<<n, 256, 0, st>>>(r);
     CU(cudaGetLastError());
     return L2B_OK;
 }
@@ -616,9 +629,9 @@ static int32_t enqueue_latent_rows(StackSession* s, int run, int n, int pos0, co
     CU(cudaGetLastError());
     ++*launches;
     const int kstages = prefill_kstages(sh, s->di);
-    if (!s->pq || pos_list || n < EXPAND_MIN_ROWS || kstages == 0) {
-        a.cl = latent_cluster((long)n * sh.heads, s->di);
-        CU(m->f32 ? (launch_latent_attention<float, float>(a, n, false, st)) : (launch_latent_attention<bf16, bf16>(a, n, false, st)));
+    if (!s->pq || pos_list || n < EXPAND_MIN_ROWS || kstages == 0 || !(sh.scale2 > 0.f)) {
+        a.status = status;
+        CU(m->f32 ? (launch_latent_attention<float, float>(a, n, false, s->di, st)) : (launch_latent_attention<bf16, bf16>(a, n, false, s->di, st)));
         ++*launches;
         return L2B_OK;
     }
@@ -634,7 +647,7 @@ static int32_t enqueue_latent_rows(StackSession* s, int run, int n, int pos0, co
     e.act = s->pv;
     e.ld = s->pv_ld;
     L2B_TRY(launch_gemm(s, w.uv, cache, sh.row, npos, e, status, st));
-    latent_queries_kernel<<<n, 256, 0, st>>>(s->qdg, a.ld, a.rope, pos0, sh, dq, s->pq);
+    latent_queries_kernel<<<dim3(n, sh.heads), 128, 0, st>>>(s->qdg, a.ld, a.rope, pos0, sh, dq, s->pq);
     CU(cudaGetLastError());
     LatentPrefillParams f;
     memset(&f, 0, sizeof(f));

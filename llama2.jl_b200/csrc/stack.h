@@ -34,8 +34,8 @@ int stack_session_max_rows(const StackSession* s);
 const float* stack_session_residual(const StackSession* s);  // after the last layer of the most recent one-position pass
 
 // One position (token and pos are device scalars): every kernel up to the logits and their per-block maxima (*nparts of them).
-int32_t stack_enqueue_token(StackSession* s, const int* token, const int* pos, float* logits, float* amax_val, int* amax_idx, cudaStream_t st, int* nlaunch,
-                            int* nparts);
+int32_t stack_enqueue_token(StackSession* s, const int* token, const int* pos, float* logits, float* amax_val, int* amax_idx, int* status, cudaStream_t st,
+                            int* nlaunch, int* nparts);
 // n rows through every layer: row r is token dev_tokens[r] at position pos0 + r of sequence 0, or at pos_list[r] of sequence r.
 int32_t stack_enqueue_rows(StackSession* s, const int* dev_tokens, int n, int pos0, const int* pos_list, int* status, cudaStream_t st, long long* launches);
 // Logits of some rows of the most recent stack_enqueue_rows (dev_index: row numbers, null: rows 0 .. n-1) -> logits [n][vocab].

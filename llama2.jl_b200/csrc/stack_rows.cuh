@@ -27,25 +27,44 @@ struct RowsParams {
     void* act;             // [rows][lda] operand of the next product (null: none)
     int lda;
 };
-template <typename AT>
+// V: values a thread takes at a time (4 when width and lda allow 16-byte accesses, else 1)
+template <typename AT, int V>
 __global__ void __launch_bounds__(256) residual_rows_kernel(const __grid_constant__ RowsParams p) {
     __shared__ float s_red[8];
+    struct alignas(4 * V) F { float v[V]; };
+    struct alignas(sizeof(AT) * V) A { AT v[V]; };
     const int src = p.index ? __ldg(p.index + blockIdx.x) : (int)blockIdx.x;
-    float* x = p.x + (size_t)src * p.width;
-    const float* y = p.upd.y ? p.upd.y + (size_t)src * p.width : nullptr;
+    F* const x = reinterpret_cast<F*>(p.x + (size_t)src * p.width);
+    const F* const y = p.upd.y ? reinterpret_cast<const F*>(p.upd.y + (size_t)src * p.width) : nullptr;
+    const int n = p.width / V;
     float scale = 0.f;
     if (y) {
         float ss = 0.f;
-        for (int i = threadIdx.x; i < p.width; i += 256) ss = fmaf(y[i], y[i], ss);
+        for (int i = threadIdx.x; i < n; i += 256) {
+            const F t = y[i];
+#pragma unroll
+            for (int k = 0; k < V; ++k) ss = fmaf(t.v[k], t.v[k], ss);
+        }
         scale = 1.f / sqrtf(block_sum_all<8>(ss, s_red) / (float)p.width + p.upd.eps);
     }
-    AT* act = p.act ? static_cast<AT*>(p.act) + (size_t)blockIdx.x * p.lda : nullptr;
-    for (int i = threadIdx.x; i < p.width; i += 256) {
-        float t = x[i];
-        if (y) t = fmaf(y[i] * scale, __ldg(p.upd.side_w + i), t);
-        if (p.upd.step) t += __ldg(p.upd.step + i);
+    A* const act = p.act ? reinterpret_cast<A*>(static_cast<AT*>(p.act) + (size_t)blockIdx.x * p.lda) : nullptr;
+    for (int i = threadIdx.x; i < n; i += 256) {
+        F t = x[i];
+        if (y) {
+            const F b = y[i];
+#pragma unroll
+            for (int k = 0; k < V; ++k) t.v[k] = fmaf(b.v[k] * scale, __ldg(p.upd.side_w + i * V + k), t.v[k]);
+        }
+        if (p.upd.step)
+#pragma unroll
+            for (int k = 0; k < V; ++k) t.v[k] += __ldg(p.upd.step + i * V + k);
         if (p.store_x) x[i] = t;
-        if (act) put(act + i, apply_norm(p.norm, t, i));
+        if (act) {
+            A o;
+#pragma unroll
+            for (int k = 0; k < V; ++k) put(&o.v[k], apply_norm(p.norm, t.v[k], i * V + k));
+            act[i] = o;
+        }
     }
 }
 
