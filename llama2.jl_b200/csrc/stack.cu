@@ -271,6 +271,9 @@ struct StackSession {
     // one position
     float *x[2] = {nullptr, nullptr}, *qdg1 = nullptr, *att1 = nullptr, *hid1 = nullptr, *y1 = nullptr;
     int x_last = 0;
+    // absorbed attention: queries and partial results of up to ABSORB_ROWS rows
+    float *qp = nullptr, *part_acc = nullptr;
+    float2* part_ml = nullptr;
     // many positions
     float *xr = nullptr, *qdg = nullptr, *y = nullptr;
     void *act = nullptr, *act2 = nullptr;        // operands of the products, [max_rows][k rounded up to 8]
@@ -280,8 +283,15 @@ struct StackSession {
 
 static size_t act_bytes(const StackModel* m) { return m->f32 ? 4 : 2; }
 
+constexpr int ABSORB_ROWS = 64;  // rows per pass of the absorbed form of the attention (bounds its scratch)
 // The expanded form of the attention (latent_prefill.cuh) is for portions of at least this many rows.
 constexpr int EXPAND_MIN_ROWS = 48;
+
+// Groups of heads and ranges of positions of the scan kernel: about one block per SM in a decode step, two for several rows.
+static int latent_groups(const LatentShape& s) { return (s.heads + LA_WARPS - 1) / LA_WARPS; }
+static int latent_splits(const LatentShape& s, int rows, const DeviceInfo& di) {
+    return std::max(1, std::min(LA_MAX_SPLIT, (rows == 1 ? 1 : 2) * di.sms / (latent_groups(s) * rows)));
+}
 
 static int prefill_kstages(const LatentShape& s, const DeviceInfo& di) {
     if (s.vp > 256) return 0;
@@ -308,13 +318,9 @@ static int32_t set_stack_kernel_attrs() {
         set((const void*)bf16_gemm_kernel<32, 1>); set((const void*)bf16_gemm_kernel<32, 2>);
         set((const void*)bf16_gemm_kernel<64, 1>); set((const void*)bf16_gemm_kernel<64, 2>);
         set((const void*)bf16_gemm_kernel<128, 1>); set((const void*)bf16_gemm_kernel<128, 2>);
-#define L2B_SET_LA(NI)                                                    \
-    set((const void*)latent_attention_kernel<bf16, float, NI, 1>);        \
-    set((const void*)latent_attention_kernel<bf16, float, NI, 2>);        \
-    set((const void*)latent_attention_kernel<bf16, bf16, NI, 1>);         \
-    set((const void*)latent_attention_kernel<bf16, bf16, NI, 2>);         \
-    set((const void*)latent_attention_kernel<float, float, NI, 1>);       \
-    set((const void*)latent_attention_kernel<float, float, NI, 2>);
+#define L2B_SET_LA(NI)                                      \
+    set((const void*)latent_scan_kernel<bf16, NI>);         \
+    set((const void*)latent_scan_kernel<float, NI>);
         L2B_SET_LA(1) L2B_SET_LA(2) L2B_SET_LA(3) L2B_SET_LA(4)
 #undef L2B_SET_LA
     });
@@ -378,6 +384,17 @@ int32_t stack_session_create(const StackModel* m, const StackSessionInfo& info, 
         L2B_TRY(alloc(s->hid1, (size_t)max_k2 * 4));
         L2B_TRY(alloc(s->y1, (size_t)c.width * 4));
     }
+    size_t qp = 0, pml = 0, pacc = 0;
+    for (const StackLayerW& w : m->layers)
+        for (int rows = 1; rows <= std::max(1, std::min(ABSORB_ROWS, info.max_rows)); ++rows) {
+            const size_t pairs = (size_t)w.shape.heads * rows, slots = pairs * latent_splits(w.shape, rows, di);
+            qp = std::max(qp, pairs * w.shape.row);
+            pml = std::max(pml, slots);
+            pacc = std::max(pacc, slots * w.shape.rp);
+        }
+    L2B_TRY(alloc(s->qp, qp * 4));
+    L2B_TRY(alloc(s->part_ml, pml * sizeof(float2)));
+    L2B_TRY(alloc(s->part_acc, pacc * 4));
     const size_t T = (size_t)info.max_rows;
     L2B_TRY(alloc(s->xr, T * c.width * 4));
     L2B_TRY(alloc(s->qdg, T * max_qdg * 4));
@@ -419,31 +436,32 @@ static LatentAttnParams latent_params(const StackSession* s, int run, const floa
     a.qdg = qdg; a.ld = w.qdg.rows; a.off_d = w.off_d; a.off_g = w.off_g;
     a.uk = w.uk.w; a.uv = w.uv.w; a.sink = w.sink; a.dnorm = w.dkv_norm; a.rope = s->rope[l];
     a.cache = s->cache[run];
+    a.qp = s->qp; a.part_ml = s->part_ml; a.part_acc = s->part_acc;
     return a;
 }
-// Heads and blocks per cluster: two heads where one head per cluster of the portable size would need more than one block per SM, then
-// as many blocks as fill the GPU once (decode) or a few times (many rows).
-template <typename CT, typename OT, int GH>
-static cudaError_t launch_latent_attention_gh(const LatentAttnParams& a, int rows, bool pdl, cudaStream_t st) {
-    const dim3 grid(a.s.heads / GH * a.cl, rows), block(LA_THREADS);
-    const size_t smem = (size_t)la_smem_layout(a.s, GH, la_stage_rows<CT>() * a.s.row * (int)sizeof(CT) / 4, a.stages).total * 4;
-    switch ((a.s.row + 255) / 256) {
-        case 1: return launch_kernel(latent_attention_kernel<CT, OT, 1, GH>, grid, block, smem, st, pdl, a, a.cl);
-        case 2: return launch_kernel(latent_attention_kernel<CT, OT, 2, GH>, grid, block, smem, st, pdl, a, a.cl);
-        case 3: return launch_kernel(latent_attention_kernel<CT, OT, 3, GH>, grid, block, smem, st, pdl, a, a.cl);
-        default: return launch_kernel(latent_attention_kernel<CT, OT, 4, GH>, grid, block, smem, st, pdl, a, a.cl);
-    }
-}
+// The absorbed form for `rows` rows (row pointers already in `a`): query, scan, output.  chained: the first launch depends
+// programmatically on the kernel before it (decode).
 template <typename CT, typename OT>
-static cudaError_t launch_latent_attention(LatentAttnParams a, int rows, bool pdl, const DeviceInfo& di, cudaStream_t st) {
-    const int gh = (long)a.s.heads * rows * LA_MAX_CL > di.sms && a.s.heads % 2 == 0 ? 2 : 1;
-    const long groups = (long)a.s.heads / gh * rows;
-    a.cl = LA_MAX_CL;
-    while (a.cl > 1 && groups * a.cl > (a.fused ? di.sms : 2L * di.sms)) a.cl >>= 1;
-    a.stages = a.fused ? LA_MAX_STAGES : 2;
-    const int stage_floats = la_stage_rows<CT>() * a.s.row * (int)sizeof(CT) / 4;
-    while (a.stages > 1 && la_smem_layout(a.s, gh, stage_floats, a.stages).total * 4 > di.max_smem_optin - 2048) --a.stages;
-    return gh == 2 ? launch_latent_attention_gh<CT, OT, 2>(a, rows, pdl, st) : launch_latent_attention_gh<CT, OT, 1>(a, rows, pdl, st);
+static cudaError_t launch_latent_attention(LatentAttnParams a, int rows, bool chained, const DeviceInfo& di, cudaStream_t st) {
+    const LatentShape& s = a.s;
+    const long pairs = (long)s.heads * rows;
+    for (a.csplit = 1; a.csplit < 8 && pairs * a.csplit < di.sms;) a.csplit *= 2;
+    for (a.vsplit = 1; a.vsplit < 4 && pairs * a.vsplit < di.sms;) a.vsplit *= 2;
+    a.nsplit = latent_splits(s, rows, di);
+    const int stage = LA_STAGE_ROWS * s.row * (int)sizeof(CT);
+    a.stages = std::max(1, std::min(LA_MAX_STAGES, (di.max_smem_optin - 2048) / stage));
+    cudaError_t e = launch_kernel(latent_query_kernel<CT>, dim3(s.heads * a.csplit + (a.fused ? 1 : 0), rows), dim3(LA_CONSUMERS), 0, st, chained, a);
+    if (e != cudaSuccess) return e;
+    const dim3 grid(latent_groups(s) * a.nsplit, rows), block(LA_SCAN_THREADS);
+    const size_t smem = (size_t)a.stages * stage;
+    switch ((s.row + 255) / 256) {
+        case 1: e = launch_kernel(latent_scan_kernel<CT, 1>, grid, block, smem, st, true, a); break;
+        case 2: e = launch_kernel(latent_scan_kernel<CT, 2>, grid, block, smem, st, true, a); break;
+        case 3: e = launch_kernel(latent_scan_kernel<CT, 3>, grid, block, smem, st, true, a); break;
+        default: e = launch_kernel(latent_scan_kernel<CT, 4>, grid, block, smem, st, true, a); break;
+    }
+    if (e != cudaSuccess) return e;
+    return launch_kernel(latent_output_kernel<OT>, dim3(s.heads * a.vsplit, rows), dim3(LA_CONSUMERS), 0, st, true, a);
 }
 
 // ---- one position ------------------------------------------------------------------------------
@@ -519,7 +537,7 @@ int32_t stack_enqueue_token(StackSession* s, const int* token, const int* pos, f
             a.fused = 1;
             a.status = status;
             CU(m->f32 ? (launch_latent_attention<float, float>(a, 1, true, s->di, st)) : (launch_latent_attention<bf16, float>(a, 1, true, s->di, st)));
-            ++count;
+            count += 3;
         }
         from_vector(p, s->att1);
         L2B_TRY(mv(w.o, p, DE_RESIDUAL, s->x[cur]));
@@ -631,8 +649,17 @@ static int32_t enqueue_latent_rows(StackSession* s, int run, int n, int pos0, co
     const int kstages = prefill_kstages(sh, s->di);
     if (!s->pq || pos_list || n < EXPAND_MIN_ROWS || kstages == 0 || !(sh.scale2 > 0.f)) {
         a.status = status;
-        CU(m->f32 ? (launch_latent_attention<float, float>(a, n, false, s->di, st)) : (launch_latent_attention<bf16, bf16>(a, n, false, s->di, st)));
-        ++*launches;
+        for (int r = 0; r < n; r += ABSORB_ROWS) {
+            const int k = std::min(ABSORB_ROWS, n - r);
+            LatentAttnParams b = a;
+            b.qdg += (size_t)r * a.ld;
+            b.pos0 += r;
+            if (pos_list) b.pos_list += r;
+            b.cache = static_cast<uint8_t*>(a.cache) + (size_t)r * a.cache_stride * act_bytes(m);
+            b.out = static_cast<uint8_t*>(a.out) + (size_t)r * ldo * act_bytes(m);
+            CU(m->f32 ? (launch_latent_attention<float, float>(b, k, false, s->di, st)) : (launch_latent_attention<bf16, bf16>(b, k, false, s->di, st)));
+            *launches += 3;
+        }
         return L2B_OK;
     }
     const int npos = pos0 + n, dq = sh.dp + up(sh.rot, 16);
