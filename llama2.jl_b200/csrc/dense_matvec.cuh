@@ -10,8 +10,9 @@
 //   prologue : the input vector goes to shared memory as f32, after the pending changes of the residual stream (the normalised
 //       per-layer token input, the step vector of a loop pass) and the norm; block 0 writes the changed residual stream back
 //       to its other buffer, because the other blocks still read this one;
-//   weights  : a consumer warp works on 4 rows x 1 chunk of every stage and adds over the stages of its rows in registers; four row
-//       sums are then reduced over the lanes together;
+//   weights  : two groups of four consumer warps take alternate stages (a stage's chain of waits, loads and lane reductions is long
+//       beside the time its bytes take); a warp works on up to two units (4 rows x 1 chunk) of a stage and adds over the
+//       stages of its rows in registers; eight row sums are then reduced over the lanes together;
 //   epilogue : the chunk sums of a row are added in a fixed order by one thread: store | residual add | gelu(gate) * up (rows
 //       2u and 2u+1 of an interleaved matrix) | gelu * token embedding | logits with the block's first maximum.
 // Every mbarrier wait is bounded, as everywhere in the library.
@@ -21,6 +22,7 @@
 namespace l2b {
 
 constexpr int DMV_WARPS = 8, DMV_CONSUMERS = DMV_WARPS * 32, DMV_THREADS = DMV_CONSUMERS + 32, DMV_ROWS = 4;
+constexpr int DMV_GROUPS = 2, DMV_GROUP_WARPS = DMV_WARPS / DMV_GROUPS;
 constexpr int DMV_STAGE = DMV_WARPS * DMV_ROWS * 512, DMV_STAGES = 4;
 
 struct DmvParams {
@@ -57,7 +59,7 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
     if (threadIdx.x == 0) {
         for (int i = 0; i < DMV_STAGES; ++i) {
             mbar_init(s_full + i, 1);
-            mbar_init(s_empty + i, DMV_WARPS);
+            mbar_init(s_empty + i, DMV_GROUP_WARPS);
         }
         fence_barrier_init();
         fence_proxy_async();
@@ -67,13 +69,14 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
     const int u0 = b * p.per_lo + min(b, p.per_rem), nu = p.per_lo + (b < p.per_rem ? 1 : 0);
     const int nr = nu * p.unit;
     const bf16* const wb = p.w + (size_t)u0 * p.unit * p.kp;
-    const int per_stage = DMV_ROWS * p.gs, nstage = (nr + per_stage - 1) / per_stage * p.nseg;
+    const int per_stage = DMV_ROWS * p.gs, nrs = (nr + per_stage - 1) / per_stage;  // row stages; group g takes g, g + 2, ...
     const int seg_vals = p.cs * 256, pitch = p.nseg == 1 ? p.kp : seg_vals;  // values between the rows of a stage
     bool dead = false;
 
     if (warp == DMV_WARPS) {
         const uint64_t policy = policy_evict_first();
-        int row = 0, seg = 0;
+        const int nstage = nrs * p.nseg;
+        int rs = 0, seg = 0;  // order: a pair of row stages at a time, their segments in turn
         for (int j = 0; j < nstage; ++j) {
             const int s = j % DMV_STAGES, use = j / DMV_STAGES;
             if (use > 0 && !mbar_wait_bounded(s_empty + s, (uint32_t)((use - 1) & 1))) {
@@ -81,7 +84,7 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
                 break;
             }
             __syncwarp();
-            const int rows = min(per_stage, nr - row), vals = p.nseg == 1 ? p.kp : min(seg_vals, p.kp - seg * seg_vals);
+            const int row = rs * per_stage, rows = min(per_stage, nr - row), vals = p.nseg == 1 ? p.kp : min(seg_vals, p.kp - seg * seg_vals);
             uint8_t* const dst = dmv_smem + s * DMV_STAGE;
             if (lane == 0) mbar_arrive_expect_tx(s_full + s, (uint32_t)(rows * vals * 2));
             __syncwarp();
@@ -91,9 +94,13 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
             } else if (lane < rows) {
                 bulk_g2s(dst + lane * seg_vals * 2, src + (size_t)lane * p.kp, (uint32_t)(vals * 2), s_full + s, policy);
             }
-            if (++seg == p.nseg) {
+            if (!(rs & 1) && rs + 1 < nrs) {
+                ++rs;
+            } else if (++seg < p.nseg) {
+                rs &= ~1;
+            } else {
                 seg = 0;
-                row += per_stage;
+                ++rs;
             }
             if (j == min(DMV_STAGES, nstage) - 1) {  // the ring is full: what follows it, into L2
                 const size_t total = min((size_t)p.prefetch, (size_t)nr * p.kp * 2);
@@ -152,50 +159,57 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
     partial_sync(DMV_CONSUMERS);
 
     {
-        const int ug = warp / p.cs, uc = warp - ug * p.cs;  // this warp's row group and chunk of a stage
-        const bool mine = ug < p.gs;
-        int row = ug * DMV_ROWS, seg = 0, s = 0;
-        uint32_t par = 0;
-        f32x2 acc[DMV_ROWS];
+        const int grp = warp / DMV_GROUP_WARPS, wg = warp % DMV_GROUP_WARPS;
+        int ug[2], uc[2];  // this warp's units of a stage: row group and chunk
+        bool mine[2];
 #pragma unroll
-        for (int i = 0; i < DMV_ROWS; ++i) acc[i] = 0ull;
-        for (int j = 0; j < nstage; ++j) {
-            if (!dead && !mbar_wait_bounded(s_full + s, par)) dead = true;
-            const int c = seg * p.cs + uc, e = uc * 256 + lane * 8;
-            if (mine && !dead && c * 256 + lane * 8 < p.kp && row < nr) {
-                const uint8_t* src = dmv_smem + s * DMV_STAGE + ((size_t)ug * DMV_ROWS * pitch + e) * 2;
-                uint4 w[DMV_ROWS];
+        for (int t = 0; t < 2; ++t) {
+            const int u = wg + t * DMV_GROUP_WARPS;
+            ug[t] = u / p.cs;
+            uc[t] = u - ug[t] * p.cs;
+            mine[t] = ug[t] < p.gs;
+        }
+#pragma unroll 1
+        for (int rs = grp; rs < nrs; rs += DMV_GROUPS) {
+            const bool paired = (rs | 1) < nrs;  // both row stages of the pair exist
+            const int j0 = (rs & ~1) * p.nseg + (rs & 1);
+            f32x2 acc[2][DMV_ROWS];
 #pragma unroll
-                for (int i = 0; i < DMV_ROWS; ++i) w[i] = *reinterpret_cast<const uint4*>(src + (size_t)i * pitch * 2);
-                const Pairs8 x = read_lane_major(xf, c, lane);
+            for (int t = 0; t < 2; ++t)
 #pragma unroll
-                for (int i = 0; i < DMV_ROWS; ++i) {
-                    acc[i] = fma2(widen2(w[i].x), x.p[0], acc[i]);
-                    acc[i] = fma2(widen2(w[i].y), x.p[1], acc[i]);
-                    acc[i] = fma2(widen2(w[i].z), x.p[2], acc[i]);
-                    acc[i] = fma2(widen2(w[i].w), x.p[3], acc[i]);
+                for (int i = 0; i < DMV_ROWS; ++i) acc[t][i] = 0ull;
+#pragma unroll 1
+            for (int seg = 0; seg < p.nseg; ++seg) {
+                const int j = j0 + (paired ? 2 * seg : seg), s = j % DMV_STAGES;
+                if (!dead && !mbar_wait_bounded(s_full + s, (uint32_t)((j / DMV_STAGES) & 1))) dead = true;
+#pragma unroll
+                for (int t = 0; t < 2; ++t) {
+                    const int c = seg * p.cs + uc[t];
+                    if (mine[t] && !dead && c * 256 + lane * 8 < p.kp) {
+                        const uint8_t* src = dmv_smem + s * DMV_STAGE + (ug[t] * DMV_ROWS * pitch + uc[t] * 256 + lane * 8) * 2;
+                        uint4 w[DMV_ROWS];
+#pragma unroll
+                        for (int i = 0; i < DMV_ROWS; ++i) w[i] = *reinterpret_cast<const uint4*>(src + i * pitch * 2);
+                        const Pairs8 x = read_lane_major(xf, c, lane);
+#pragma unroll
+                        for (int i = 0; i < DMV_ROWS; ++i) {
+                            acc[t][i] = fma2(widen2(w[i].x), x.p[0], acc[t][i]);
+                            acc[t][i] = fma2(widen2(w[i].y), x.p[1], acc[t][i]);
+                            acc[t][i] = fma2(widen2(w[i].z), x.p[2], acc[t][i]);
+                            acc[t][i] = fma2(widen2(w[i].w), x.p[3], acc[t][i]);
+                        }
+                    }
                 }
+                __syncwarp();
+                if (lane == 0) mbar_arrive(s_empty + s);
             }
-            __syncwarp();
-            if (lane == 0) mbar_arrive(s_empty + s);
-            if (++s == DMV_STAGES) s = 0, par ^= 1u;
-            if (++seg == p.nseg) {
-                seg = 0;
-                if (mine) {  // (uniform over the warp) four sums over the lanes at once: lanes 8q .. 8q+7 end up with row q
-                    float a[DMV_ROWS];
+            float a[2 * DMV_ROWS];
 #pragma unroll
-                    for (int i = 0; i < DMV_ROWS; ++i) a[i] = sum2(acc[i]), acc[i] = 0ull;
-                    const bool hi = lane & 16, mid = lane & 8;
-                    float v0 = (hi ? a[2] : a[0]) + __shfl_xor_sync(0xffffffffu, hi ? a[0] : a[2], 16);
-                    float v1 = (hi ? a[3] : a[1]) + __shfl_xor_sync(0xffffffffu, hi ? a[1] : a[3], 16);
-                    float v = (mid ? v1 : v0) + __shfl_xor_sync(0xffffffffu, mid ? v0 : v1, 8);
-                    v += __shfl_xor_sync(0xffffffffu, v, 4);
-                    v += __shfl_xor_sync(0xffffffffu, v, 2);
-                    v += __shfl_xor_sync(0xffffffffu, v, 1);
-                    if ((lane & 7) == 0) part[(row + (lane >> 3)) * p.cs + uc] = v;
-                }
-                row += per_stage;
-            }
+            for (int i = 0; i < 2 * DMV_ROWS; ++i) a[i] = sum2(acc[i / DMV_ROWS][i % DMV_ROWS]);
+            const float v = warp_sums_spread<2 * DMV_ROWS>(a);  // lanes 4i .. 4i+3 hold sum i
+            const int i = lane >> 2, t = i / DMV_ROWS;
+            if ((lane & 3) == 0 && (t ? mine[1] : mine[0]))
+                part[(rs * per_stage + (t ? ug[1] : ug[0]) * DMV_ROWS + i % DMV_ROWS) * p.cs + (t ? uc[1] : uc[0])] = v;
         }
         if (dead && lane == 0) atomicExch(p.status, DEV_ERR_TMA_TIMEOUT);
     }

@@ -48,10 +48,10 @@ __device__ __forceinline__ Pairs8 read_lane_major(const float* x, int c, int lan
     return o;
 }
 
-// N sums over the lanes of a warp at once; every lane gets all of them.  While more than one value is left, a step exchanges half of
-// the values across a lane bit and halves their number; the remaining bits are reduced as usual.
+// N sums over the lanes of a warp at once.  While more than one value is left, a step exchanges half of the values across a lane bit
+// and halves their number; the remaining bits are reduced as usual.  Lanes i * 32/N .. end up with sum i.
 template <int N>
-__device__ __forceinline__ void warp_sums(float (&v)[N]) {
+__device__ __forceinline__ float warp_sums_spread(const float (&v)[N]) {
     static_assert(N == 1 || N == 2 || N == 4 || N == 8, "number of sums");
     const int lane = threadIdx.x & 31;
     float t[N];
@@ -69,13 +69,14 @@ __device__ __forceinline__ void warp_sums(float (&v)[N]) {
     }
 #pragma unroll
     for (; o > 0; o >>= 1) t[0] += __shfl_xor_sync(0xffffffffu, t[0], o);
+    return t[0];
+}
+// The same with every lane getting all sums.
+template <int N>
+__device__ __forceinline__ void warp_sums(float (&v)[N]) {
+    const float t = warp_sums_spread<N>(v);
 #pragma unroll
-    for (int i = 0; i < N; ++i) {  // value i sits in the lanes whose upper bits spell i
-        int src = 0, bit = 16;
-#pragma unroll
-        for (int n = N; n > 1; n >>= 1, bit >>= 1) src += (i & (n / 2)) ? bit : 0;
-        v[i] = N > 1 ? __shfl_sync(0xffffffffu, t[0], src) : t[0];
-    }
+    for (int i = 0; i < N; ++i) v[i] = N > 1 ? __shfl_sync(0xffffffffu, t, i * (32 / N)) : t;
 }
 
 // eight consecutive values (16-byte aligned bf16, 32-byte aligned f32) as f32
