@@ -17,13 +17,15 @@
 //       2u and 2u+1 of an interleaved matrix) | gelu * token embedding | logits with the block's first maximum.
 // Every mbarrier wait is bounded, as everywhere in the library.
 #pragma once
+#include <algorithm>
+
 #include "dense_ops.cuh"
 
 namespace l2b {
 
 constexpr int DMV_WARPS = 8, DMV_CONSUMERS = DMV_WARPS * 32, DMV_THREADS = DMV_CONSUMERS + 32, DMV_ROWS = 4;
 constexpr int DMV_GROUPS = 2, DMV_GROUP_WARPS = DMV_WARPS / DMV_GROUPS;
-constexpr int DMV_STAGE = DMV_WARPS * DMV_ROWS * 512, DMV_STAGES = 4;
+constexpr int DMV_STAGE = DMV_WARPS * DMV_ROWS * 512, DMV_MAX_STAGES = 11;
 
 struct DmvParams {
     const bf16* w;          // [rows][kp], kp a multiple of 8
@@ -32,6 +34,7 @@ struct DmvParams {
     int per_lo, per_rem;    // results of block b: per_lo + (b < per_rem), contiguous
     int nchunk;             // 256-value chunks per row
     int gs, cs, nseg;       // a stage: 4 * gs rows x cs chunks (gs * cs <= 8); nseg stages per row group, gs = 1 when nseg > 1
+    int stages;             // ring slots
     int prefetch;           // bytes of the block's rows to have in flight before the wait, ring included
     const float* x;         // input vector [k]
     ResidualUpdate upd;
@@ -42,22 +45,29 @@ struct DmvParams {
     int* amax_idx;
     int* status;
 };
-inline size_t dmv_smem_bytes(const DmvParams& p) {
+// Shared memory beside the ring, and ring slots: as many as fit and are of use (bytes in flight are what the HBM rate needs: with
+// 64 KiB per SM the stream stays below 4.2 TB/s).
+inline size_t dmv_fixed_bytes(const DmvParams& p) {
     const int rows = p.unit * (p.per_lo + (p.per_rem ? 1 : 0)), per_stage = DMV_ROWS * p.gs;
-    return (size_t)DMV_STAGES * DMV_STAGE + ((size_t)p.nchunk * 256 + (size_t)((rows + per_stage - 1) / per_stage * per_stage) * p.cs) * 4;
+    return ((size_t)p.nchunk * 256 + (size_t)((rows + per_stage - 1) / per_stage * per_stage) * p.cs) * 4;
+}
+inline int dmv_choose_stages(const DmvParams& p, size_t max_smem) {
+    const int rows = p.unit * (p.per_lo + (p.per_rem ? 1 : 0)), per_stage = DMV_ROWS * p.gs;
+    const long fit = ((long)max_smem - (long)dmv_fixed_bytes(p)) / DMV_STAGE, use = (long)((rows + per_stage - 1) / per_stage) * p.nseg;
+    return (int)std::min<long>(DMV_MAX_STAGES, std::min<long>(fit, std::max<long>(use, 2)));
 }
 
 __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __grid_constant__ DmvParams p) {
     extern __shared__ __align__(128) uint8_t dmv_smem[];
-    __shared__ __align__(8) uint64_t s_full[DMV_STAGES], s_empty[DMV_STAGES];
+    __shared__ __align__(8) uint64_t s_full[DMV_MAX_STAGES], s_empty[DMV_MAX_STAGES];
     __shared__ float s_red[DMV_WARPS];
     __shared__ int s_idx[DMV_WARPS];
-    float* const xf = reinterpret_cast<float*>(dmv_smem + DMV_STAGES * DMV_STAGE);
+    float* const xf = reinterpret_cast<float*>(dmv_smem + p.stages * DMV_STAGE);
     float* const part = xf + p.nchunk * 256;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     pdl_launch_dependents();
     if (threadIdx.x == 0) {
-        for (int i = 0; i < DMV_STAGES; ++i) {
+        for (int i = 0; i < p.stages; ++i) {
             mbar_init(s_full + i, 1);
             mbar_init(s_empty + i, DMV_GROUP_WARPS);
         }
@@ -76,9 +86,9 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
     if (warp == DMV_WARPS) {
         const uint64_t policy = policy_evict_first();
         const int nstage = nrs * p.nseg;
+        int s = 0, use = 0;
         int rs = 0, seg = 0;  // order: a pair of row stages at a time, their segments in turn
         for (int j = 0; j < nstage; ++j) {
-            const int s = j % DMV_STAGES, use = j / DMV_STAGES;
             if (use > 0 && !mbar_wait_bounded(s_empty + s, (uint32_t)((use - 1) & 1))) {
                 dead = true;
                 break;
@@ -102,7 +112,8 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
                 seg = 0;
                 ++rs;
             }
-            if (j == min(DMV_STAGES, nstage) - 1) {  // the ring is full: what follows it, into L2
+            if (++s == p.stages) s = 0, ++use;
+            if (j == min(p.stages, nstage) - 1) {  // the ring is full: what follows it, into L2
                 const size_t total = min((size_t)p.prefetch, (size_t)nr * p.kp * 2);
                 for (size_t o = (size_t)row * p.kp * 2 + (size_t)lane * 4096; o < total; o += 32 * 4096)
                     asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(reinterpret_cast<const char*>(wb) + o), "r"((uint32_t)min((size_t)4096, total - o))
@@ -162,6 +173,8 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
         const int grp = warp / DMV_GROUP_WARPS, wg = warp % DMV_GROUP_WARPS;
         int ug[2], uc[2];  // this warp's units of a stage: row group and chunk
         bool mine[2];
+        int s = grp;       // ring slot of this group's next stage
+        uint32_t par = 0;
 #pragma unroll
         for (int t = 0; t < 2; ++t) {
             const int u = wg + t * DMV_GROUP_WARPS;
@@ -172,7 +185,6 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
 #pragma unroll 1
         for (int rs = grp; rs < nrs; rs += DMV_GROUPS) {
             const bool paired = (rs | 1) < nrs;  // both row stages of the pair exist
-            const int j0 = (rs & ~1) * p.nseg + (rs & 1);
             f32x2 acc[2][DMV_ROWS];
 #pragma unroll
             for (int t = 0; t < 2; ++t)
@@ -180,8 +192,7 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
                 for (int i = 0; i < DMV_ROWS; ++i) acc[t][i] = 0ull;
 #pragma unroll 1
             for (int seg = 0; seg < p.nseg; ++seg) {
-                const int j = j0 + (paired ? 2 * seg : seg), s = j % DMV_STAGES;
-                if (!dead && !mbar_wait_bounded(s_full + s, (uint32_t)((j / DMV_STAGES) & 1))) dead = true;
+                if (!dead && !mbar_wait_bounded(s_full + s, par)) dead = true;
 #pragma unroll
                 for (int t = 0; t < 2; ++t) {
                     const int c = seg * p.cs + uc[t];
@@ -202,6 +213,8 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
                 }
                 __syncwarp();
                 if (lane == 0) mbar_arrive(s_empty + s);
+                s += paired ? 2 : 1;  // the other group's stage of the pair lies between
+                if (s >= p.stages) s -= p.stages, par ^= 1u;
             }
             float a[2 * DMV_ROWS];
 #pragma unroll

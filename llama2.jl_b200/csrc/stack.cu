@@ -477,8 +477,9 @@ static int32_t launch_dense_matvec(const StackSession* s, const StackMatrix& w, 
     p.nseg = (p.nchunk + p.cs - 1) / p.cs;
     p.gs = p.nseg == 1 ? DMV_WARPS / p.cs : 1;
     p.prefetch = 256 * 1024;
-    const size_t smem = dmv_smem_bytes(p);
-    if (smem > (size_t)s->di.max_smem_optin - 1024) return fail(L2B_ERR_BAD_ARG, "input vector too long for shared memory");
+    p.stages = dmv_choose_stages(p, (size_t)s->di.max_smem_optin - 2048);
+    if (p.stages < 2) return fail(L2B_ERR_BAD_ARG, "input vector too long for shared memory");
+    const size_t smem = (size_t)p.stages * DMV_STAGE + dmv_fixed_bytes(p);
     CU(launch_kernel(dense_matvec_kernel, dim3(grid), dim3(DMV_THREADS), smem, st, true, p));
     if (nblocks) *nblocks = grid;
     return L2B_OK;
