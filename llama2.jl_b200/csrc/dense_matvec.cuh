@@ -4,9 +4,7 @@
 // One block per SM, 8 consumer warps and a producer warp, every block a contiguous range of rows.
 //   producer : a stage is 4 * gs rows x cs 256-value chunks (16 KiB at most); stages come into a ring with bulk asynchronous copies
 //       (one copy of adjacent whole rows, or one per row when rows are longer than a stage).  Weights are constants, so
-//       the ring is filled, and the rows behind it are prefetched into L2, BEFORE the wait on the previous kernel
-//       (programmatic dependent launch).  The block is small enough in shared memory for the next kernel's block to do the same
-//       beside it;
+//       the ring is filled BEFORE the wait on the previous kernel (programmatic dependent launch);
 //   prologue : the input vector goes to shared memory as f32, after the pending changes of the residual stream (the normalised
 //       per-layer token input, the step vector of a loop pass) and the norm; block 0 writes the changed residual stream back
 //       to its other buffer, because the other blocks still read this one;
@@ -35,7 +33,6 @@ struct DmvParams {
     int nchunk;             // 256-value chunks per row
     int gs, cs, nseg;       // a stage: 4 * gs rows x cs chunks (gs * cs <= 8); nseg stages per row group, gs = 1 when nseg > 1
     int stages;             // ring slots
-    int prefetch;           // bytes of the block's rows to have in flight before the wait, ring included
     const float* x;         // input vector [k]
     ResidualUpdate upd;
     float* x_out;           // block 0 writes the updated vector here (null: no update)
@@ -113,12 +110,6 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
                 ++rs;
             }
             if (++s == p.stages) s = 0, ++use;
-            if (j == min(p.stages, nstage) - 1) {  // the ring is full: what follows it, into L2
-                const size_t total = min((size_t)p.prefetch, (size_t)nr * p.kp * 2);
-                for (size_t o = (size_t)row * p.kp * 2 + (size_t)lane * 4096; o < total; o += 32 * 4096)
-                    asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(reinterpret_cast<const char*>(wb) + o), "r"((uint32_t)min((size_t)4096, total - o))
-                                 : "memory");
-            }
         }
         if (dead) {
             if (lane == 0) atomicExch(p.status, DEV_ERR_TMA_TIMEOUT);

@@ -476,7 +476,6 @@ static int32_t launch_dense_matvec(const StackSession* s, const StackMatrix& w, 
     p.cs = (p.nchunk + p.nseg - 1) / p.nseg;
     p.nseg = (p.nchunk + p.cs - 1) / p.cs;
     p.gs = p.nseg == 1 ? DMV_WARPS / p.cs : 1;
-    p.prefetch = 256 * 1024;
     p.stages = dmv_choose_stages(p, (size_t)s->di.max_smem_optin - 2048);
     if (p.stages < 2) return fail(L2B_ERR_BAD_ARG, "input vector too long for shared memory");
     const size_t smem = (size_t)p.stages * DMV_STAGE + dmv_fixed_bytes(p);
