@@ -214,6 +214,15 @@ __device__ __forceinline__ float apply_norm(const NormParams& n, float x, int i)
 // Barrier over the first `threads` threads of the block.
 __device__ __forceinline__ void partial_sync(int threads) { asm volatile("bar.sync 1, %0;" ::"r"(threads) : "memory"); }
 
+__device__ __forceinline__ void partial_sync_2(int threads) { asm volatile("bar.sync 2, %0;" ::"r"(threads) : "memory"); }  // any `threads` threads
+
+// 2^x as one special-function instruction (about 2 ulp; results below the normal range become 0)
+__device__ __forceinline__ float fast_exp2(float x) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+    return r;
+}
+
 // Sum over the first NW warps of a block; each of their threads gets it.  s holds NW floats and may be reused after the next barrier.
 template <int NW>
 __device__ __forceinline__ float block_sum_all(float v, float* s) {

@@ -6,8 +6,10 @@
 // One block = 128 queries of one head:
 //   warp 0     producer: TMA tiled copies of Q (once), [K | kr] and V per key tile
 //   warp 1     MMA issue: S_j = Q K_j^T into one of two 128-column buffers of tensor memory, one tile ahead of O += P_j V_j
-//   warps 2-5  thread = query: scores from tensor memory, scale, causal mask, running maximum and sum in f32 (exp2 domain);
-//              P_j as bf16 into shared memory in operand layout.  O is rescaled in tensor memory only when a row's maximum has
+//   warps 2-9  two threads per query, each with half of the tile's keys: scores from tensor memory, scale, causal mask, running
+//              maximum (shared between the two) and sum in f32 (exp2 domain); P_j as bf16 into shared memory in operand
+//              layout.  The scores are read twice, for the maximum and for the exponentials, in short loops: with all of them in
+//              registers the unrolled code no longer fits the instruction cache.  O is rescaled in tensor memory only when a row's maximum has
 //              grown by more than 2^8 since it was last taken; the end divides by sum + exp(sink), applies the output gate
 //              and stores the operand of the output projection.
 // Every mbarrier wait is bounded, as in the GEMM.
@@ -17,7 +19,7 @@
 
 namespace l2b {
 
-constexpr int LP_TILE = 128, LP_THREADS = 192, LP_SUB = 128 * 128;  // bytes of a 128-row x 64-value operand tile
+constexpr int LP_TILE = 128, LP_WARPS = 8, LP_THREADS = 64 + LP_WARPS * 32, LP_SUB = 128 * 128;  // bytes of a 128-row x 64-value operand tile
 
 struct LatentPrefillParams {
     int n, pos0;              // queries at positions pos0 .. pos0 + n - 1
@@ -55,6 +57,7 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prefill_kernel(const __grid
     extern __shared__ __align__(1024) uint8_t lp_raw[];
     __shared__ __align__(8) uint64_t s_q, s_k[2], s_kfree[2], s_v, s_s[2], s_sfree[2], s_p, s_o;
     __shared__ uint32_t s_tmem;
+    __shared__ float s_row[2][2][LP_TILE];  // [tile parity][half][query]: the halves' maxima (at the end: sums)
     uint8_t* smem = lp_raw + ((1024u - (smem_u32(lp_raw) & 1023u)) & 1023u);
     const LpSmem L = lp_smem_layout(p.dim, p.rot, p.vp, p.kstages);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -64,13 +67,13 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prefill_kernel(const __grid
     if (threadIdx.x == 0) {
         mbar_init(&s_q, 1);
         mbar_init(&s_v, 1);
-        mbar_init(&s_p, 4);
+        mbar_init(&s_p, LP_WARPS);
         mbar_init(&s_o, 1);
         for (int i = 0; i < 2; ++i) {
             mbar_init(s_k + i, 1);
             mbar_init(s_kfree + i, 1);
             mbar_init(s_s + i, 1);
-            mbar_init(s_sfree + i, 4);
+            mbar_init(s_sfree + i, LP_WARPS);
         }
         fence_barrier_init();
         fence_proxy_async();
@@ -148,51 +151,44 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prefill_kernel(const __grid
             if (!ok) atomicExch(p.status, DEV_ERR_TMA_TIMEOUT);
         }
     } else {
-        const int qd = warp & 3, r = 32 * qd + lane;
+        const int qd = warp & 3, half = (warp - 2) >> 2, r = 32 * qd + lane;
         const uint32_t lane_off = (uint32_t)(32 * qd) << 16;
         const int qi = q0 + r, qpos = p.pos0 + qi;
         float m = -INFINITY, l = 0.f;
         bool ok = true;
         for (int j = 0; j < nt; ++j) {
             const int b = j & 1;
-            if (!__all_sync(0xffffffffu, mbar_wait_bounded(s_s + b, (uint32_t)((j >> 1) & 1)))) {
-                ok = false;
-                break;
-            }
+            if (ok && !__all_sync(0xffffffffu, mbar_wait_bounded(s_s + b, (uint32_t)((j >> 1) & 1)))) ok = false;
             tc_fence_after();
-            float s[4][32];
-#pragma unroll
-            for (int c = 0; c < 4; ++c) tmem_ld32f(tmem + lane_off + (uint32_t)(b * 128 + 32 * c), s[c]);
-            tc_fence_before();
-            __syncwarp();
-            if (lane == 0) mbar_arrive(s_sfree + b);
-            const int lim = qpos - j * LP_TILE;  // keys 0 .. lim of the tile are seen
-            if (j * LP_TILE + LP_TILE - 1 > p.pos0 + q0) {  // (the last tiles only)
-#pragma unroll
-                for (int c = 0; c < 4; ++c)
+            const uint32_t ts = tmem + lane_off + (uint32_t)(b * 128 + half * 64);
+            const int lim = qpos - j * LP_TILE - half * 64;                       // keys 0 .. lim of this half are seen
+            const bool masked = j * LP_TILE + LP_TILE - 1 > p.pos0 + q0;           // (the last tiles only)
+            float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll 1
+            for (int c = 0; c < 64; c += 32) {
+                float s[32];
+                tmem_ld32f(ts + (uint32_t)c, s);
+                if (masked) {
 #pragma unroll
                     for (int k = 0; k < 32; ++k)
-                        if (32 * c + k > lim) s[c][k] = -INFINITY;
-            }
-            float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+                        if (c + k > lim) s[k] = -INFINITY;
+                }
 #pragma unroll
-            for (int c = 0; c < 4; ++c)
-#pragma unroll
-                for (int k = 0; k < 32; ++k) m4[k & 3] = fmaxf(m4[k & 3], s[c][k]);
-            const float mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3])) * p.scale2;  // (scale2 > 0)
-            if (j > 0 && !__all_sync(0xffffffffu, mbar_wait_bounded(&s_o, (uint32_t)((j - 1) & 1)))) {  // P and O are free
-                ok = false;
-                break;
+                for (int k = 0; k < 32; ++k) m4[k & 3] = fmaxf(m4[k & 3], s[k]);
             }
+            s_row[b][half][r] = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3]));
+            partial_sync_2(LP_WARPS * 32);
+            const float mx = fmaxf(s_row[b][0][r], s_row[b][1][r]) * p.scale2;  // (scale2 > 0; key 0 is seen, so the first is finite)
+            if (ok && j > 0 && !__all_sync(0xffffffffu, mbar_wait_bounded(&s_o, (uint32_t)((j - 1) & 1)))) ok = false;  // P and O are free
             tc_fence_after();
             if (j == 0) {
                 m = mx;
-            } else if (__any_sync(0xffffffffu, mx > m + 8.f)) {
-                const float mn = mx > m + 8.f ? mx : m, corr = exp2f(m - mn);
+            } else if (__any_sync(0xffffffffu, mx > m + 8.f)) {  // (the same decision in both halves)
+                const float mn = mx > m + 8.f ? mx : m, corr = fast_exp2(m - mn);
                 l *= corr;
                 m = mn;
 #pragma unroll 1
-                for (int c = 0; c < p.vp; c += 32) {
+                for (int c = 32 * half; c < p.vp; c += 64) {
                     float o[32];
                     tmem_ld32f(tmem_o + lane_off + (uint32_t)c, o);
 #pragma unroll
@@ -201,39 +197,55 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prefill_kernel(const __grid
                 }
             }
             float l4[4] = {0.f, 0.f, 0.f, 0.f};
+            uint8_t* const pr = smem + L.p + half * LP_SUB + r * 128;
+#pragma unroll 1
+            for (int c = 0; c < 64; c += 32) {
+                float s[32];
+                tmem_ld32f(ts + (uint32_t)c, s);
 #pragma unroll
-            for (int c = 0; c < 4; ++c)
+                for (int k = 0; k < 32; ++k) s[k] = fast_exp2(fmaf(s[k], p.scale2, -m));
+                if (masked) {
+#pragma unroll
+                    for (int k = 0; k < 32; ++k)
+                        if (c + k > lim) s[k] = 0.f;
+                }
+#pragma unroll
+                for (int k = 0; k < 32; ++k) l4[k & 3] += s[k];
 #pragma unroll
                 for (int g = 0; g < 4; ++g) {  // 8 keys = one 16-byte chunk of the operand row, chunk index xor row (128-byte swizzle)
                     uint32_t w[4];
 #pragma unroll
                     for (int k = 0; k < 4; ++k) {
-                        const float e0 = exp2f(fmaf(s[c][8 * g + 2 * k], p.scale2, -m)), e1 = exp2f(fmaf(s[c][8 * g + 2 * k + 1], p.scale2, -m));
-                        l4[k] += e0 + e1;
-                        const __nv_bfloat162 pk = __floats2bfloat162_rn(e0, e1);
+                        const __nv_bfloat162 pk = __floats2bfloat162_rn(s[8 * g + 2 * k], s[8 * g + 2 * k + 1]);
                         w[k] = *reinterpret_cast<const uint32_t*>(&pk);
                     }
-                    const int chunk = 4 * (c & 1) + g;
-                    *reinterpret_cast<uint4*>(smem + L.p + (c >> 1) * LP_SUB + r * 128 + ((chunk ^ (r & 7)) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);
+                    *reinterpret_cast<uint4*>(pr + (((c >> 3) + g) ^ (r & 7)) * 16) = make_uint4(w[0], w[1], w[2], w[3]);
                 }
+            }
             l += (l4[0] + l4[1]) + (l4[2] + l4[3]);
             fence_proxy_async();
             tc_fence_before();
             __syncwarp();
-            if (lane == 0) mbar_arrive(&s_p);
+            if (lane == 0) {
+                mbar_arrive(s_sfree + b);
+                mbar_arrive(&s_p);
+            }
         }
         if (ok && !__all_sync(0xffffffffu, mbar_wait_bounded(&s_o, (uint32_t)((nt - 1) & 1)))) ok = false;
+        s_row[nt & 1][half][r] = l;
+        partial_sync_2(LP_WARPS * 32);
         if (!ok) {
             if (lane == 0) atomicExch(p.status, DEV_ERR_TMA_TIMEOUT);
         } else {
             tc_fence_after();
+            l = s_row[nt & 1][0][r] + s_row[nt & 1][1][r];
             const float inv = 1.f / (l + exp2f(__ldg(p.sink + h) * 1.4426950408889634f - m));  // the sink: a term of the denominator only
             bf16* out = p.out + (size_t)qi * p.ldo + h * p.vdim;
             const bool wide = ((p.vdim | p.ldo) & 7) == 0;
-            // gates of this warp's 32 queries, 32 values at a time, through the shared memory that held P (its last product is done)
-            float* const sg = reinterpret_cast<float*>(smem + L.p) + qd * (32 * 33);
+            // gates of this warp's 32 queries, 32 values at a time, through the shared memory that held Q and K (all products are done)
+            float* const sg = reinterpret_cast<float*>(smem + L.q) + (warp - 2) * (32 * 33);
 #pragma unroll 1
-            for (int c = 0; c < p.vdim; c += 32) {
+            for (int c = 32 * half; c < p.vdim; c += 64) {
                 float o[32];
                 __syncwarp();
 #pragma unroll
@@ -242,12 +254,12 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prefill_kernel(const __grid
                     o[i] = t < p.n && c + lane < p.vdim ? __ldg(p.gate + (size_t)t * p.ld + h * p.vdim + c + lane) : 0.f;
                 }
 #pragma unroll
-                for (int i = 0; i < 32; ++i) sg[i * 33 + lane] = o[i];
+                for (int i = 0; i < 32; ++i) sg[i * 33 + lane] = sigmoid(o[i]);
                 __syncwarp();
                 tmem_ld32f(tmem_o + lane_off + (uint32_t)c, o);
                 const int nv = qi < p.n ? p.vdim - c : 0;  // values of this query to store
 #pragma unroll
-                for (int k = 0; k < 32; ++k) o[k] *= inv * sigmoid(sg[lane * 33 + k]);
+                for (int k = 0; k < 32; ++k) o[k] *= inv * sg[lane * 33 + k];
                 if (wide) {
 #pragma unroll
                     for (int g = 0; g < 4; ++g)

@@ -595,9 +595,14 @@ static int32_t launch_gemm(const StackSession* s, const StackMatrix& w, const vo
         CU(cudaGetLastError());
         return L2B_OK;
     }
-    const int bn = n <= 32 ? 32 : n <= 64 ? 64 : 128;
-    const long tiles = (long)((rows + 127) / 128) * ((n + bn - 1) / bn);
-    const int na = w.pair == 2 || tiles > 2L * s->di.sms ? 2 : 1;
+    // Token tile: as wide as the rows there are, narrower while the tiles do not fill the GPU.  Weight tiles per block: what takes fewer
+    // rounds of the GPU, a round of two weight tiles costing about 1.55 rounds of one (2 when short products leave the epilogue exposed).
+    auto up_div = [](long a, long b) { return (a + b - 1) / b; };
+    const long sms = s->di.sms;
+    int bn = n <= 32 ? 32 : n <= 64 ? 64 : 128;
+    while (bn > 32 && up_div(rows, 128) * up_div(n, bn) < sms) bn /= 2;
+    const double one = (double)up_div(up_div(rows, 128) * up_div(n, bn), sms), two = (w.k < 1024 ? 2.0 : 1.55) * (double)up_div(up_div(rows, 256) * up_div(n, bn), sms);
+    const int na = w.pair == 2 || two < one ? 2 : 1;
     GemmDenseParams g;
     memset(&g, 0, sizeof(g));
     g.rows = rows; g.n_tok = n; g.k = w.k; g.epi = epi; g.status = status;
