@@ -59,6 +59,9 @@ __device__ __forceinline__ int latent_position(const LatentAttnParams& p, int ro
 // positions per range
 __device__ __forceinline__ int latent_range(int npos, int nsplit) { return max(LA_MIN_RANGE, (npos + nsplit - 1) / nsplit); }
 
+__device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory"); }
+__device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory"); }
+
 // Latent (normalised) and rotated key of one position into its cache row; NW warps.
 template <typename CT, int NW>
 __device__ __forceinline__ void store_latent_row(const LatentAttnParams& p, int row, int pos, float* s_red) {
@@ -287,22 +290,31 @@ __global__ void __launch_bounds__(LA_SCAN_THREADS) latent_scan_kernel(const __gr
     }
 }
 
-// Grid (heads * vsplit, rows): merge of the ranges, then this block's rows of W_uv (four at a time per warp), gated.
+// Grid (heads * vsplit, rows), clusters of the vsplit blocks of a head: each merges the ranges for its part of the latent and hands
+// that part to the others through distributed shared memory, then applies its rows of W_uv (four at a time per warp) and the gate.
 template <typename OT>
 __global__ void __launch_bounds__(LA_CONSUMERS) latent_output_kernel(const __grid_constant__ LatentAttnParams p) {
     __shared__ float s_w[LA_MAX_SPLIT];
     __shared__ __align__(16) float s_c[1024];
-    constexpr int UR = 4;
+    __shared__ float2 s_part[512];
+    constexpr int UR = 4, PRE = 2;  // rows per warp at a time; 256-value pieces of the first rows fetched before the wait
     const LatentShape& S = p.s;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, row = (int)blockIdx.y;
-    const int h = (int)blockIdx.x / p.vsplit, part = (int)blockIdx.x % p.vsplit;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, row = (int)blockIdx.y, cl = p.vsplit;
+    const int h = (int)blockIdx.x / cl, part = (int)blockIdx.x % cl;
     pdl_launch_dependents();
-    const int vpc = (S.vdim + p.vsplit - 1) / p.vsplit, v0 = min(S.vdim, part * vpc), v1 = min(S.vdim, v0 + vpc);
+    if (cl > 1) cluster_arrive();  // (waited for before the first store into another block's shared memory)
+    const int vpc = (S.vdim + cl - 1) / cl, v0 = min(S.vdim, part * vpc), v1 = min(S.vdim, v0 + vpc);
     const bf16* const uv = p.uv + (size_t)h * S.vp * S.rp;
-    {
-        const char* w = reinterpret_cast<const char*>(uv + (size_t)v0 * S.rp);
-        for (size_t o = (size_t)tid * 128; o < (size_t)(v1 - v0) * S.rp * 2; o += LA_CONSUMERS * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(w + o));
-    }
+    const int rw = v0 + warp * UR;
+    Raw8<bf16> pre[PRE][UR];
+#pragma unroll
+    for (int i = 0; i < PRE; ++i)
+#pragma unroll
+        for (int u = 0; u < UR; ++u) {
+            const int e = (i * 32 + lane) * 8;
+            pre[i][u].zero();
+            if (rw < v1 && e < S.rp) pre[i][u].load(uv + (size_t)min(rw + u, v1 - 1) * S.rp + e);
+        }
     const int npos = latent_position(p, row) + 1, range = latent_range(npos, p.nsplit), ns = (npos + range - 1) / range;
     pdl_wait();
     const size_t slot = ((size_t)row * S.heads + h) * p.nsplit;
@@ -316,42 +328,75 @@ __global__ void __launch_bounds__(LA_CONSUMERS) latent_output_kernel(const __gri
         s_w[lane] = wa * inv;
         s_w[lane + 32] = wb * inv;
     }
-    __syncthreads();
-    for (int i = tid * 2; i < S.rp; i += LA_CONSUMERS * 2) {
-        float2 a = make_float2(0.f, 0.f);
-        const float* src = p.part_acc + slot * S.rp + i;
-#pragma unroll 8
-        for (int r = 0; r < ns; ++r, src += S.rp) {
-            const float2 x = __ldcg(reinterpret_cast<const float2*>(src));
-            a.x = fmaf(x.x, s_w[r], a.x);
-            a.y = fmaf(x.y, s_w[r], a.y);
-        }
-        *reinterpret_cast<float2*>(s_c + i) = a;
-    }
-    __syncthreads();
     const float* const gate = p.qdg + (size_t)row * p.ld + p.off_g + h * S.vdim;
+    const float g0 = lane < UR && rw + lane < v1 ? __ldcg(gate + rw + lane) : 0.f;
+    __syncthreads();
+    {
+        const int cs = (S.rp / 8 + cl - 1) / cl * 8, c0 = min(S.rp, part * cs), np = (min(S.rp, c0 + cs) - c0) / 2;  // this block's column pairs
+        const int nsg = np > 0 ? max(1, min(LA_CONSUMERS / np, 8)) : 0;                                              // threads per pair
+        for (int i = tid; i < np * nsg; i += LA_CONSUMERS) {
+            const int cp = i % np, sg = i / np;
+            float2 a = make_float2(0.f, 0.f);
+            const float* const src = p.part_acc + slot * S.rp + c0 + 2 * cp;
+#pragma unroll 8
+            for (int r = sg; r < ns; r += nsg) {
+                const float2 x = __ldcg(reinterpret_cast<const float2*>(src + (size_t)r * S.rp));
+                a.x = fmaf(x.x, s_w[r], a.x);
+                a.y = fmaf(x.y, s_w[r], a.y);
+            }
+            s_part[i] = a;
+        }
+        __syncthreads();
+        if (cl > 1) cluster_wait();
+        for (int i = tid; i < np; i += LA_CONSUMERS) {
+            float2 a = s_part[i];
+            for (int k = 1; k < nsg; ++k) {
+                const float2 x = s_part[k * np + i];
+                a.x += x.x;
+                a.y += x.y;
+            }
+            float* const at = s_c + c0 + 2 * i;
+            if (cl == 1) *reinterpret_cast<float2*>(at) = a;
+            else
+                for (int r = 0; r < cl; ++r) {
+                    st_cluster_f32(cluster_map(at, (uint32_t)r), a.x);
+                    st_cluster_f32(cluster_map(at + 1, (uint32_t)r), a.y);
+                }
+        }
+        if (cl > 1) cluster_sync_all();
+        else __syncthreads();
+    }
     OT* const out = static_cast<OT*>(p.out) + (size_t)row * p.ldo + h * S.vdim;
 #pragma unroll 1
-    for (int r0 = v0 + warp * UR; r0 < v1; r0 += LA_WARPS * UR) {
+    for (int r0 = rw; r0 < v1; r0 += LA_WARPS * UR) {
         float d[UR];
 #pragma unroll
         for (int u = 0; u < UR; ++u) d[u] = 0.f;
-#pragma unroll 2
-        for (int e = lane * 8; e < S.rp; e += 256) {
-            Raw8<bf16> w[UR];
-#pragma unroll
-            for (int u = 0; u < UR; ++u) w[u].load(uv + (size_t)min(r0 + u, v1 - 1) * S.rp + e);
-            const ulonglong2 c0 = *reinterpret_cast<const ulonglong2*>(s_c + e), c1 = *reinterpret_cast<const ulonglong2*>(s_c + e + 4);
+        auto piece = [&](const Raw8<bf16>(&w)[UR], int e) {
+            const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(s_c + e), b = *reinterpret_cast<const ulonglong2*>(s_c + e + 4);
 #pragma unroll
             for (int u = 0; u < UR; ++u) {
                 const Pairs8 x = w[u].pairs();
-                d[u] += sum2(fma2(x.p[0], c0.x, fma2(x.p[1], c0.y, fma2(x.p[2], c1.x, mul2(x.p[3], c1.y)))));
+                d[u] += sum2(fma2(x.p[0], a.x, fma2(x.p[1], a.y, fma2(x.p[2], b.x, mul2(x.p[3], b.y)))));
             }
+        };
+        int e = lane * 8;
+        if (r0 == rw) {
+#pragma unroll
+            for (int i = 0; i < PRE; ++i, e += 256)
+                if (e < S.rp) piece(pre[i], e);
+        }
+#pragma unroll 1
+        for (; e < S.rp; e += 256) {
+            Raw8<bf16> w[UR];
+#pragma unroll
+            for (int u = 0; u < UR; ++u) w[u].load(uv + (size_t)min(r0 + u, v1 - 1) * S.rp + e);
+            piece(w, e);
         }
         __syncwarp();
         warp_sums<UR>(d);
         const float v = lane == 0 ? d[0] : lane == 1 ? d[1] : lane == 2 ? d[2] : d[3];
-        if (lane < UR && r0 + lane < v1) put(out + r0 + lane, v * sigmoid(__ldcg(gate + r0 + lane)));
+        if (lane < UR && r0 + lane < v1) put(out + r0 + lane, v * sigmoid(r0 == rw ? g0 : __ldcg(gate + r0 + lane)));
     }
 }
 

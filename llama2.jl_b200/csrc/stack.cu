@@ -461,7 +461,7 @@ static cudaError_t launch_latent_attention(LatentAttnParams a, int rows, bool ch
         default: e = launch_kernel(latent_scan_kernel<CT, 4>, grid, block, smem, st, true, a); break;
     }
     if (e != cudaSuccess) return e;
-    return launch_kernel(latent_output_kernel<OT>, dim3(s.heads * a.vsplit, rows), dim3(LA_CONSUMERS), 0, st, true, a);
+    return launch_kernel(latent_output_kernel<OT>, dim3(s.heads * a.vsplit, rows), dim3(LA_CONSUMERS), 0, st, true, a, a.vsplit);
 }
 
 // ---- one position ------------------------------------------------------------------------------
