@@ -5,9 +5,11 @@
 // alike, and nothing per head is cached.  Three kernels, chained with programmatic dependent launch in a decode step:
 //   latent_query_kernel   q' and the rotated query part of every (row, head); in a decode step one more block normalises and
 //                         rotates the new position's latent and key and writes them to the cache;
-//   latent_scan_kernel    a block takes 8 heads (one per warp) and a range of positions, whose cache rows (contiguous) a producer warp
-//                         brings into shared memory with bulk asynchronous copies; running softmax in the exp2 domain, f32;
-//                         one partial result (maximum, sum, unnormalised latent) per head and range;
+//   latent_scan_mma_kernel (bf16 cache)  a block takes 16 heads and a range of positions, whose cache rows a producer warp brings into
+//                         shared memory with bulk asynchronous copies; scores and weighted sums on the tensor cores with q' and
+//                         the weights as two bf16 terms (high and low part: 16 significant bits), running softmax in the
+//                         exp2 domain in f32; one partial result (maximum, sum, unnormalised latent) per head and range;
+//   latent_scan_kernel    (f32 cache)  the same on the CUDA cores, 8 heads per block, one per warp;
 //   latent_output_kernel  merges the ranges and the sink, applies W_uv and the gate.
 // (One kernel with clusters that exchange q' and the partial results through distributed shared memory was about twice as slow: its
 // code is several times as long and runs once per launch, so that fetching instructions bounds it.)
@@ -20,7 +22,7 @@
 namespace l2b {
 
 constexpr int LA_WARPS = 8, LA_CONSUMERS = LA_WARPS * 32, LA_SCAN_THREADS = LA_CONSUMERS + 32;
-constexpr int LA_STAGE_ROWS = 16, LA_MAX_STAGES = 4, LA_MAX_SPLIT = 64, LA_MIN_RANGE = 16;
+constexpr int LA_STAGE_ROWS = 16, LA_MAX_STAGES = 4, LA_MAX_SPLIT = 64, LA_MIN_RANGE = 32;
 
 struct LatentShape {
     int heads, dim, rot, rdims, vdim, rank;  // rdims: rotated dimensions of the rot part
@@ -156,6 +158,187 @@ __global__ void __launch_bounds__(LA_CONSUMERS) latent_query_kernel(const __grid
     }
 }
 
+// ---- scan on the tensor cores -----------------------------------------------------------------------------------
+constexpr int LM_HEADS = 16;  // heads per block = M of mma.m16n8k16
+
+// Bytes between cache rows in shared memory: 16 mod 128, so that eight rows of a fragment load fall in different banks; at least
+// 16 bytes of zeros follow the row (the last K = 16 step may reach 8 values beyond it).
+__host__ __device__ inline int lm_pitch(int row) { return (row * 2 + 127) / 128 * 128 + 16; }
+__host__ __device__ inline int lm_stage_bytes(int row) { return LA_STAGE_ROWS * lm_pitch(row); }
+
+__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ldmatrix4_trans(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+// x = hi + lo with both bf16: two values -> two packed words
+__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+    const float2 f = __bfloat1622float2(h);
+    const __nv_bfloat162 l = __floats2bfloat162_rn(x - f.x, y - f.y);
+    hi = *reinterpret_cast<const uint32_t*>(&h);
+    lo = *reinterpret_cast<const uint32_t*>(&l);
+}
+
+// Grid (nsplit * groups of 16 heads, rows).  N: K = 16 steps of a cache row, and pairs of 8-column tiles of the latent, per warp at most.
+template <int N>
+__global__ void __launch_bounds__(LA_SCAN_THREADS) latent_scan_mma_kernel(const __grid_constant__ LatentAttnParams p) {
+    extern __shared__ __align__(128) uint8_t la_ring[];  // [stages][LA_STAGE_ROWS][pitch]
+    __shared__ __align__(8) uint64_t s_full[LA_MAX_STAGES], s_empty[LA_MAX_STAGES];
+    __shared__ float s_s[LA_WARPS][LM_HEADS][LA_STAGE_ROWS + 1];             // the warps' shares of the scores
+    __shared__ __align__(16) uint32_t s_hi[LM_HEADS][12], s_lo[LM_HEADS][12];  // weights of a stage: 16 bf16 per head (rows padded)
+    __shared__ float s_corr[LM_HEADS];
+    constexpr int KS = N, NT = N;
+    const LatentShape& S = p.s;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, row = (int)blockIdx.y;
+    const int split = (int)blockIdx.x % p.nsplit, h0 = (int)blockIdx.x / p.nsplit * LM_HEADS;
+    const int pitch = lm_pitch(S.row), stage_bytes = lm_stage_bytes(S.row);
+    pdl_launch_dependents();
+    if (tid == 0) {
+        for (int i = 0; i < p.stages; ++i) {
+            mbar_init(s_full + i, 1);
+            mbar_init(s_empty + i, LA_WARPS);
+        }
+        fence_barrier_init();
+        fence_proxy_async();
+    }
+    for (int i = tid; i < p.stages * LA_STAGE_ROWS; i += LA_SCAN_THREADS)  // zeros behind every row
+        for (int k = S.row * 2; k < pitch; k += 16) *reinterpret_cast<uint4*>(la_ring + (size_t)i * pitch + k) = make_uint4(0u, 0u, 0u, 0u);
+    __syncthreads();
+    const int npos = latent_position(p, row) + 1, range = latent_range(npos, p.nsplit);
+    const int t0 = min(npos, split * range), t1 = min(npos, t0 + range);
+    const int nstage = (t1 - t0 + LA_STAGE_ROWS - 1) / LA_STAGE_ROWS;
+
+    if (warp == LA_WARPS) {
+        const bf16* const cache = static_cast<const bf16*>(p.cache) + (size_t)row * p.cache_stride;
+        bool waited = false;
+        for (int j = 0; j < nstage; ++j) {
+            const int s = j % p.stages, use = j / p.stages, t = t0 + j * LA_STAGE_ROWS, te = min(t1, t + LA_STAGE_ROWS);
+            if (!waited && (!p.fused || te == npos)) {  // rows of earlier tokens need not be waited for
+                pdl_wait();
+                waited = true;
+            }
+            if (!__all_sync(0xffffffffu, use == 0 || mbar_wait_bounded(s_empty + s, (uint32_t)((use - 1) & 1)))) {
+                if (lane == 0) atomicExch(p.status, DEV_ERR_TMA_TIMEOUT);
+                for (int i = 0; i < 2000; ++i) __nanosleep(1000);  // copies in flight land within microseconds
+                break;
+            }
+            if (lane == 0) mbar_arrive_expect_tx(s_full + s, (uint32_t)((te - t) * S.row * 2));
+            __syncwarp();
+            if (lane < te - t) bulk_g2s_plain(la_ring + (size_t)s * stage_bytes + lane * pitch, cache + (size_t)(t + lane) * S.row, (uint32_t)(S.row * 2), s_full + s);
+        }
+        return;
+    }
+    pdl_wait();
+    const int g = lane >> 2, t4 = lane & 3;
+    // this warp's K steps (warp, warp + 8, ...) of q', as A fragments in two terms
+    uint32_t qhi[KS][4], qlo[KS][4];
+#pragma unroll
+    for (int i = 0; i < KS; ++i)
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const int h = h0 + g + 8 * (k & 1), e = (warp + LA_WARPS * i) * 16 + 8 * (k >> 1) + 2 * t4;
+            float2 v = make_float2(0.f, 0.f);
+            if (h < S.heads && e < S.row) v = __ldcg(reinterpret_cast<const float2*>(p.qp + ((size_t)row * S.heads + h) * S.row + e));
+            split2(v.x, v.y, qhi[i][k], qlo[i][k]);
+        }
+    float acc[NT][2][4];
+#pragma unroll
+    for (int i = 0; i < NT; ++i)
+#pragma unroll
+        for (int k = 0; k < 8; ++k) acc[i][k >> 2][k & 3] = 0.f;
+    const int sh = tid >> 4, sp = tid & 15;  // softmax: this thread's head and position of a stage
+    float m = -INFINITY, l = 0.f;
+    bool dead = false;
+#pragma unroll 1
+    for (int j = 0; j < nstage; ++j) {
+        const int s = j % p.stages, n = min(LA_STAGE_ROWS, t1 - t0 - j * LA_STAGE_ROWS);
+        if (!dead && !__all_sync(0xffffffffu, mbar_wait_bounded(s_full + s, (uint32_t)((j / p.stages) & 1)))) dead = true;
+        __syncwarp();
+        const uint8_t* const st = la_ring + (size_t)s * stage_bytes;
+        {
+            float d[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+#pragma unroll
+            for (int i = 0; i < KS; ++i) {
+                const int k0 = (warp + LA_WARPS * i) * 16;
+                if (k0 < S.row)
+#pragma unroll
+                    for (int t = 0; t < 2; ++t) {  // positions 8t .. 8t+7 of the stage
+                        const uint8_t* at = st + (8 * t + g) * pitch + (k0 + 2 * t4) * 2;
+                        const uint32_t b0 = *reinterpret_cast<const uint32_t*>(at), b1 = *reinterpret_cast<const uint32_t*>(at + 16);
+                        mma_bf16(d[t], qhi[i], b0, b1);
+                        mma_bf16(d[t], qlo[i], b0, b1);
+                    }
+            }
+#pragma unroll
+            for (int t = 0; t < 2; ++t)
+#pragma unroll
+                for (int k = 0; k < 4; ++k) s_s[warp][g + 8 * (k >> 1)][8 * t + 2 * t4 + (k & 1)] = d[t][k];
+        }
+        // rows that were not copied (a last, partial stage) weigh nothing, but must hold numbers
+        for (int i = n * (pitch / 16) + tid; i < LA_STAGE_ROWS * (pitch / 16); i += LA_CONSUMERS)
+            *reinterpret_cast<uint4*>(la_ring + (size_t)s * stage_bytes + (size_t)i * 16) = make_uint4(0u, 0u, 0u, 0u);
+        partial_sync(LA_CONSUMERS);
+        {
+            float v = 0.f;
+#pragma unroll
+            for (int w = 0; w < LA_WARPS; ++w) v += s_s[w][sh][sp];
+            if (sp >= n) v = -INFINITY;  // (positions beyond the range: stale rows)
+            float mx = v;
+#pragma unroll
+            for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+            mx = fmaxf(m, mx);
+            const float corr = exp2f(m - mx), w = exp2f(v - mx);
+            float sum = w;
+#pragma unroll
+            for (int o = 8; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+            l = fmaf(l, corr, sum);
+            m = mx;
+            const float w1 = __shfl_down_sync(0xffffffffu, w, 1);
+            if ((sp & 1) == 0) split2(w, w1, s_hi[sh][sp >> 1], s_lo[sh][sp >> 1]);
+            if (sp == 0) s_corr[sh] = corr;
+        }
+        partial_sync(LA_CONSUMERS);
+        {
+            const float ca = s_corr[g], cb = s_corr[g + 8];
+            const uint32_t ahi[4] = {s_hi[g][t4], s_hi[g + 8][t4], s_hi[g][t4 + 4], s_hi[g + 8][t4 + 4]};
+            const uint32_t alo[4] = {s_lo[g][t4], s_lo[g + 8][t4], s_lo[g][t4 + 4], s_lo[g + 8][t4 + 4]};
+#pragma unroll
+            for (int i = 0; i < NT; ++i) {
+                const int c0 = (warp + LA_WARPS * i) * 16;  // columns c0 .. c0+15: two tiles
+                if (c0 >= S.rp) continue;                   // (uniform over the warp)
+#pragma unroll
+                for (int k = 0; k < 8; ++k) acc[i][k >> 2][k & 3] *= (k & 2) ? cb : ca;
+                uint32_t b[4];
+                // lanes 0-7: positions 0-7, columns c0..; 8-15: positions 8-15; 16-31: the same for columns c0+8..
+                ldmatrix4_trans(b, smem_u32(st + (lane & 15) * pitch + (c0 + 8 * (lane >> 4)) * 2));
+                mma_bf16(acc[i][0], ahi, b[0], b[1]);
+                mma_bf16(acc[i][0], alo, b[0], b[1]);
+                mma_bf16(acc[i][1], ahi, b[2], b[3]);
+                mma_bf16(acc[i][1], alo, b[2], b[3]);
+            }
+        }
+        __syncwarp();
+        if (lane == 0) mbar_arrive(s_empty + s);
+    }
+    if (dead && lane == 0) atomicExch(p.status, DEV_ERR_TMA_TIMEOUT);
+    if (t0 >= t1) return;  // (a range without positions is not read by the merge)
+    if (sp == 0 && h0 + sh < S.heads) p.part_ml[((size_t)row * S.heads + h0 + sh) * p.nsplit + split] = make_float2(m, l);
+#pragma unroll
+    for (int i = 0; i < NT; ++i)
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {  // tile k & 1, row half k >> 1
+            const int h = h0 + g + 8 * (k >> 1), c = (warp + LA_WARPS * i) * 16 + 8 * (k & 1) + 2 * t4;
+            if (h < S.heads && c < S.rp)
+                *reinterpret_cast<float2*>(p.part_acc + (((size_t)row * S.heads + h) * p.nsplit + split) * S.rp + c) =
+                    make_float2(acc[i][k & 1][2 * (k >> 1)], acc[i][k & 1][2 * (k >> 1) + 1]);
+        }
+}
+
+// ---- scan on the CUDA cores ---------------------------------------------------------------------------------------
 // Grid (nsplit * groups of 8 heads, rows).  NI: 256-value pieces a cache row is spread over (32 lanes x 8 values each).
 template <typename CT, int NI>
 __global__ void __launch_bounds__(LA_SCAN_THREADS) latent_scan_kernel(const __grid_constant__ LatentAttnParams p) {

@@ -288,9 +288,9 @@ constexpr int ABSORB_ROWS = 64;  // rows per pass of the absorbed form of the at
 constexpr int EXPAND_MIN_ROWS = 48;
 
 // Groups of heads and ranges of positions of the scan kernel: about one block per SM in a decode step, two for several rows.
-static int latent_groups(const LatentShape& s) { return (s.heads + LA_WARPS - 1) / LA_WARPS; }
-static int latent_splits(const LatentShape& s, int rows, const DeviceInfo& di) {
-    return std::max(1, std::min(LA_MAX_SPLIT, (rows == 1 ? 1 : 2) * di.sms / (latent_groups(s) * rows)));
+static int latent_groups(const LatentShape& s, bool f32) { return f32 ? (s.heads + LA_WARPS - 1) / LA_WARPS : (s.heads + LM_HEADS - 1) / LM_HEADS; }
+static int latent_splits(const LatentShape& s, bool f32, int rows, const DeviceInfo& di) {
+    return std::max(1, std::min(LA_MAX_SPLIT, (rows == 1 ? 1 : 2) * di.sms / (latent_groups(s, f32) * rows)));
 }
 
 static int prefill_kstages(const LatentShape& s, const DeviceInfo& di) {
@@ -318,11 +318,10 @@ static int32_t set_stack_kernel_attrs() {
         set((const void*)bf16_gemm_kernel<32, 1>); set((const void*)bf16_gemm_kernel<32, 2>);
         set((const void*)bf16_gemm_kernel<64, 1>); set((const void*)bf16_gemm_kernel<64, 2>);
         set((const void*)bf16_gemm_kernel<128, 1>); set((const void*)bf16_gemm_kernel<128, 2>);
-#define L2B_SET_LA(NI)                                      \
-    set((const void*)latent_scan_kernel<bf16, NI>);         \
-    set((const void*)latent_scan_kernel<float, NI>);
-        L2B_SET_LA(1) L2B_SET_LA(2) L2B_SET_LA(3) L2B_SET_LA(4)
-#undef L2B_SET_LA
+        set((const void*)latent_scan_kernel<float, 1>); set((const void*)latent_scan_kernel<float, 2>);
+        set((const void*)latent_scan_kernel<float, 3>); set((const void*)latent_scan_kernel<float, 4>);
+        set((const void*)latent_scan_mma_kernel<1>); set((const void*)latent_scan_mma_kernel<2>); set((const void*)latent_scan_mma_kernel<3>);
+        set((const void*)latent_scan_mma_kernel<5>); set((const void*)latent_scan_mma_kernel<8>);
     });
     if (g_stack_attr_err != cudaSuccess) return fail(L2B_ERR_CUDA, std::string("cudaFuncSetAttribute: ") + cudaGetErrorString(g_stack_attr_err));
     return L2B_OK;
@@ -387,7 +386,7 @@ int32_t stack_session_create(const StackModel* m, const StackSessionInfo& info, 
     size_t qp = 0, pml = 0, pacc = 0;
     for (const StackLayerW& w : m->layers)
         for (int rows = 1; rows <= std::max(1, std::min(ABSORB_ROWS, info.max_rows)); ++rows) {
-            const size_t pairs = (size_t)w.shape.heads * rows, slots = pairs * latent_splits(w.shape, rows, di);
+            const size_t pairs = (size_t)w.shape.heads * rows, slots = pairs * latent_splits(w.shape, m->f32, rows, di);
             qp = std::max(qp, pairs * w.shape.row);
             pml = std::max(pml, slots);
             pacc = std::max(pacc, slots * w.shape.rp);
@@ -447,18 +446,21 @@ static cudaError_t launch_latent_attention(LatentAttnParams a, int rows, bool ch
     const long pairs = (long)s.heads * rows;
     for (a.csplit = 1; a.csplit < 8 && pairs * a.csplit < di.sms;) a.csplit *= 2;
     for (a.vsplit = 1; a.vsplit < 4 && pairs * a.vsplit < di.sms;) a.vsplit *= 2;
-    a.nsplit = latent_splits(s, rows, di);
-    const int stage = LA_STAGE_ROWS * s.row * (int)sizeof(CT);
-    a.stages = std::max(1, std::min(LA_MAX_STAGES, (di.max_smem_optin - 2048) / stage));
+    constexpr bool f32 = sizeof(CT) == 4;
+    a.nsplit = latent_splits(s, f32, rows, di);
+    const int stage = f32 ? LA_STAGE_ROWS * s.row * 4 : lm_stage_bytes(s.row);
+    a.stages = std::max(1, std::min(LA_MAX_STAGES, (di.max_smem_optin - 16 * 1024) / stage));
     cudaError_t e = launch_kernel(latent_query_kernel<CT>, dim3(s.heads * a.csplit + (a.fused ? 1 : 0), rows), dim3(LA_CONSUMERS), 0, st, chained, a);
     if (e != cudaSuccess) return e;
-    const dim3 grid(latent_groups(s) * a.nsplit, rows), block(LA_SCAN_THREADS);
+    const dim3 grid(latent_groups(s, f32) * a.nsplit, rows), block(LA_SCAN_THREADS);
     const size_t smem = (size_t)a.stages * stage;
-    switch ((s.row + 255) / 256) {
-        case 1: e = launch_kernel(latent_scan_kernel<CT, 1>, grid, block, smem, st, true, a); break;
-        case 2: e = launch_kernel(latent_scan_kernel<CT, 2>, grid, block, smem, st, true, a); break;
-        case 3: e = launch_kernel(latent_scan_kernel<CT, 3>, grid, block, smem, st, true, a); break;
-        default: e = launch_kernel(latent_scan_kernel<CT, 4>, grid, block, smem, st, true, a); break;
+    auto go = [&](auto k) { return launch_kernel(k, grid, block, smem, st, true, a); };
+    if (f32) {
+        const int pieces = (s.row + 255) / 256;
+        e = pieces == 1 ? go(latent_scan_kernel<float, 1>) : pieces == 2 ? go(latent_scan_kernel<float, 2>) : pieces == 3 ? go(latent_scan_kernel<float, 3>) : go(latent_scan_kernel<float, 4>);
+    } else {
+        e = s.row <= 128 ? go(latent_scan_mma_kernel<1>) : s.row <= 256 ? go(latent_scan_mma_kernel<2>) : s.row <= 384 ? go(latent_scan_mma_kernel<3>)
+            : s.row <= 640 ? go(latent_scan_mma_kernel<5>) : go(latent_scan_mma_kernel<8>);
     }
     if (e != cudaSuccess) return e;
     return launch_kernel(latent_output_kernel<OT>, dim3(s.heads * a.vsplit, rows), dim3(LA_CONSUMERS), 0, st, true, a, a.vsplit);
