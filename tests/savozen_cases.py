@@ -103,5 +103,6 @@ CASES = {
     # latents that spread over two, three and four pieces of a cache row; head sizes beyond one operand tile
     "rank_300": config([(M(heads=2, dim=72, rot_dim=40, vdim=144, kv_rank=300, scale=0.1), 96)], width=136, vocab=151, side=8),
     "rank_512": config([(M(heads=9, dim=128, rot_dim=64, vdim=128, kv_rank=512, scale=0.08), 200)], width=256, vocab=400),
+    "wide_values": config([(M(heads=2, dim=40, rot_dim=24, vdim=272, kv_rank=120, scale=0.15), None)], width=88, vocab=115),
     "rank_900": config([(M(heads=2, dim=32, rot_dim=96, vdim=200, kv_rank=900, scale=0.1), None)], width=120, vocab=130, side=20),
 }

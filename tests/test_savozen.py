@@ -251,6 +251,26 @@ def test_one_far_key_stands_out(pkg, compute):
 
 @pytest.mark.gpu
 @pytest.mark.parametrize("compute", COMPUTE)
+def test_prompts_of_several_passes(pkg, compute):
+    """A prompt longer than one many-token pass, logits wanted on both sides of the cut, then decode steps whose ranges of positions
+    are longer than the shortest one."""
+    cfg = sc.config([(sc.mixer(heads=2, dim=16, rot_dim=16, vdim=16, kv_rank=24, scale=0.5), 40)], width=40, vocab=64, side=8)
+    n = 2230
+    w, t = sc.weights(cfg, 45), sc.tokens(cfg, n, 46)
+    want = expected(cfg, w, t)
+    model = build(pkg, cfg, w, n, compute)
+    state = pkg.RunState(model)
+    places = [0, 1, 500, 2046, 2047, 2048, 2049, 2199]
+    check(pkg.extend(state, t[:2200], 0, places), want, compute, places)
+    got = [pkg.extend(state, t[p:p + 1], p, [0]) for p in range(2200, n)]
+    check(np.concatenate(got), want, compute, slice(2200, n))
+    assert pkg.prefill(state, t[:2150]) == int(np.argmax(state.logits))
+    check(state.logits[None], want, compute, slice(2149, 2150))
+    model.close()
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("compute", COMPUTE)
 def test_sessions_are_used_again(pkg, compute):
     """A session's cache holds nothing of the sequence before, with or without a reset; two sessions do not see one another."""
     from llama2_jl_b200 import _lib as L
