@@ -79,28 +79,13 @@ __device__ __forceinline__ void warp_sums(float (&v)[N]) {
     for (int i = 0; i < N; ++i) v[i] = N > 1 ? __shfl_sync(0xffffffffu, t, i * (32 / N)) : t;
 }
 
-// eight consecutive values (16-byte aligned bf16, 32-byte aligned f32) as f32
-struct Vec8 {
-    float v[8];
-};
-__device__ __forceinline__ Vec8 unpack8(uint4 r) {
-    Vec8 o;
-    const uint32_t w[4] = {r.x, r.y, r.z, r.w};
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-        o.v[2 * i] = __uint_as_float(w[i] << 16);
-        o.v[2 * i + 1] = __uint_as_float(w[i] & 0xFFFF0000u);
-    }
-    return o;
-}
 template <typename T>
-struct Raw8;  // the same eight values as loaded, before conversion
+struct Raw8;  // eight consecutive values (16-byte aligned bf16 or f32) as loaded, before conversion
 template <>
 struct Raw8<bf16> {
     uint4 r;
     __device__ __forceinline__ void zero() { r = make_uint4(0u, 0u, 0u, 0u); }
     __device__ __forceinline__ void load(const bf16* p) { r = __ldcg(reinterpret_cast<const uint4*>(p)); }
-    __device__ __forceinline__ Vec8 get() const { return unpack8(r); }
     __device__ __forceinline__ void read(const void* smem) { r = *static_cast<const uint4*>(smem); }
     __device__ __forceinline__ Pairs8 pairs() const {
         Pairs8 o;
@@ -112,16 +97,6 @@ template <>
 struct Raw8<float> {
     float4 a, b;
     __device__ __forceinline__ void zero() { a = b = make_float4(0.f, 0.f, 0.f, 0.f); }
-    __device__ __forceinline__ void load(const float* p) {
-        a = __ldcg(reinterpret_cast<const float4*>(p));
-        b = __ldcg(reinterpret_cast<const float4*>(p) + 1);
-    }
-    __device__ __forceinline__ Vec8 get() const {
-        Vec8 o;
-        o.v[0] = a.x; o.v[1] = a.y; o.v[2] = a.z; o.v[3] = a.w;
-        o.v[4] = b.x; o.v[5] = b.y; o.v[6] = b.z; o.v[7] = b.w;
-        return o;
-    }
     __device__ __forceinline__ void read(const void* smem) {
         a = static_cast<const float4*>(smem)[0];
         b = static_cast<const float4*>(smem)[1];
@@ -135,8 +110,6 @@ struct Raw8<float> {
 
 __device__ __forceinline__ void put(float* p, float v) { *p = v; }
 __device__ __forceinline__ void put(bf16* p, float v) { *p = __float2bfloat16_rn(v); }
-__device__ __forceinline__ float as_stored(const float*, float v) { return v; }  // the value a store of that type keeps
-__device__ __forceinline__ float as_stored(const bf16*, float v) { return __bfloat162float(__float2bfloat16_rn(v)); }
 
 __device__ __forceinline__ float gelu_tanh(float z) {
     const float t = tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z));  // sqrt(2 / pi)
