@@ -125,12 +125,15 @@ int32_t l2b_gguf_inspect(const char* path, l2b_config* config_out, int32_t* arch
 /* ---- layer-stack models (no counterpart in the reference) -------------------------------------------------
  * Decoders whose config.json lists their layers one by one and names the design under "architecture" (Savozen: latent attention
  * with a sink and an output gate, dynamic-tanh norms, tanh-gelu feed-forward, per-layer token input, a stretch of layers run
- * several times).  Every session, batch and sampling entry point below serves them; tensor parallelism does not.
- *   seq_len       positions a session holds;
- *   compute_type  L2B_TYPE_BF16: bf16 matrix operands and latent cache, everything else f32; L2B_TYPE_F32: f32 throughout.
+ * several times; Perezen: differential attention within chunks and mLSTM layers, learned position vectors, rms norms before and
+ * after every sublayer, silu feed-forward).  Every session, batch and sampling entry point below serves them; tensor parallelism does not.
+ *   seq_len       positions a session holds (at most as many as the design has learned position vectors);
+ *   compute_type  L2B_TYPE_BF16: bf16 matrix operands and caches, everything else f32; L2B_TYPE_F32: f32 throughout.
  * l2b_model_load_dir reads DIR/config.json and DIR/model.safetensors.  l2b_model_create_stack builds an empty model from the
  * text of a config.json; its tensors are then given by their names (bf16; vectors may be f32), and l2b_model_finalize checks
- * that all are there.  config_out (may be NULL) receives dim, vocab_size, n_layers, seq_len. */
+ * that all are there.  config_out (may be NULL) receives dim, vocab_size, n_layers, seq_len.
+ * A model with a recurrent state (mLSTM) takes positions in order: a call of a session, or a sequence of a batch, starts at
+ * position 0 (afresh, whatever was there before) or where the last call ended; anything else is L2B_ERR_STATE. */
 int32_t l2b_model_load_dir(const char* dir, int32_t seq_len, int32_t compute_type, int32_t device, l2b_config* config_out, l2b_model** model);
 int32_t l2b_model_create_stack(const char* config_json, int32_t seq_len, int32_t compute_type, int32_t device, l2b_config* config_out, l2b_model** model);
 int32_t l2b_model_upload_named(l2b_model* model, const char* name, int32_t type, const void* host_data, const int64_t* shape, int32_t ndim);

@@ -482,6 +482,7 @@ struct l2b_model {
 struct l2b_session {
     l2b_model* model = nullptr;
     StackSession* stack = nullptr;  // layer-stack models: caches and activations
+    int state_pos = 0;              // models with a recurrent state: the position it is ready for (-1: none but 0, which starts afresh)
     cudaStream_t stream = nullptr;
     bool own_stream = false;
     DeviceInfo di;
@@ -894,8 +895,10 @@ extern "C" int32_t l2b_model_create_stack(const char* config_json, int32_t seq_l
         l2b_config& c = m->cfg;
         memset(&c, 0, sizeof(c));
         c.dim = check.width; c.vocab_size = check.vocab; c.n_layers = (int32_t)check.layers.size(); c.seq_len = seq_len;
-        c.hidden_dim = check.layers[0].ff; c.n_heads = c.n_kv_heads = check.layers[0].mix.heads;
-        c.rope_freq_base = (float)check.layers[0].mix.rot.base;
+        if (check.max_positions) c.seq_len = std::min(seq_len, check.max_positions);  // there are no vectors for positions beyond
+        const MixerConfig& mix = check.layers[0].mix;
+        c.hidden_dim = check.layers[0].ff; c.n_heads = mix.heads; c.n_kv_heads = mix.kv_heads ? mix.kv_heads : mix.heads;
+        c.rope_freq_base = (float)mix.rot.base;
         c.device = device; c.tp_size = 1;
         return L2B_OK;
     };
@@ -1717,6 +1720,19 @@ static int32_t check_status_word(l2b_session* s) {
     return L2B_OK;
 }
 
+// Models with a recurrent state go from position to position: a call starts at 0 or where the state stands.  A call marks the state
+// unusable (-1) before it changes it, until it has succeeded (state_at).
+static int32_t check_state(const l2b_model* m, int state_pos, int pos0) {
+    if (!m->stack || !stack_model_config(m->stack).recurrent()) return L2B_OK;
+    if (pos0 != 0 && pos0 != state_pos)
+        return fail(L2B_ERR_STATE, "the recurrent state does not stand at position " + std::to_string(pos0) + ": start at position 0, or go on where the last call ended");
+    return L2B_OK;
+}
+static int32_t state_at(int32_t status, int& state_pos, int pos) {
+    if (status == L2B_OK) state_pos = pos;
+    return status;
+}
+
 // One graph launch with the control block set from the host.
 static int32_t run_one(l2b_session* s, int token, int pos, float temperature, double uniform) {
     const l2b_config& c = s->model->cfg;
@@ -1724,6 +1740,8 @@ static int32_t run_one(l2b_session* s, int token, int pos, float temperature, do
     if (pos < 0 || pos >= c.seq_len) return fail(L2B_ERR_BAD_ARG, "position out of range (seq_len)");
     if (temperature < 0.f) return fail(L2B_ERR_BAD_ARG, "temperature must be >= 0");
     if (!s->graph) return fail(L2B_ERR_STATE, "tensor-parallel session: call l2b_session_tp_connect first");
+    L2B_TRY(check_state(s->model, s->state_pos, pos));
+    s->state_pos = -1;
     CU(cudaSetDevice(s->model->device));
     Control& h = *s->h_ctl;
     memset(&h, 0, sizeof(h));
@@ -1740,7 +1758,7 @@ static int32_t run_one(l2b_session* s, int token, int pos, float temperature, do
     CU(cudaEventRecord(s->ev1, s->stream));
     CU(cudaStreamSynchronize(s->stream));
     CU(cudaEventElapsedTime(&s->last_ms, s->ev0, s->ev1));
-    return check_status_word(s);
+    return state_at(check_status_word(s), s->state_pos, pos + 1);
 }
 
 // ---- many-token prompt pass ---------------------------------------------------------------------------------
@@ -1984,6 +2002,8 @@ extern "C" int32_t l2b_prefill(l2b_session* s, const int32_t* tokens, int32_t n,
     for (int i = 0; i < n; ++i)
         if (tokens[i] < 0 || tokens[i] >= c.vocab_size) return fail(L2B_ERR_BAD_ARG, "prompt token id out of range");
     if (!s->graph) return fail(L2B_ERR_STATE, "tensor-parallel session: call l2b_session_tp_connect first");
+    L2B_TRY(check_state(s->model, s->state_pos, pos0));
+    s->state_pos = -1;
     CU(cudaSetDevice(s->model->device));
     Control& h = *s->h_ctl;
     memset(&h, 0, sizeof(h));
@@ -2004,7 +2024,7 @@ extern "C" int32_t l2b_prefill(l2b_session* s, const int32_t* tokens, int32_t n,
     CU(cudaStreamSynchronize(s->stream));
     CU(cudaEventElapsedTime(&s->last_ms, s->ev0, s->ev1));
     if (next) *next = s->h_small[0];
-    return check_status_word(s);
+    return state_at(check_status_word(s), s->state_pos, end);
 }
 
 // Feed a portion of n tokens at positions pos0 .. and return the logits at n_want places among them (ascending).  Layer-stack
@@ -2030,6 +2050,8 @@ extern "C" int32_t l2b_session_extend(l2b_session* s, const int32_t* tokens, int
         }
         return L2B_OK;
     }
+    L2B_TRY(check_state(s->model, s->state_pos, pos0));
+    s->state_pos = -1;
     CU(cudaSetDevice(s->model->device));
     constexpr int WANT_ROWS = 128;  // rows per classifier pass
     const int max_rows = stack_session_max_rows(s->stack);
@@ -2061,7 +2083,7 @@ extern "C" int32_t l2b_session_extend(l2b_session* s, const int32_t* tokens, int
     CU(cudaEventRecord(s->ev1, s->stream));
     CU(cudaStreamSynchronize(s->stream));
     CU(cudaEventElapsedTime(&s->last_ms, s->ev0, s->ev1));
-    return check_status_word(s);
+    return state_at(check_status_word(s), s->state_pos, pos0 + n);
 }
 
 extern "C" int32_t l2b_session_prefill_gemm(l2b_session* s, int32_t* min_tokens) {
@@ -2087,6 +2109,8 @@ extern "C" int32_t l2b_generate(l2b_session* s, const int32_t* prompt, int32_t n
     for (int i = 0; i < n_prompt; ++i)
         if (prompt[i] < 0 || prompt[i] >= c.vocab_size) return fail(L2B_ERR_BAD_ARG, "prompt token id out of range");
     if (!s->graph) return fail(L2B_ERR_STATE, "tensor-parallel session: call l2b_session_tp_connect first");
+    L2B_TRY(check_state(s->model, s->state_pos, 0));
+    s->state_pos = -1;
     CU(cudaSetDevice(s->model->device));
     Control& h = *s->h_ctl;
     memset(&h, 0, sizeof(h));
@@ -2122,7 +2146,7 @@ extern "C" int32_t l2b_generate(l2b_session* s, const int32_t* prompt, int32_t n
     CU(cudaEventElapsedTime(&s->last_prompt_ms, s->ev0, s->ev_mid));
     CU(cudaEventElapsedTime(&s->last_decode_ms, s->ev_mid, s->ev1));
     if (device_ms) *device_ms = s->last_ms;
-    return check_status_word(s);
+    return state_at(check_status_word(s), s->state_pos, n_positions);
 }
 
 extern "C" int32_t l2b_session_logits(l2b_session* s, float* host_logits) {
@@ -2181,6 +2205,7 @@ extern "C" int32_t l2b_session_kernels_per_token(l2b_session* s, int32_t* n) {
 struct l2b_batch {
     l2b_model* model = nullptr;
     StackSession* stack = nullptr;       // layer-stack models: caches of all sequences and activations
+    std::vector<int> state_pos;          // as in l2b_session, per sequence
     int n_seq = 0;
     cudaStream_t stream = nullptr;
     DeviceInfo di;
@@ -2219,6 +2244,7 @@ extern "C" int32_t l2b_batch_create(l2b_model* m, int32_t n_seq, l2b_batch** out
     l2b_batch* b = new l2b_batch();
     b->model = m;
     b->n_seq = n_seq;
+    b->state_pos.assign(n_seq, 0);
     auto run = [&]() -> int32_t {
         L2B_TRY(query_device(b->di));
         CU(cudaStreamCreateWithFlags(&b->stream, cudaStreamNonBlocking));
@@ -2326,6 +2352,8 @@ extern "C" int32_t l2b_batch_decode_next(l2b_batch* b, const int32_t* tokens, co
         if (tokens[i] < 0 || tokens[i] >= c.vocab_size) return fail(L2B_ERR_BAD_ARG, "token id out of range");
         if (positions[i] < 0 || positions[i] >= c.seq_len) return fail(L2B_ERR_BAD_ARG, "position out of range (seq_len)");
     }
+    for (int i = 0; i < n; ++i) L2B_TRY(check_state(m, b->state_pos[i], positions[i]));
+    b->state_pos.assign(n, -1);
     CU(cudaSetDevice(m->device));
     cudaStream_t st = b->stream;
     memcpy(b->h_io, tokens, (size_t)n * 4);
@@ -2350,6 +2378,7 @@ extern "C" int32_t l2b_batch_decode_next(l2b_batch* b, const int32_t* tokens, co
         if (dev_status == DEV_ERR_BAD_INDEX) return fail(L2B_ERR_CUDA, "no valid token could be chosen (the logits are not finite); token 0 was substituted");
         return fail(dev_status == DEV_ERR_TMA_TIMEOUT ? L2B_ERR_TIMEOUT : L2B_ERR_CUDA, "kernel reported device status " + std::to_string(dev_status));
     }
+    for (int i = 0; i < n; ++i) b->state_pos[i] = positions[i] + 1;
     memcpy(next_tokens, b->h_io + 2 * n, (size_t)n * 4);
     return L2B_OK;
 }

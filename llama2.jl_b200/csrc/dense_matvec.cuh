@@ -6,13 +6,14 @@
 //       (one copy of adjacent whole rows, or one per row when rows are longer than a stage).  Weights are constants, so
 //       the ring is filled BEFORE the wait on the previous kernel (programmatic dependent launch);
 //   prologue : the input vector goes to shared memory as f32, after the pending changes of the residual stream (the normalised
-//       per-layer token input, the step vector of a loop pass) and the norm; block 0 writes the changed residual stream back
-//       to its other buffer, because the other blocks still read this one;
+//       per-layer token input or sublayer result, the step vector of a loop pass) and the norm; block 0 writes the changed
+//       residual stream back to its other buffer, because the other blocks still read this one.  The scalar 1 / rms(x) of an rms
+//       norm is applied to the results, so that its reduction needs no barrier of its own;
 //   weights  : two groups of four consumer warps take alternate stages (a stage's chain of waits, loads and lane reductions is long
 //       beside the time its bytes take); a warp works on up to two units (4 rows x 1 chunk) of a stage and adds over the
 //       stages of its rows in registers; eight row sums are then reduced over the lanes together;
-//   epilogue : the chunk sums of a row are added in a fixed order by one thread: store | residual add | gelu(gate) * up (rows
-//       2u and 2u+1 of an interleaved matrix) | gelu * token embedding | logits with the block's first maximum.
+//   epilogue : the chunk sums of a row are added in a fixed order by one thread: store | residual add | gelu(gate) * up or silu(gate) *
+//       up (rows 2u and 2u+1 of an interleaved matrix) | gelu * token embedding | logits with the block's first maximum.
 // Every mbarrier wait is bounded, as everywhere in the library.
 #pragma once
 #include <algorithm>
@@ -57,7 +58,7 @@ inline int dmv_choose_stages(const DmvParams& p, size_t max_smem) {
 __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __grid_constant__ DmvParams p) {
     extern __shared__ __align__(128) uint8_t dmv_smem[];
     __shared__ __align__(8) uint64_t s_full[DMV_MAX_STAGES], s_empty[DMV_MAX_STAGES];
-    __shared__ float s_red[DMV_WARPS];
+    __shared__ float s_red[DMV_WARPS], s_ss[DMV_WARPS];
     __shared__ int s_idx[DMV_WARPS];
     float* const xf = reinterpret_cast<float*>(dmv_smem + p.stages * DMV_STAGE);
     float* const part = xf + p.nchunk * 256;
@@ -139,6 +140,7 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
             }
             scale = 1.f / sqrtf(block_sum_all<DMV_WARPS>(ss, s_red) / (float)k + p.upd.eps);
         }
+        float xs = 0.f;
         for (int i0 = threadIdx.x; i0 < kc; i0 += U * DMV_CONSUMERS) {
             float v[U];
 #pragma unroll
@@ -148,14 +150,19 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
                 const int i = i0 + u * DMV_CONSUMERS, at = lane_major(i);
                 if (i < k) {
                     float t = v[u];
-                    if (p.upd.y) t = fmaf(xf[at] * scale, __ldg(p.upd.side_w + i), t);
+                    if (p.upd.y) t = fmaf(xf[at] * scale, __ldg(p.upd.w + i), t);
                     if (p.upd.step) t += __ldg(p.upd.step + i);
                     if (p.x_out && b == 0) p.x_out[i] = t;
+                    xs = fmaf(t, t, xs);
                     xf[at] = apply_norm(p.norm, t, i);
                 } else if (i < kc) {
                     xf[at] = 0.f;
                 }
             }
+        }
+        if (p.norm.kind == NORM_RMS) {
+            xs = warp_sum(xs);
+            if (lane == 0) s_ss[warp] = xs;  // (read after the last barrier)
         }
     }
     partial_sync(DMV_CONSUMERS);
@@ -219,6 +226,13 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
     }
     __syncthreads();
 
+    float rms_scale = 1.f;
+    if (p.norm.kind == NORM_RMS) {
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < DMV_WARPS; ++i) ss += s_ss[i];
+        rms_scale = 1.f / sqrtf(ss / (float)p.k + p.norm.eps);
+    }
     float best = -INFINITY;
     int best_i = 0x7fffffff;
     for (int u = threadIdx.x; u < nu; u += DMV_CONSUMERS) {
@@ -227,7 +241,10 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
         for (int s = 0; s < p.cs; ++s) v += pr[s];
         if (p.unit == 2)
             for (int s = 0; s < p.cs; ++s) v2 += pr[p.cs + s];
+        v *= rms_scale;
+        v2 *= rms_scale;
         dense_epilogue<float>(p.epi, 0, u0 + u, v, v2);
+        if (p.epi.kind == DE_LOGITS) v = scaled_biased(p.epi, u0 + u, v);
         if (v > best) {
             best = v;
             best_i = u0 + u;

@@ -116,6 +116,8 @@ __device__ __forceinline__ float gelu_tanh(float z) {
     return 0.5f * z * (1.f + t);
 }
 __device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float silu(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float dynamic_tanh(float x, float alpha, float w, float b) { return fmaf(tanhf(alpha * x), w, b); }
 
 // element d of a vector whose first rdims elements are interleaved rotary pairs; get(i) reads element i, cs = this position's row
@@ -134,10 +136,13 @@ enum : int {
     DE_SIDE = 3,      // act[t][f] = gelu_tanh(v) * e, e = element e_off + f of the token's row of an embedding table
     DE_LOGITS = 4,    // as DE_STORE, and the block's first maximum
     DE_STORE_ACT = 5, // act[t][f]
-    DE_STORE_T = 6    // act[f][t] (transposed)
+    DE_STORE_T = 6,   // act[f][t] (transposed)
+    DE_SWIGLU = 7     // act[t][f] = silu(gate) * up (two weight rows per result)
 };
 struct DenseEpilogue {
     int kind;
+    float mul;            // DE_STORE, DE_LOGITS: factor of the product, and
+    const float* bias;    // what is added to it per result (null: nothing)
     float* y;
     void* act;
     int ld;               // elements between rows of y / act
@@ -146,6 +151,16 @@ struct DenseEpilogue {
     const int* tokens;    // DE_SIDE: token of result row t
     int vocab;            // DE_SIDE: rows of the table (an id outside it contributes zero)
 };
+inline DenseEpilogue dense_epilogue_of(int kind, float* y, void* act, int ld) {
+    DenseEpilogue e = {};
+    e.kind = kind;
+    e.mul = 1.f;
+    e.y = y;
+    e.act = act;
+    e.ld = ld;
+    return e;
+}
+__device__ __forceinline__ float scaled_biased(const DenseEpilogue& e, int f, float v) { return e.bias ? fmaf(v, e.mul, __ldg(e.bias + f)) : v * e.mul; }
 __device__ __forceinline__ float side_value(const DenseEpilogue& e, int t, int f) {
     const int tok = __ldg(e.tokens + t);
     const bool valid = tok >= 0 && tok < e.vocab;  // (the load does not depend on it: several are in flight together)
@@ -157,31 +172,35 @@ __device__ __forceinline__ void dense_epilogue(const DenseEpilogue& e, int t, in
     const size_t o = (size_t)t * e.ld + f;
     AT* act = static_cast<AT*>(e.act);
     switch (e.kind) {
-        case DE_STORE: case DE_LOGITS: e.y[o] = v; break;
+        case DE_STORE: case DE_LOGITS: e.y[o] = scaled_biased(e, f, v); break;
         case DE_RESIDUAL: e.y[o] += v; break;
         case DE_GEGLU: put(act + o, gelu_tanh(v) * v2); break;
         case DE_SIDE: put(act + o, gelu_tanh(v) * side_value(e, t, f)); break;
         case DE_STORE_ACT: put(act + o, v); break;
         case DE_STORE_T: put(act + (size_t)f * e.ld + t, v); break;
+        case DE_SWIGLU: put(act + o, silu(v) * v2); break;
     }
 }
 
-// Pending changes of the residual stream that the next reader applies: x' = x + y / rms(y) * side_w + step.
+// Pending changes of the residual stream that the next reader applies: x' = x + y / rms(y) * w + step.
 struct ResidualUpdate {
-    const float* y;       // output of the per-layer token input, before its norm (null: none)
-    const float* side_w;  // that norm's weight
+    const float* y;       // result whose norm comes before it is added: a sublayer's, or the per-layer token input's (null: none)
+    const float* w;       // that norm's weight
     float eps;
     const float* step;    // vector added at the beginning of a loop pass (null: none)
 };
 // The norm in front of a dense product.
+enum : int { NORM_NONE = 0, NORM_DYNAMIC_TANH = 1, NORM_RMS = 2 };
 struct NormParams {
-    int kind;             // 0: none; 1: dynamic tanh
-    float alpha;
+    int kind;
+    float alpha;          // dynamic tanh
+    float eps;            // rms
     const float* w;
-    const float* b;
+    const float* b;       // dynamic tanh
 };
+// One value; rms: without the factor 1 / rms(x).
 __device__ __forceinline__ float apply_norm(const NormParams& n, float x, int i) {
-    return n.kind ? dynamic_tanh(x, n.alpha, __ldg(n.w + i), __ldg(n.b + i)) : x;
+    return n.kind == NORM_DYNAMIC_TANH ? dynamic_tanh(x, n.alpha, __ldg(n.w + i), __ldg(n.b + i)) : n.kind == NORM_RMS ? x * __ldg(n.w + i) : x;
 }
 
 // Barrier over the first `threads` threads of the block.

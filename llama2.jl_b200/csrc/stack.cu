@@ -9,8 +9,10 @@
 
 #include "dense_gemm.cuh"
 #include "dense_matvec.cuh"
+#include "head_attention.cuh"
 #include "latent_attention.cuh"
 #include "latent_prefill.cuh"
+#include "mlstm.cuh"
 #include "stack_rows.cuh"
 
 using namespace l2b;
@@ -35,12 +37,24 @@ struct StackNorm {
     float alpha = 1.f;
 };
 struct StackLayerW {
-    StackNorm norm1, norm2;
-    StackMatrix qdg;  // query, down and gate projections, one below the other
-    StackMatrix uk, uv, o, gu, down, side_gate, side_proj;
-    float *dkv_norm = nullptr, *sink = nullptr, *side_norm = nullptr;
-    LatentShape shape;
-    int off_d = 0, off_g = 0;
+    StackNorm norm1, norm2, norm1b, norm2b;
+    StackMatrix in;               // what the mixer projects its input to, one below the other: latent attention q, down, gate;
+    float* in_bias = nullptr;     // differential attention q, k, v, gate; mLSTM q, k, v, gate, input gate, forget gate
+    StackMatrix o, gu, down, side_gate, side_proj;
+    float* side_norm = nullptr;
+    int off_k = 0, off_v = 0, off_g = 0, off_d = 0, off_i = 0, off_f = 0;  // first rows of the parts of `in`
+    CacheScan scan = {};          // attention: its shape
+    // latent attention
+    StackMatrix uk, uv;
+    float *dkv_norm = nullptr, *sink = nullptr;
+    LatentShape latent;
+    // differential attention
+    float *q_norm = nullptr, *k_norm = nullptr;
+    std::vector<float> lq1, lk1, lq2, lk2;
+    HeadShape head;
+    // mLSTM
+    float* out_norm = nullptr;
+    MlstmShape mlstm;
 };
 
 // Where a tensor of the file goes.
@@ -48,8 +62,10 @@ struct TensorSlot {
     std::vector<int64_t> shape;
     StackMatrix* mat = nullptr;    // matrix rows row0, row0 + row_step, ...; heads > 0: rows of a head are head_pad apart
     int row0 = 0, row_step = 1, head_rows = 0, head_pad = 0;
-    float** vec = nullptr;         // f32 vector (any shape, flattened)
+    float** vec = nullptr;         // f32 vector (any shape, flattened), vec_at values into its allocation
+    size_t vec_at = 0;
     float* scalar = nullptr;       // host scalar
+    std::vector<float>* host = nullptr;  // vector that stays on the host
     bool loaded = false;
 };
 
@@ -60,7 +76,7 @@ struct StackModel {
     bool f32 = false;
     std::vector<StackLayerW> layers;
     std::vector<LayerRun> runs;
-    StackMatrix embed, head, side_embed;
+    StackMatrix embed, head, side_embed, positions;
     StackNorm final_norm;
     float* loop_step = nullptr;  // [times][width]
     std::map<std::string, TensorSlot> slots;
@@ -92,34 +108,51 @@ static void add_matrix(StackModel* m, const std::string& name, StackMatrix& w, i
     s.head_pad = head_pad;
     m->slots[name] = s;
 }
-static void add_vector(StackModel* m, const std::string& name, float** v, std::vector<int64_t> shape) {
+static void add_vector(StackModel* m, const std::string& name, float** v, std::vector<int64_t> shape, size_t at = 0) {
     TensorSlot s;
     s.shape = std::move(shape);
     s.vec = v;
+    s.vec_at = at;
     m->slots[name] = s;
+}
+static void add_host_vector(StackModel* m, const std::string& name, std::vector<float>& v, int n) {
+    TensorSlot s;
+    s.shape = {n};
+    s.host = &v;
+    m->slots[name] = s;
+}
+// A table that is read row by row (not padded).
+static int32_t add_table(StackModel* m, const std::string& name, StackMatrix& t, int rows, int width) {
+    t.rows = rows; t.k = t.kp = width;
+    L2B_TRY(alloc_owned(m->owned, (void**)&t.w, (size_t)t.bytes()));
+    add_matrix(m, name, t, rows);
+    return L2B_OK;
 }
 static void add_norm(StackModel* m, const std::string& name, StackNorm& n) {
     add_vector(m, name, &n.w, {m->cfg.width});
     switch (m->cfg.norm) {
-        case NormKind::DynamicTanh:
+        case NormKind::DynamicTanh: {
             add_vector(m, name + ".b", &n.b, {m->cfg.width});
             TensorSlot s;
             s.scalar = &n.alpha;
             m->slots[name + ".alpha"] = s;
             break;
+        }
+        case NormKind::Rms: break;
     }
 }
 static NormParams norm_params(const StackModel* m, const StackNorm& n) {
-    NormParams p = {0, 0.f, nullptr, nullptr};
+    NormParams p = {NORM_NONE, 0.f, 0.f, nullptr, nullptr};
     switch (m->cfg.norm) {
-        case NormKind::DynamicTanh: p = {1, n.alpha, n.w, n.b}; break;
+        case NormKind::DynamicTanh: p = {NORM_DYNAMIC_TANH, n.alpha, 0.f, n.w, n.b}; break;
+        case NormKind::Rms: p = {NORM_RMS, 0.f, m->cfg.eps, n.w, nullptr}; break;
     }
     return p;
 }
 
 static int32_t build_latent_attention(StackModel* m, StackLayerW& w, const MixerConfig& c, const std::string& p) {
     const int width = m->cfg.width;
-    LatentShape& s = w.shape;
+    LatentShape& s = w.latent;
     s.heads = c.heads; s.dim = c.dim; s.rot = c.rot_dim; s.rdims = c.rot.dims; s.vdim = c.vdim; s.rank = c.kv_rank;
     s.rp = up(c.kv_rank, 8);
     s.row = s.rp + up(c.rot_dim, 8);
@@ -127,14 +160,17 @@ static int32_t build_latent_attention(StackModel* m, StackLayerW& w, const Mixer
     s.vp = up(c.vdim, 16);
     s.scale2 = (float)((double)c.scale * 1.4426950408889634);
     s.eps = m->cfg.eps;
-    if (s.row > 1024) return fail(L2B_ERR_UNSUPPORTED_TYPE, "latent attention takes kv_rank + rot_dim up to 1024");
+    if (s.row > CS_MAX_ROW) return fail(L2B_ERR_UNSUPPORTED_TYPE, "latent attention takes kv_rank + rot_dim up to " + std::to_string(CS_MAX_ROW));
+    w.scan.heads = w.scan.per_group = s.heads;
+    w.scan.row = s.row;
+    w.scan.vcols = s.rp;
     const int nq = c.heads * (c.dim + c.rot_dim), nd = c.kv_rank + c.rot_dim, ng = c.heads * c.vdim;
     w.off_d = nq;
     w.off_g = nq + nd;
-    L2B_TRY(make_matrix(m, w.qdg, nq + nd + ng, width));
-    add_matrix(m, p + "q", w.qdg, nq, 0);
-    add_matrix(m, p + "dkv", w.qdg, nd, nq);
-    add_matrix(m, p + "g", w.qdg, ng, nq + nd);
+    L2B_TRY(make_matrix(m, w.in, nq + nd + ng, width));
+    add_matrix(m, p + "q", w.in, nq, 0);
+    add_matrix(m, p + "dkv", w.in, nd, nq);
+    add_matrix(m, p + "g", w.in, ng, nq + nd);
     L2B_TRY(make_matrix(m, w.uk, c.heads * s.dp, c.kv_rank));
     add_matrix(m, p + "uk", w.uk, c.heads * c.dim, 0, 1, c.dim, s.dp);
     L2B_TRY(make_matrix(m, w.uv, c.heads * s.vp, c.kv_rank));
@@ -143,6 +179,83 @@ static int32_t build_latent_attention(StackModel* m, StackLayerW& w, const Mixer
     add_matrix(m, p + "o", w.o, width);
     add_vector(m, p + "dkv.norm", &w.dkv_norm, {c.kv_rank});
     add_vector(m, p + "sink", &w.sink, {c.heads});
+    return L2B_OK;
+}
+
+static int32_t build_differential_attention(StackModel* m, StackLayerW& w, const MixerConfig& c, const std::string& p) {
+    const int width = m->cfg.width;
+    HeadShape& s = w.head;
+    s.heads = c.heads; s.kv_heads = c.kv_heads; s.dim = c.dim; s.vdim = c.vdim; s.rdims = c.rot.dims;
+    s.dp = up(c.dim, 8);
+    s.vp = up(c.vdim, 8);
+    s.row = s.vp + 2 * s.dp;
+    s.scale2 = (float)((double)c.scale * 1.4426950408889634);
+    s.eps = m->cfg.eps;
+    s.lambda = c.diff;  // (completed by stack_model_finalize)
+    s.out_scale = 1.f - c.diff;
+    if (s.row > CS_MAX_ROW) return fail(L2B_ERR_UNSUPPORTED_TYPE, "differential attention takes vdim + 2 dim up to " + std::to_string(CS_MAX_ROW));
+    w.scan.heads = 2 * s.heads;
+    w.scan.per_group = 2 * (s.heads / s.kv_heads);
+    w.scan.row = s.row;
+    w.scan.vcols = s.vp;
+    w.scan.chunk = c.chunk;
+    const bool own = c.kv_from < 0;
+    const int nq = 2 * c.heads * c.dim, nk = own ? 2 * c.kv_heads * c.dim : 0, nv = own ? c.kv_heads * c.vdim : 0, ng = c.heads * c.vdim;
+    w.off_k = nq;
+    w.off_v = nq + nk;
+    w.off_g = nq + nk + nv;
+    L2B_TRY(make_matrix(m, w.in, nq + nk + nv + ng, width));
+    L2B_TRY(alloc_owned(m->owned, (void**)&w.in_bias, (size_t)w.in.rows * 4));
+    add_matrix(m, p + "q", w.in, nq, 0);
+    add_vector(m, p + "q.b", &w.in_bias, {nq}, 0);
+    add_vector(m, p + "q.norm", &w.q_norm, {c.dim});
+    if (own) {
+        add_matrix(m, p + "k", w.in, nk, w.off_k);
+        add_vector(m, p + "k.b", &w.in_bias, {nk}, w.off_k);
+        add_vector(m, p + "k.norm", &w.k_norm, {c.dim});
+        add_matrix(m, p + "v", w.in, nv, w.off_v);
+        add_vector(m, p + "v.b", &w.in_bias, {nv}, w.off_v);
+    }
+    add_matrix(m, p + "g", w.in, ng, w.off_g);
+    L2B_TRY(make_matrix(m, w.o, width, ng));
+    add_matrix(m, p + "o", w.o, width);
+    add_host_vector(m, p + "lq1", w.lq1, c.dim);
+    add_host_vector(m, p + "lk1", w.lk1, c.dim);
+    add_host_vector(m, p + "lq2", w.lq2, c.dim);
+    add_host_vector(m, p + "lk2", w.lk2, c.dim);
+    return L2B_OK;
+}
+
+static int32_t build_mlstm(StackModel* m, StackLayerW& w, const MixerConfig& c, const std::string& p) {
+    const int width = m->cfg.width;
+    MlstmShape& s = w.mlstm;
+    s.heads = c.heads; s.dim = c.dim; s.vdim = c.vdim;
+    s.cap = c.gate_cap;
+    s.qscale = (float)(1.0 / std::sqrt((double)c.dim));
+    s.eps = m->cfg.eps;
+    for (s.cpl = 1; s.cpl < ML_MAX_COLS && 32 * s.cpl * ML_MAX_CLUSTER < c.vdim;) s.cpl *= 2;
+    for (s.cl = 1; 32 * s.cpl * s.cl < c.vdim;) s.cl *= 2;
+    if (s.cl > ML_MAX_CLUSTER || c.dim > ML_MAX_DIM)
+        return fail(L2B_ERR_UNSUPPORTED_TYPE, "mLSTM takes dim up to " + std::to_string(ML_MAX_DIM) + " and vdim up to " + std::to_string(32 * ML_MAX_COLS * ML_MAX_CLUSTER));
+    const int nk = c.heads * c.dim, nv = c.heads * c.vdim;
+    w.off_k = nk;
+    w.off_v = 2 * nk;
+    w.off_g = w.off_v + nv;
+    w.off_i = w.off_g + nv;
+    w.off_f = w.off_i + c.heads;
+    L2B_TRY(make_matrix(m, w.in, w.off_f + c.heads, width));
+    L2B_TRY(alloc_owned(m->owned, (void**)&w.in_bias, (size_t)w.in.rows * 4));
+    add_matrix(m, p + "q", w.in, nk, 0);
+    add_matrix(m, p + "k", w.in, nk, w.off_k);
+    add_matrix(m, p + "v", w.in, nv, w.off_v);
+    add_matrix(m, p + "g", w.in, nv, w.off_g);
+    add_matrix(m, p + "i", w.in, c.heads, w.off_i);
+    add_vector(m, p + "i.b", &w.in_bias, {c.heads}, w.off_i);
+    add_matrix(m, p + "f", w.in, c.heads, w.off_f);
+    add_vector(m, p + "f.b", &w.in_bias, {c.heads}, w.off_f);
+    add_vector(m, p + "norm", &w.out_norm, {nv});
+    L2B_TRY(make_matrix(m, w.o, width, nv));
+    add_matrix(m, p + "o", w.o, width);
     return L2B_OK;
 }
 
@@ -157,28 +270,28 @@ int32_t stack_model_create(const char* json, size_t n, bool f32, StackModel** ou
     m->layers.resize(c.layers.size());
     L2B_TRY(make_matrix(m.get(), m->head, c.vocab, c.width));
     add_matrix(m.get(), "head", m->head, c.vocab);
-    m->embed.rows = c.vocab; m->embed.k = m->embed.kp = c.width;  // read row by row: not padded
-    L2B_TRY(alloc_owned(m->owned, (void**)&m->embed.w, (size_t)m->embed.bytes()));
-    add_matrix(m.get(), "embed", m->embed, c.vocab);
+    L2B_TRY(add_table(m.get(), "embed", m->embed, c.vocab, c.width));
+    if (c.max_positions) L2B_TRY(add_table(m.get(), "pos", m->positions, c.max_positions, c.width));
     add_norm(m.get(), "final.norm", m->final_norm);
     if (c.has_loop()) add_vector(m.get(), "loop.step", &m->loop_step, {c.loop_times, c.width});
-    if (c.side_dim) {
-        m->side_embed.rows = c.vocab; m->side_embed.k = m->side_embed.kp = c.side_dim * (int)c.layers.size();
-        L2B_TRY(alloc_owned(m->owned, (void**)&m->side_embed.w, (size_t)m->side_embed.bytes()));
-        add_matrix(m.get(), "side.embed", m->side_embed, c.vocab);
-    }
+    if (c.side_dim) L2B_TRY(add_table(m.get(), "side.embed", m->side_embed, c.vocab, c.side_dim * (int)c.layers.size()));
     for (size_t i = 0; i < c.layers.size(); ++i) {
         const StackLayerConfig& l = c.layers[i];
         StackLayerW& w = m->layers[i];
         const std::string p = "l" + std::to_string(i) + ".";
         add_norm(m.get(), p + "norm1", w.norm1);
+        if (c.post_norm) add_norm(m.get(), p + "norm1b", w.norm1b);
         switch (l.mix.kind) {
             case MixerKind::LatentAttention: L2B_TRY(build_latent_attention(m.get(), w, l.mix, p + "mix.")); break;
+            case MixerKind::DifferentialAttention: L2B_TRY(build_differential_attention(m.get(), w, l.mix, p + "mix.")); break;
+            case MixerKind::Mlstm: L2B_TRY(build_mlstm(m.get(), w, l.mix, p + "mix.")); break;
         }
         switch (l.mlp) {
             case MlpKind::None: break;
             case MlpKind::GatedGeluTanh:
+            case MlpKind::GatedSilu:
                 add_norm(m.get(), p + "norm2", w.norm2);
+                if (c.post_norm) add_norm(m.get(), p + "norm2b", w.norm2b);
                 L2B_TRY(make_matrix(m.get(), w.gu, 2 * l.ff, c.width, 2));
                 add_matrix(m.get(), p + "mlp.gate", w.gu, l.ff, 0, 2);
                 add_matrix(m.get(), p + "mlp.up", w.gu, l.ff, 1, 2);
@@ -227,9 +340,10 @@ int32_t stack_model_upload(StackModel* m, const char* name, int dtype, const voi
             }
         }
         if (s.scalar) *s.scalar = v[0];
+        else if (s.host) *s.host = std::move(v);
         else {
             if (!*s.vec) L2B_TRY(alloc_owned(m->owned, (void**)s.vec, (size_t)count * 4));
-            CU(cudaMemcpy(*s.vec, v.data(), (size_t)count * 4, cudaMemcpyHostToDevice));
+            CU(cudaMemcpy(*s.vec + s.vec_at, v.data(), (size_t)count * 4, cudaMemcpyHostToDevice));
         }
     }
     s.loaded = true;
@@ -239,6 +353,16 @@ int32_t stack_model_upload(StackModel* m, const char* name, int dtype, const voi
 int32_t stack_model_finalize(StackModel* m) {
     for (const auto& s : m->slots)
         if (!s.second.loaded) return fail(L2B_ERR_STATE, "tensor " + s.first + " is missing");
+    for (size_t i = 0; i < m->layers.size(); ++i) {
+        StackLayerW& w = m->layers[i];
+        if (m->cfg.layers[i].mix.kind != MixerKind::DifferentialAttention) continue;
+        auto dot = [](const std::vector<float>& a, const std::vector<float>& b) {
+            double v = 0.0;
+            for (size_t k = 0; k < a.size(); ++k) v += (double)a[k] * b[k];
+            return v;
+        };
+        w.head.lambda = (float)(std::exp(dot(w.lq1, w.lk1)) - std::exp(dot(w.lq2, w.lk2)) + (double)m->cfg.layers[i].mix.diff);
+    }
     return L2B_OK;
 }
 
@@ -252,7 +376,7 @@ int64_t stack_model_bytes_per_token(const StackModel* m) {
     int64_t b = m->head.bytes() + (int64_t)m->cfg.width * 2;
     for (const LayerRun& r : m->runs) {
         const StackLayerW& w = m->layers[r.layer];
-        b += w.qdg.bytes() + w.uk.bytes() + w.uv.bytes() + w.o.bytes() + w.gu.bytes() + w.down.bytes() + w.side_gate.bytes() + w.side_proj.bytes();
+        b += w.in.bytes() + w.uk.bytes() + w.uv.bytes() + w.o.bytes() + w.gu.bytes() + w.down.bytes() + w.side_gate.bytes() + w.side_proj.bytes();
     }
     return b;
 }
@@ -265,17 +389,20 @@ struct StackSession {
     StackSessionInfo info;
     DeviceInfo di;
     std::vector<void*> owned;
-    std::vector<void*> cache;                    // per run: [n_seq][seq_len][row] of bf16 or f32
+    // per run, attention: rows of every position in bf16 or f32, [n_seq][groups][seq_len][row] (null: another run's are used)
+    // mLSTM: the f32 states [n_seq][size]
+    std::vector<void*> cache;
     std::vector<size_t> cache_bytes;
+    std::vector<int> cache_run;                  // per run: the run whose cache it uses
     std::vector<const float2*> rope;             // per layer
     // one position
-    float *x[2] = {nullptr, nullptr}, *qdg1 = nullptr, *att1 = nullptr, *hid1 = nullptr, *y1 = nullptr;
+    float *x[2] = {nullptr, nullptr}, *in1 = nullptr, *att1 = nullptr, *hid1 = nullptr, *y1 = nullptr;
     int x_last = 0;
     // absorbed attention: queries and partial results of up to ABSORB_ROWS rows
     float *qp = nullptr, *part_acc = nullptr;
     float2* part_ml = nullptr;
     // many positions
-    float *xr = nullptr, *qdg = nullptr, *y = nullptr;
+    float *xr = nullptr, *in = nullptr, *y = nullptr;
     void *act = nullptr, *act2 = nullptr;        // operands of the products, [max_rows][k rounded up to 8]
     bf16 *pq = nullptr, *pk = nullptr, *pv = nullptr;  // expanded attention: queries, keys, transposed values
     int pv_ld = 0;
@@ -287,10 +414,13 @@ constexpr int ABSORB_ROWS = 64;  // rows per pass of the absorbed form of the at
 // The expanded form of the attention (latent_prefill.cuh) is for portions of at least this many rows.
 constexpr int EXPAND_MIN_ROWS = 48;
 
-// Groups of heads and ranges of positions of the scan kernel: about one block per SM in a decode step, two for several rows.
-static int latent_groups(const LatentShape& s, bool f32) { return f32 ? (s.heads + LA_WARPS - 1) / LA_WARPS : (s.heads + LM_HEADS - 1) / LM_HEADS; }
-static int latent_splits(const LatentShape& s, bool f32, int rows, const DeviceInfo& di) {
-    return std::max(1, std::min(LA_MAX_SPLIT, (rows == 1 ? 1 : 2) * di.sms / (latent_groups(s, f32) * rows)));
+// Blocks of query vectors and ranges of positions of the scan kernel: about one block per SM in a decode step, two for several rows.
+static int scan_blocks(const CacheScan& c, bool f32) {
+    const int per = f32 ? CS_WARPS : CS_MMA_HEADS;
+    return c.heads / c.per_group * ((c.per_group + per - 1) / per);
+}
+static int scan_splits(const CacheScan& c, bool f32, int rows, const DeviceInfo& di) {
+    return std::max(1, std::min(CS_MAX_SPLIT, (rows == 1 ? 1 : 2) * di.sms / (scan_blocks(c, f32) * rows)));
 }
 
 static int prefill_kstages(const LatentShape& s, const DeviceInfo& di) {
@@ -318,10 +448,10 @@ static int32_t set_stack_kernel_attrs() {
         set((const void*)bf16_gemm_kernel<32, 1>); set((const void*)bf16_gemm_kernel<32, 2>);
         set((const void*)bf16_gemm_kernel<64, 1>); set((const void*)bf16_gemm_kernel<64, 2>);
         set((const void*)bf16_gemm_kernel<128, 1>); set((const void*)bf16_gemm_kernel<128, 2>);
-        set((const void*)latent_scan_kernel<float, 1>); set((const void*)latent_scan_kernel<float, 2>);
-        set((const void*)latent_scan_kernel<float, 3>); set((const void*)latent_scan_kernel<float, 4>);
-        set((const void*)latent_scan_mma_kernel<1>); set((const void*)latent_scan_mma_kernel<2>); set((const void*)latent_scan_mma_kernel<3>);
-        set((const void*)latent_scan_mma_kernel<5>); set((const void*)latent_scan_mma_kernel<8>);
+        set((const void*)cache_scan_kernel<float, 1>); set((const void*)cache_scan_kernel<float, 2>);
+        set((const void*)cache_scan_kernel<float, 3>); set((const void*)cache_scan_kernel<float, 4>);
+        set((const void*)cache_scan_mma_kernel<1>); set((const void*)cache_scan_mma_kernel<2>); set((const void*)cache_scan_mma_kernel<3>);
+        set((const void*)cache_scan_mma_kernel<5>); set((const void*)cache_scan_mma_kernel<8>);
     });
     if (g_stack_attr_err != cudaSuccess) return fail(L2B_ERR_CUDA, std::string("cudaFuncSetAttribute: ") + cudaGetErrorString(g_stack_attr_err));
     return L2B_OK;
@@ -331,6 +461,10 @@ static int32_t build_rope(StackSession* s) {
     std::map<std::pair<double, int>, const float2*> made;
     for (const StackLayerConfig& l : s->m->cfg.layers) {
         const RotaryConfig& r = l.mix.rot;
+        if (r.dims == 0) {
+            s->rope.push_back(nullptr);
+            continue;
+        }
         const float2*& t = made[{r.base, r.dims}];
         if (!t) {
             const int h = r.dims / 2;
@@ -357,50 +491,62 @@ int32_t stack_session_create(const StackModel* m, const StackSessionInfo& info, 
     s->info = info;
     s->di = di;
     const StackConfig& c = m->cfg;
-    int max_qdg = 1, max_k = c.width, max_k2 = 1;
+    int max_in = 1, max_k = c.width, max_k2 = 1;
     size_t pq = 0, pk = 0, pv = 0;
     s->pv_ld = up(info.seq_len, 8);
-    for (const StackLayerW& w : m->layers) {
-        max_qdg = std::max(max_qdg, w.qdg.rows);
+    for (size_t i = 0; i < m->layers.size(); ++i) {
+        const StackLayerW& w = m->layers[i];
+        max_in = std::max(max_in, w.in.rows);
         max_k2 = std::max(std::max(max_k2, w.o.k), std::max(w.down.k, w.side_proj.k));
-        pq = std::max(pq, (size_t)w.shape.heads * (w.shape.dp + up(w.shape.rot, 16)));
-        pk = std::max(pk, (size_t)w.shape.heads * w.shape.dp);
-        pv = std::max(pv, (size_t)w.shape.heads * w.shape.vp);
+        if (c.layers[i].mix.kind != MixerKind::LatentAttention) continue;
+        pq = std::max(pq, (size_t)w.latent.heads * (w.latent.dp + up(w.latent.rot, 16)));
+        pk = std::max(pk, (size_t)w.latent.heads * w.latent.dp);
+        pv = std::max(pv, (size_t)w.latent.heads * w.latent.vp);
     }
     auto alloc = [&](auto*& p, size_t bytes) { return alloc_owned(s->owned, (void**)&p, bytes); };
-    for (const LayerRun& r : m->runs) {
-        const size_t b = (size_t)info.n_seq * info.seq_len * m->layers[r.layer].shape.row * act_bytes(m);
+    std::map<int, int> last_run;  // of a layer
+    for (size_t r = 0; r < m->runs.size(); ++r) {
+        const int l = m->runs[r].layer;
+        const MixerConfig& mix = c.layers[l].mix;
+        const StackLayerW& w = m->layers[l];
+        last_run[l] = (int)r;
+        size_t b = 0;
+        if (mix.kind == MixerKind::Mlstm) b = (size_t)info.n_seq * w.mlstm.size() * 4;
+        else if (mix.kv_from < 0) b = (size_t)info.n_seq * (w.scan.heads / w.scan.per_group) * info.seq_len * w.scan.row * act_bytes(m);
         void* p = nullptr;
-        L2B_TRY(alloc_owned(s->owned, &p, b));
+        if (b) L2B_TRY(alloc_owned(s->owned, &p, b));
         s->cache.push_back(p);
         s->cache_bytes.push_back(b);
+        s->cache_run.push_back(mix.kv_from < 0 ? (int)r : last_run[mix.kv_from]);
     }
     L2B_TRY(build_rope(s.get()));
     if (info.decode) {
         for (float*& x : s->x) L2B_TRY(alloc(x, (size_t)c.width * 4));
-        L2B_TRY(alloc(s->qdg1, (size_t)max_qdg * 4));
+        L2B_TRY(alloc(s->in1, (size_t)max_in * 4));
         L2B_TRY(alloc(s->att1, (size_t)max_k2 * 4));
         L2B_TRY(alloc(s->hid1, (size_t)max_k2 * 4));
         L2B_TRY(alloc(s->y1, (size_t)c.width * 4));
     }
     size_t qp = 0, pml = 0, pacc = 0;
-    for (const StackLayerW& w : m->layers)
+    for (const StackLayerW& w : m->layers) {
+        if (!w.scan.heads) continue;
         for (int rows = 1; rows <= std::max(1, std::min(ABSORB_ROWS, info.max_rows)); ++rows) {
-            const size_t pairs = (size_t)w.shape.heads * rows, slots = pairs * latent_splits(w.shape, m->f32, rows, di);
-            qp = std::max(qp, pairs * w.shape.row);
+            const size_t pairs = (size_t)w.scan.heads * rows, slots = pairs * scan_splits(w.scan, m->f32, rows, di);
+            qp = std::max(qp, pairs * w.scan.row);
             pml = std::max(pml, slots);
-            pacc = std::max(pacc, slots * w.shape.rp);
+            pacc = std::max(pacc, slots * w.scan.vcols);
         }
-    L2B_TRY(alloc(s->qp, qp * 4));
-    L2B_TRY(alloc(s->part_ml, pml * sizeof(float2)));
-    L2B_TRY(alloc(s->part_acc, pacc * 4));
+    }
+    L2B_TRY(alloc(s->qp, std::max<size_t>(qp, 1) * 4));
+    L2B_TRY(alloc(s->part_ml, std::max<size_t>(pml, 1) * sizeof(float2)));
+    L2B_TRY(alloc(s->part_acc, std::max<size_t>(pacc, 1) * 4));
     const size_t T = (size_t)info.max_rows;
     L2B_TRY(alloc(s->xr, T * c.width * 4));
-    L2B_TRY(alloc(s->qdg, T * max_qdg * 4));
+    L2B_TRY(alloc(s->in, T * max_in * 4));
     L2B_TRY(alloc(s->y, T * c.width * 4));
     L2B_TRY(alloc(s->act, T * up(max_k, 8) * act_bytes(m)));
     L2B_TRY(alloc(s->act2, T * up(max_k2, 8) * act_bytes(m)));
-    if (!m->f32 && info.n_seq == 1 && info.max_rows >= EXPAND_MIN_ROWS) {
+    if (!m->f32 && info.n_seq == 1 && info.max_rows >= EXPAND_MIN_ROWS && pq) {
         L2B_TRY(alloc(s->pq, T * pq * 2));
         L2B_TRY(alloc(s->pk, (size_t)info.seq_len * pk * 2));
         L2B_TRY(alloc(s->pv, pv * s->pv_ld * 2));
@@ -418,24 +564,49 @@ void stack_session_free(StackSession* s) {
 }
 
 int32_t stack_session_reset(StackSession* s, cudaStream_t st) {
-    for (size_t i = 0; i < s->cache.size(); ++i) CU(cudaMemsetAsync(s->cache[i], 0, s->cache_bytes[i], st));
+    for (size_t i = 0; i < s->cache.size(); ++i)
+        if (s->cache[i]) CU(cudaMemsetAsync(s->cache[i], 0, s->cache_bytes[i], st));
     return L2B_OK;
 }
 int stack_session_max_rows(const StackSession* s) { return s->info.max_rows; }
 const float* stack_session_residual(const StackSession* s) { return s->x[s->x_last]; }
 
-// ---- latent attention launch -------------------------------------------------------------------
-static LatentAttnParams latent_params(const StackSession* s, int run, const float* qdg) {
-    const StackModel* m = s->m;
-    const int l = m->runs[run].layer;
-    const StackLayerW& w = m->layers[l];
+// ---- attention launches ------------------------------------------------------------------------
+// The scan of a run with everything but the rows' positions.
+static CacheScan scan_params(const StackSession* s, int run) {
+    const StackLayerW& w = s->m->layers[s->m->runs[run].layer];
+    CacheScan c = w.scan;
+    c.group_stride = (size_t)s->info.seq_len * c.row;
+    c.cache = s->cache[s->cache_run[run]];
+    c.qp = s->qp; c.part_ml = s->part_ml; c.part_acc = s->part_acc;
+    return c;
+}
+static void plan_scan(CacheScan& c, bool f32, int rows, const DeviceInfo& di) {
+    c.nsplit = scan_splits(c, f32, rows, di);
+    const int stage = f32 ? CS_STAGE_ROWS * c.row * 4 : cs_mma_stage_bytes(c.row);
+    c.stages = std::max(1, std::min(CS_MAX_STAGES, (di.max_smem_optin - 16 * 1024) / stage));
+}
+static cudaError_t launch_scan(const CacheScan& c, bool f32, int rows, cudaStream_t st) {
+    const dim3 grid(scan_blocks(c, f32) * c.nsplit, rows), block(CS_SCAN_THREADS);
+    const size_t smem = (size_t)c.stages * (f32 ? CS_STAGE_ROWS * c.row * 4 : cs_mma_stage_bytes(c.row));
+    auto go = [&](auto k) { return launch_kernel(k, grid, block, smem, st, true, c); };
+    if (f32) {
+        const int pieces = (c.row + 255) / 256;
+        return pieces == 1 ? go(cache_scan_kernel<float, 1>) : pieces == 2 ? go(cache_scan_kernel<float, 2>) : pieces == 3 ? go(cache_scan_kernel<float, 3>) : go(cache_scan_kernel<float, 4>);
+    }
+    return c.row <= 128 ? go(cache_scan_mma_kernel<1>) : c.row <= 256 ? go(cache_scan_mma_kernel<2>) : c.row <= 384 ? go(cache_scan_mma_kernel<3>)
+           : c.row <= 640 ? go(cache_scan_mma_kernel<5>) : go(cache_scan_mma_kernel<8>);
+}
+
+static LatentAttnParams latent_params(const StackSession* s, int run, const float* in) {
+    const int l = s->m->runs[run].layer;
+    const StackLayerW& w = s->m->layers[l];
     LatentAttnParams a;
     memset(&a, 0, sizeof(a));
-    a.s = w.shape;
-    a.qdg = qdg; a.ld = w.qdg.rows; a.off_d = w.off_d; a.off_g = w.off_g;
+    a.s = w.latent;
+    a.c = scan_params(s, run);
+    a.qdg = in; a.ld = w.in.rows; a.off_d = w.off_d; a.off_g = w.off_g;
     a.uk = w.uk.w; a.uv = w.uv.w; a.sink = w.sink; a.dnorm = w.dkv_norm; a.rope = s->rope[l];
-    a.cache = s->cache[run];
-    a.qp = s->qp; a.part_ml = s->part_ml; a.part_acc = s->part_acc;
     return a;
 }
 // The absorbed form for `rows` rows (row pointers already in `a`): query, scan, output.  chained: the first launch depends
@@ -447,23 +618,63 @@ static cudaError_t launch_latent_attention(LatentAttnParams a, int rows, bool ch
     for (a.csplit = 1; a.csplit < 8 && pairs * a.csplit < di.sms;) a.csplit *= 2;
     for (a.vsplit = 1; a.vsplit < 4 && pairs * a.vsplit < di.sms;) a.vsplit *= 2;
     constexpr bool f32 = sizeof(CT) == 4;
-    a.nsplit = latent_splits(s, f32, rows, di);
-    const int stage = f32 ? LA_STAGE_ROWS * s.row * 4 : lm_stage_bytes(s.row);
-    a.stages = std::max(1, std::min(LA_MAX_STAGES, (di.max_smem_optin - 16 * 1024) / stage));
-    cudaError_t e = launch_kernel(latent_query_kernel<CT>, dim3(s.heads * a.csplit + (a.fused ? 1 : 0), rows), dim3(LA_CONSUMERS), 0, st, chained, a);
+    plan_scan(a.c, f32, rows, di);
+    cudaError_t e = launch_kernel(latent_query_kernel<CT>, dim3(s.heads * a.csplit + (a.c.fused ? 1 : 0), rows), dim3(LA_CONSUMERS), 0, st, chained, a);
     if (e != cudaSuccess) return e;
-    const dim3 grid(latent_groups(s, f32) * a.nsplit, rows), block(LA_SCAN_THREADS);
-    const size_t smem = (size_t)a.stages * stage;
-    auto go = [&](auto k) { return launch_kernel(k, grid, block, smem, st, true, a); };
-    if (f32) {
-        const int pieces = (s.row + 255) / 256;
-        e = pieces == 1 ? go(latent_scan_kernel<float, 1>) : pieces == 2 ? go(latent_scan_kernel<float, 2>) : pieces == 3 ? go(latent_scan_kernel<float, 3>) : go(latent_scan_kernel<float, 4>);
-    } else {
-        e = s.row <= 128 ? go(latent_scan_mma_kernel<1>) : s.row <= 256 ? go(latent_scan_mma_kernel<2>) : s.row <= 384 ? go(latent_scan_mma_kernel<3>)
-            : s.row <= 640 ? go(latent_scan_mma_kernel<5>) : go(latent_scan_mma_kernel<8>);
-    }
+    e = launch_scan(a.c, f32, rows, st);
     if (e != cudaSuccess) return e;
     return launch_kernel(latent_output_kernel<OT>, dim3(s.heads * a.vsplit, rows), dim3(LA_CONSUMERS), 0, st, true, a, a.vsplit);
+}
+
+static HeadAttnParams head_params(const StackSession* s, int run, const float* in) {
+    const int l = s->m->runs[run].layer;
+    const StackLayerW& w = s->m->layers[l];
+    HeadAttnParams a;
+    memset(&a, 0, sizeof(a));
+    a.s = w.head;
+    a.c = scan_params(s, run);
+    a.in = in; a.ld = w.in.rows; a.off_k = w.off_k; a.off_v = w.off_v; a.off_g = w.off_g;
+    a.own_kv = s->cache_run[run] == run;
+    a.qnorm = w.q_norm; a.knorm = w.k_norm; a.rope = s->rope[l];
+    return a;
+}
+template <typename CT>
+static cudaError_t launch_head_rows(const HeadAttnParams& a, int rows, bool chained, cudaStream_t st) {
+    const int items = 2 * a.s.heads + (a.own_kv ? 3 * a.s.kv_heads : 0);
+    return launch_kernel(head_rows_kernel<CT>, dim3((items + HA_WARPS - 1) / HA_WARPS, rows), dim3(HA_WARPS * 32), 0, st, chained, a);
+}
+// Differential attention of `rows` rows: query vectors and new cache rows, scan, output.
+template <typename CT, typename OT>
+static cudaError_t launch_head_attention(HeadAttnParams a, int rows, bool chained, const DeviceInfo& di, cudaStream_t st) {
+    constexpr bool f32 = sizeof(CT) == 4;
+    plan_scan(a.c, f32, rows, di);
+    cudaError_t e = launch_head_rows<CT>(a, rows, chained, st);
+    if (e != cudaSuccess) return e;
+    e = launch_scan(a.c, f32, rows, st);
+    if (e != cudaSuccess) return e;
+    return launch_kernel(head_output_kernel<OT>, dim3(a.s.heads, rows), dim3(HA_WARPS * 32), 0, st, true, a);
+}
+
+// ---- mLSTM launches ----------------------------------------------------------------------------
+static MlstmParams mlstm_params(const StackSession* s, int run, const float* in) {
+    const StackLayerW& w = s->m->layers[s->m->runs[run].layer];
+    MlstmParams a;
+    memset(&a, 0, sizeof(a));
+    a.s = w.mlstm;
+    a.in = in; a.ld = w.in.rows; a.off_k = w.off_k; a.off_v = w.off_v; a.off_g = w.off_g; a.off_i = w.off_i; a.off_f = w.off_f;
+    a.norm = w.out_norm;
+    a.state = static_cast<float*>(s->cache[run]);
+    a.tokens = 1;
+    return a;
+}
+// `rows` sequences by one token each, or (rows = 1) a.tokens tokens of one sequence.
+template <typename OT>
+static cudaError_t launch_mlstm_step(const MlstmParams& a, int rows, bool chained, cudaStream_t st) {
+    const dim3 grid(a.s.heads * a.s.cl, rows);
+    auto go = [&](auto k) { return launch_kernel(k, grid, dim3(ML_THREADS), 0, st, chained, a, a.s.cl); };
+    if (a.s.dim <= ML_WARPS * 16)
+        return a.s.cpl == 1 ? go(mlstm_step_kernel<16, 1, OT>) : a.s.cpl == 2 ? go(mlstm_step_kernel<16, 2, OT>) : go(mlstm_step_kernel<16, 4, OT>);
+    return a.s.cpl == 1 ? go(mlstm_step_kernel<32, 1, OT>) : a.s.cpl == 2 ? go(mlstm_step_kernel<32, 2, OT>) : go(mlstm_step_kernel<32, 4, OT>);
 }
 
 // ---- one position ------------------------------------------------------------------------------
@@ -486,15 +697,26 @@ static int32_t launch_dense_matvec(const StackSession* s, const StackMatrix& w, 
     return L2B_OK;
 }
 
+static EmbedParams embed_params(const StackModel* m, const int* tokens, float* x) {
+    EmbedParams e;
+    memset(&e, 0, sizeof(e));
+    e.table = m->embed.w; e.tokens = tokens; e.width = m->cfg.width; e.vocab = m->cfg.vocab; e.scale = m->cfg.embed_scale;
+    e.pos_table = m->positions.w; e.max_positions = m->cfg.max_positions;
+    e.x = x;
+    return e;
+}
+static int mlp_epilogue(MlpKind k) { return k == MlpKind::GatedSilu ? DE_SWIGLU : DE_GEGLU; }
+
 int32_t stack_enqueue_token(StackSession* s, const int* token, const int* pos, float* logits, float* amax_val, int* amax_idx, int* status, cudaStream_t st,
                             int* nlaunch, int* nparts) {
     const StackModel* m = s->m;
     const StackConfig& c = m->cfg;
     int count = 0, cur = 0;
-    CU(launch_kernel_args(scaled_embed_kernel, dim3(std::max(1, std::min(32, c.width / 256))), dim3(256), 0, st, false, 1, (const bf16*)m->embed.w, token, c.width, c.vocab,
-                          c.embed_scale, s->x[0]));
+    EmbedParams ep = embed_params(m, token, s->x[0]);
+    ep.pos = pos;
+    CU(launch_kernel(embed_positions_kernel, dim3(std::max(1, std::min(32, c.width / 256)), 1), dim3(256), 0, st, false, ep));
     ++count;
-    const float* side_w = nullptr;  // non-null: y1 awaits its norm and its place in the residual stream
+    const float* add_w = nullptr;  // non-null: y1 awaits its norm (this is its weight) and its place in the residual stream
     const float* step = nullptr;
     // the residual stream as input of a product, with whatever is pending applied on the way
     auto from_residual = [&](DmvParams& p, const StackNorm* norm) {
@@ -503,26 +725,31 @@ int32_t stack_enqueue_token(StackSession* s, const int* token, const int* pos, f
         if (norm) p.norm = norm_params(m, *norm);
         p.upd.eps = c.eps;
         p.upd.step = step;
-        if (side_w) {
+        if (add_w) {
             p.upd.y = s->y1;
-            p.upd.side_w = side_w;
+            p.upd.w = add_w;
         }
-        if (step || side_w) {
+        if (step || add_w) {
             cur ^= 1;
             p.x_out = s->x[cur];
         }
-        step = side_w = nullptr;
+        step = add_w = nullptr;
     };
     auto from_vector = [&](DmvParams& p, const float* x) {
         memset(&p, 0, sizeof(p));
         p.x = x;
     };
-    auto mv = [&](const StackMatrix& w, DmvParams& p, int kind, float* out, int* nb = nullptr) -> int32_t {
-        p.epi.kind = kind;
-        p.epi.y = out;
-        p.epi.act = out;
+    auto mv_epi = [&](const StackMatrix& w, DmvParams& p, const DenseEpilogue& e, int* nb = nullptr) -> int32_t {
+        p.epi = e;
         ++count;
         return launch_dense_matvec(s, w, p, status, st, nb);
+    };
+    auto mv = [&](const StackMatrix& w, DmvParams& p, int kind, float* out) -> int32_t { return mv_epi(w, p, dense_epilogue_of(kind, out, out, 0)); };
+    // a sublayer's result: added to the residual stream, or kept for its norm
+    auto result = [&](const StackMatrix& w, DmvParams& p, const StackNorm& post) -> int32_t {
+        if (!c.post_norm) return mv(w, p, DE_RESIDUAL, s->x[cur]);
+        add_w = post.w;
+        return mv(w, p, DE_STORE, s->y1);
     };
     DmvParams p;
     for (size_t r = 0; r < m->runs.size(); ++r) {
@@ -530,43 +757,71 @@ int32_t stack_enqueue_token(StackSession* s, const int* token, const int* pos, f
         const StackLayerW& w = m->layers[l];
         if (m->runs[r].pass >= 0) step = m->loop_step + (size_t)m->runs[r].pass * c.width;
         from_residual(p, &w.norm1);
-        L2B_TRY(mv(w.qdg, p, DE_STORE, s->qdg1));
-        {
-            LatentAttnParams a = latent_params(s, (int)r, s->qdg1);
-            a.pos = pos;
-            a.out = s->att1;
-            a.ldo = w.o.k;
-            a.fused = 1;
-            a.status = status;
-            CU(m->f32 ? (launch_latent_attention<float, float>(a, 1, true, s->di, st)) : (launch_latent_attention<bf16, float>(a, 1, true, s->di, st)));
-            count += 3;
+        DenseEpilogue proj = dense_epilogue_of(DE_STORE, s->in1, nullptr, 0);
+        proj.bias = w.in_bias;
+        L2B_TRY(mv_epi(w.in, p, proj));
+        switch (c.layers[l].mix.kind) {
+            case MixerKind::LatentAttention: {
+                LatentAttnParams a = latent_params(s, (int)r, s->in1);
+                a.c.pos = pos;
+                a.c.fused = 1;
+                a.c.status = status;
+                a.out = s->att1;
+                a.ldo = w.o.k;
+                CU(m->f32 ? (launch_latent_attention<float, float>(a, 1, true, s->di, st)) : (launch_latent_attention<bf16, float>(a, 1, true, s->di, st)));
+                count += 3;
+                break;
+            }
+            case MixerKind::DifferentialAttention: {
+                HeadAttnParams a = head_params(s, (int)r, s->in1);
+                a.c.pos = pos;
+                a.c.fused = 1;
+                a.c.status = status;
+                a.out = s->att1;
+                a.ldo = w.o.k;
+                CU(m->f32 ? (launch_head_attention<float, float>(a, 1, true, s->di, st)) : (launch_head_attention<bf16, float>(a, 1, true, s->di, st)));
+                count += 3;
+                break;
+            }
+            case MixerKind::Mlstm: {
+                MlstmParams a = mlstm_params(s, (int)r, s->in1);
+                a.pos = pos;
+                a.out = s->att1;
+                a.ldo = w.o.k;
+                CU(launch_mlstm_step<float>(a, 1, true, st));
+                ++count;
+                break;
+            }
         }
         from_vector(p, s->att1);
-        L2B_TRY(mv(w.o, p, DE_RESIDUAL, s->x[cur]));
+        L2B_TRY(result(w.o, p, w.norm1b));
         if (w.gu.w) {
             from_residual(p, &w.norm2);
-            L2B_TRY(mv(w.gu, p, DE_GEGLU, s->hid1));
+            L2B_TRY(mv(w.gu, p, mlp_epilogue(c.layers[l].mlp), s->hid1));
             from_vector(p, s->hid1);
-            L2B_TRY(mv(w.down, p, DE_RESIDUAL, s->x[cur]));
+            L2B_TRY(result(w.down, p, w.norm2b));
         }
         if (c.side_dim) {
             from_residual(p, nullptr);
-            p.epi.etab = m->side_embed.w;
-            p.epi.e_ld = m->side_embed.kp;
-            p.epi.e_off = l * c.side_dim;
-            p.epi.tokens = token;
-            p.epi.vocab = c.vocab;
-            L2B_TRY(mv(w.side_gate, p, DE_SIDE, s->hid1));
+            DenseEpilogue e = dense_epilogue_of(DE_SIDE, nullptr, s->hid1, 0);
+            e.etab = m->side_embed.w;
+            e.e_ld = m->side_embed.kp;
+            e.e_off = l * c.side_dim;
+            e.tokens = token;
+            e.vocab = c.vocab;
+            L2B_TRY(mv_epi(w.side_gate, p, e));
             from_vector(p, s->hid1);
             L2B_TRY(mv(w.side_proj, p, DE_STORE, s->y1));
-            side_w = w.side_norm;
+            add_w = w.side_norm;
         }
     }
     from_residual(p, &m->final_norm);
     s->x_last = cur;
     p.amax_val = amax_val;
     p.amax_idx = amax_idx;
-    L2B_TRY(mv(m->head, p, DE_LOGITS, logits, nparts));
+    DenseEpilogue e = dense_epilogue_of(DE_LOGITS, logits, nullptr, 0);
+    e.mul = c.logit_scale;
+    L2B_TRY(mv_epi(m->head, p, e, nparts));
     if (nlaunch) *nlaunch = count;
     return L2B_OK;
 }
@@ -637,16 +892,31 @@ static int32_t launch_residual_rows(const StackSession* s, const RowsParams& r, 
     return L2B_OK;
 }
 
-// Attention of n rows: latents and rotated keys into the cache, then the expanded form (long portions of one sequence, bf16) or the
-// absorbed form.  Result (gated) in act2 [n][ldo].
+// A pass over rows in parts of at most ABSORB_ROWS: go(parameters of the part, its rows).
+template <class P, class Go>
+static int32_t rows_in_parts(const StackSession* s, const P& a, int n, const Go& go) {
+    for (int r = 0; r < n; r += ABSORB_ROWS) {
+        P b = a;
+        b.c.pos0 += r;
+        if (b.c.pos_list) b.c.pos_list += r;
+        b.c.cache = static_cast<uint8_t*>(a.c.cache) + (size_t)r * a.c.cache_stride * act_bytes(s->m);
+        b.out = static_cast<uint8_t*>(a.out) + (size_t)r * a.ldo * act_bytes(s->m);
+        CU(go(b, r, std::min(ABSORB_ROWS, n - r)));
+    }
+    return L2B_OK;
+}
+
+// Latent attention of n rows: latents and rotated keys into the cache, then the expanded form (long portions of one sequence, bf16) or
+// the absorbed form.  Result (gated) in act2 [n][ldo].
 static int32_t enqueue_latent_rows(StackSession* s, int run, int n, int pos0, const int* pos_list, int ldo, int* status, cudaStream_t st, long long* launches) {
     const StackModel* m = s->m;
     const StackLayerW& w = m->layers[m->runs[run].layer];
-    const LatentShape& sh = w.shape;
-    LatentAttnParams a = latent_params(s, run, s->qdg);
-    a.pos0 = pos0;
-    a.pos_list = pos_list;
-    a.cache_stride = pos_list ? (size_t)s->info.seq_len * sh.row : 0;
+    const LatentShape& sh = w.latent;
+    LatentAttnParams a = latent_params(s, run, s->in);
+    a.c.pos0 = pos0;
+    a.c.pos_list = pos_list;
+    a.c.cache_stride = pos_list ? (size_t)s->info.seq_len * sh.row : 0;
+    a.c.status = status;
     a.out = s->act2;
     a.ldo = ldo;
     if (m->f32) latent_rows_kernel<float><<<n, 128, 0, st>>>(a);
@@ -654,39 +924,22 @@ static int32_t enqueue_latent_rows(StackSession* s, int run, int n, int pos0, co
     CU(cudaGetLastError());
     ++*launches;
     const int kstages = prefill_kstages(sh, s->di);
-    if (!s->pq || pos_list || n < EXPAND_MIN_ROWS || kstages == 0 || !(sh.scale2 > 0.f)) {
-        a.status = status;
-        for (int r = 0; r < n; r += ABSORB_ROWS) {
-            const int k = std::min(ABSORB_ROWS, n - r);
-            LatentAttnParams b = a;
+    if (!s->pq || pos_list || n < EXPAND_MIN_ROWS || kstages == 0 || !(sh.scale2 > 0.f))
+        return rows_in_parts(s, a, n, [&](LatentAttnParams& b, int r, int k) {
             b.qdg += (size_t)r * a.ld;
-            b.pos0 += r;
-            if (pos_list) b.pos_list += r;
-            b.cache = static_cast<uint8_t*>(a.cache) + (size_t)r * a.cache_stride * act_bytes(m);
-            b.out = static_cast<uint8_t*>(a.out) + (size_t)r * ldo * act_bytes(m);
-            CU(m->f32 ? (launch_latent_attention<float, float>(b, k, false, s->di, st)) : (launch_latent_attention<bf16, bf16>(b, k, false, s->di, st)));
             *launches += 3;
-        }
-        return L2B_OK;
-    }
+            return m->f32 ? (launch_latent_attention<float, float>(b, k, false, s->di, st)) : (launch_latent_attention<bf16, bf16>(b, k, false, s->di, st));
+        });
     const int npos = pos0 + n, dq = sh.dp + up(sh.rot, 16);
-    const bf16* cache = static_cast<const bf16*>(a.cache);
-    DenseEpilogue e;
-    memset(&e, 0, sizeof(e));
-    e.kind = DE_STORE_ACT;
-    e.act = s->pk;
-    e.ld = sh.heads * sh.dp;
-    L2B_TRY(launch_gemm(s, w.uk, cache, sh.row, npos, e, status, st));
-    e.kind = DE_STORE_T;
-    e.act = s->pv;
-    e.ld = s->pv_ld;
-    L2B_TRY(launch_gemm(s, w.uv, cache, sh.row, npos, e, status, st));
-    latent_queries_kernel<<<dim3(n, sh.heads), 128, 0, st>>>(s->qdg, a.ld, a.rope, pos0, sh, dq, s->pq);
+    const bf16* cache = static_cast<const bf16*>(a.c.cache);
+    L2B_TRY(launch_gemm(s, w.uk, cache, sh.row, npos, dense_epilogue_of(DE_STORE_ACT, nullptr, s->pk, sh.heads * sh.dp), status, st));
+    L2B_TRY(launch_gemm(s, w.uv, cache, sh.row, npos, dense_epilogue_of(DE_STORE_T, nullptr, s->pv, s->pv_ld), status, st));
+    latent_queries_kernel<<<dim3(n, sh.heads), 128, 0, st>>>(s->in, a.ld, a.rope, pos0, sh, dq, s->pq);
     CU(cudaGetLastError());
     LatentPrefillParams f;
     memset(&f, 0, sizeof(f));
     f.n = n; f.pos0 = pos0; f.dim = sh.dim; f.rot = sh.rot; f.vdim = sh.vdim; f.dp = sh.dp; f.dq = dq; f.vp = sh.vp; f.kstages = kstages;
-    f.scale2 = sh.scale2; f.sink = w.sink; f.gate = s->qdg + w.off_g; f.ld = a.ld; f.out = static_cast<bf16*>(s->act2); f.ldo = ldo; f.status = status;
+    f.scale2 = sh.scale2; f.sink = w.sink; f.gate = s->in + w.off_g; f.ld = a.ld; f.out = static_cast<bf16*>(s->act2); f.ldo = ldo; f.status = status;
     CUtensorMap mq, mk, mkr, mv;
     L2B_TRY(bf16_map(mq, s->pq, (int64_t)sh.heads * dq, n, (int64_t)sh.heads * dq, LP_TILE));
     L2B_TRY(bf16_map(mk, s->pk, (int64_t)sh.heads * sh.dp, npos, (int64_t)sh.heads * sh.dp, LP_TILE));
@@ -698,16 +951,51 @@ static int32_t enqueue_latent_rows(StackSession* s, int run, int n, int pos0, co
     return L2B_OK;
 }
 
+// Differential attention of n rows.  Result (gated) in act2 [n][ldo].
+static int32_t enqueue_head_rows(StackSession* s, int run, int n, int pos0, const int* pos_list, int ldo, int* status, cudaStream_t st, long long* launches) {
+    const StackModel* m = s->m;
+    HeadAttnParams a = head_params(s, run, s->in);
+    a.c.pos0 = pos0;
+    a.c.pos_list = pos_list;
+    a.c.cache_stride = pos_list ? (size_t)a.s.kv_heads * a.c.group_stride : 0;
+    a.c.status = status;
+    a.out = s->act2;
+    a.ldo = ldo;
+    return rows_in_parts(s, a, n, [&](HeadAttnParams& b, int r, int k) {
+        b.in += (size_t)r * a.ld;
+        *launches += 3;
+        return m->f32 ? (launch_head_attention<float, float>(b, k, false, s->di, st)) : (launch_head_attention<bf16, bf16>(b, k, false, s->di, st));
+    });
+}
+
+// mLSTM of n rows: n tokens of one sequence, or one of every sequence.  Result (gated) in act2 [n][ldo].
+static int32_t enqueue_mlstm_rows(StackSession* s, int run, int n, int pos0, const int* pos_list, int ldo, cudaStream_t st, long long* launches) {
+    const StackModel* m = s->m;
+    MlstmParams a = mlstm_params(s, run, s->in);
+    a.pos0 = pos0;
+    a.pos_list = pos_list;
+    a.state_stride = pos_list ? a.s.size() : 0;
+    a.tokens = pos_list ? 1 : n;
+    a.out = s->act2;
+    a.ldo = ldo;
+    const int rows = pos_list ? n : 1;
+    CU(m->f32 ? launch_mlstm_step<float>(a, rows, false, st) : launch_mlstm_step<bf16>(a, rows, false, st));
+    ++*launches;
+    return L2B_OK;
+}
+
 int32_t stack_enqueue_rows(StackSession* s, const int* dev_tokens, int n, int pos0, const int* pos_list, int* status, cudaStream_t st, long long* launches) {
     const StackModel* m = s->m;
     const StackConfig& c = m->cfg;
     if (n < 1 || n > s->info.max_rows) return fail(L2B_ERR_BAD_ARG, "too many rows for one pass");
     long long count = 0;
-    CU(launch_kernel_args(scaled_embed_kernel, dim3(std::max(1, std::min(16, c.width / 256)), n), dim3(256), 0, st, false, 1, (const bf16*)m->embed.w, dev_tokens, c.width,
-                          c.vocab, c.embed_scale, s->xr));
+    EmbedParams ep = embed_params(m, dev_tokens, s->xr);
+    ep.pos0 = pos0;
+    ep.pos_list = pos_list;
+    CU(launch_kernel(embed_positions_kernel, dim3(std::max(1, std::min(16, c.width / 256)), n), dim3(256), 0, st, false, ep));
     ++count;
     const int lda = up(c.width, 8);
-    const float* side_w = nullptr;
+    const float* add_w = nullptr;  // non-null: y awaits its norm (this is its weight) and its place in the residual stream
     const float* step = nullptr;
     // the residual stream, with whatever is pending applied, normed into the operand buffer
     auto from_residual = [&](const StackNorm* norm, bool operand) -> int32_t {
@@ -717,60 +1005,62 @@ int32_t stack_enqueue_rows(StackSession* s, const int* dev_tokens, int n, int po
         r.width = c.width;
         r.upd.eps = c.eps;
         r.upd.step = step;
-        if (side_w) {
+        if (add_w) {
             r.upd.y = s->y;
-            r.upd.side_w = side_w;
+            r.upd.w = add_w;
         }
-        r.store_x = step || side_w;
+        r.store_x = step || add_w;
         if (norm) r.norm = norm_params(m, *norm);
         if (operand) r.act = s->act;
         r.lda = lda;
-        step = side_w = nullptr;
+        step = add_w = nullptr;
         ++count;
         return launch_residual_rows(s, r, n, st);
     };
-    auto gemm = [&](const StackMatrix& w, const void* x, int kind, float* y, void* act, int ld) -> int32_t {
-        DenseEpilogue e;
-        memset(&e, 0, sizeof(e));
-        e.kind = kind;
-        e.y = y;
-        e.act = act;
-        e.ld = ld;
+    auto gemm_epi = [&](const StackMatrix& w, const void* x, const DenseEpilogue& e) -> int32_t {
         ++count;
         return launch_gemm(s, w, x, up(w.k, 8), n, e, status, st);
+    };
+    auto gemm = [&](const StackMatrix& w, const void* x, int kind, float* y, void* act, int ld) -> int32_t { return gemm_epi(w, x, dense_epilogue_of(kind, y, act, ld)); };
+    // a sublayer's result: added to the residual stream, or kept for its norm
+    auto result = [&](const StackMatrix& w, const StackNorm& post) -> int32_t {
+        if (!c.post_norm) return gemm(w, s->act2, DE_RESIDUAL, s->xr, nullptr, c.width);
+        add_w = post.w;
+        return gemm(w, s->act2, DE_STORE, s->y, nullptr, c.width);
     };
     for (size_t r = 0; r < m->runs.size(); ++r) {
         const int l = m->runs[r].layer;
         const StackLayerW& w = m->layers[l];
         if (m->runs[r].pass >= 0) step = m->loop_step + (size_t)m->runs[r].pass * c.width;
         L2B_TRY(from_residual(&w.norm1, true));
-        L2B_TRY(gemm(w.qdg, s->act, DE_STORE, s->qdg, nullptr, w.qdg.rows));
-        L2B_TRY(enqueue_latent_rows(s, (int)r, n, pos0, pos_list, up(w.o.k, 8), status, st, &count));
-        L2B_TRY(gemm(w.o, s->act2, DE_RESIDUAL, s->xr, nullptr, c.width));
+        DenseEpilogue proj = dense_epilogue_of(DE_STORE, s->in, nullptr, w.in.rows);
+        proj.bias = w.in_bias;
+        L2B_TRY(gemm_epi(w.in, s->act, proj));
+        switch (c.layers[l].mix.kind) {
+            case MixerKind::LatentAttention: L2B_TRY(enqueue_latent_rows(s, (int)r, n, pos0, pos_list, up(w.o.k, 8), status, st, &count)); break;
+            case MixerKind::DifferentialAttention: L2B_TRY(enqueue_head_rows(s, (int)r, n, pos0, pos_list, up(w.o.k, 8), status, st, &count)); break;
+            case MixerKind::Mlstm: L2B_TRY(enqueue_mlstm_rows(s, (int)r, n, pos0, pos_list, up(w.o.k, 8), st, &count)); break;
+        }
+        L2B_TRY(result(w.o, w.norm1b));
         if (w.gu.w) {
             L2B_TRY(from_residual(&w.norm2, true));
-            L2B_TRY(gemm(w.gu, s->act, DE_GEGLU, nullptr, s->act2, up(w.down.k, 8)));
-            L2B_TRY(gemm(w.down, s->act2, DE_RESIDUAL, s->xr, nullptr, c.width));
+            L2B_TRY(gemm(w.gu, s->act, mlp_epilogue(c.layers[l].mlp), nullptr, s->act2, up(w.down.k, 8)));
+            L2B_TRY(result(w.down, w.norm2b));
         }
         if (c.side_dim) {
             L2B_TRY(from_residual(nullptr, true));
-            DenseEpilogue e;
-            memset(&e, 0, sizeof(e));
-            e.kind = DE_SIDE;
-            e.act = s->act2;
-            e.ld = up(c.side_dim, 8);
+            DenseEpilogue e = dense_epilogue_of(DE_SIDE, nullptr, s->act2, up(c.side_dim, 8));
             e.etab = m->side_embed.w;
             e.e_ld = m->side_embed.kp;
             e.e_off = l * c.side_dim;
             e.tokens = dev_tokens;
             e.vocab = c.vocab;
-            L2B_TRY(launch_gemm(s, w.side_gate, s->act, lda, n, e, status, st));
-            ++count;
+            L2B_TRY(gemm_epi(w.side_gate, s->act, e));
             L2B_TRY(gemm(w.side_proj, s->act2, DE_STORE, s->y, nullptr, c.width));
-            side_w = w.side_norm;
+            add_w = w.side_norm;
         }
     }
-    if (side_w) L2B_TRY(from_residual(nullptr, false));
+    if (add_w) L2B_TRY(from_residual(nullptr, false));
     if (launches) *launches += count;
     return L2B_OK;
 }
@@ -786,11 +1076,8 @@ int32_t stack_enqueue_logits(StackSession* s, const int* dev_index, int n, float
     r.act = s->act;
     r.lda = up(m->cfg.width, 8);
     L2B_TRY(launch_residual_rows(s, r, n, st));
-    DenseEpilogue e;
-    memset(&e, 0, sizeof(e));
-    e.kind = DE_STORE;
-    e.y = logits;
-    e.ld = m->cfg.vocab;
+    DenseEpilogue e = dense_epilogue_of(DE_STORE, logits, nullptr, m->cfg.vocab);
+    e.mul = m->cfg.logit_scale;
     L2B_TRY(launch_gemm(s, m->head, s->act, r.lda, n, e, status, st));
     if (launches) *launches += 2;
     return L2B_OK;

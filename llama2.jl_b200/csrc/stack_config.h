@@ -11,11 +11,11 @@
 
 namespace l2b {
 
-enum class MixerKind { LatentAttention };
-enum class MlpKind { None, GatedGeluTanh };
-enum class NormKind { DynamicTanh };
+enum class MixerKind { LatentAttention, DifferentialAttention, Mlstm };
+enum class MlpKind { None, GatedGeluTanh, GatedSilu };
+enum class NormKind { DynamicTanh, Rms };
 
-struct RotaryConfig {  // interleaved pairs (2i, 2i+1), i < dims/2, turned by position * base^(-2i/dims)
+struct RotaryConfig {  // pair i < dims/2 is turned by position * base^(-2i/dims); which two dimensions form it is the mixer's
     double base = 10000.0;
     int dims = 0;
 };
@@ -23,12 +23,20 @@ struct RotaryConfig {  // interleaved pairs (2i, 2i+1), i < dims/2, turned by po
 struct MixerConfig {
     MixerKind kind = MixerKind::LatentAttention;
     int heads = 0;
-    int dim = 0;      // unrotated query / key dimensions per head
-    int rot_dim = 0;  // rotated ones; the rotated key part is shared by all heads
+    int dim = 0;      // query / key dimensions per head (latent attention: the unrotated ones; differential attention: per map)
     int vdim = 0;     // value dimensions per head
-    int kv_rank = 0;  // size of the cached latent
     float scale = 1.f;
     RotaryConfig rot;
+    // latent attention
+    int rot_dim = 0;  // rotated dimensions; the rotated key part is shared by all heads
+    int kv_rank = 0;  // size of the cached latent
+    // differential attention
+    int kv_heads = 0;
+    int chunk = 0;      // a position sees its own chunk of this many positions (0: everything before it)
+    float diff = 0.f;   // constant part of the second map's weight
+    int kv_from = -1;   // layer whose cached keys and values are used (-1: this layer has its own)
+    // matrix memory (mLSTM)
+    float gate_cap = 1.f;
 };
 
 struct StackLayerConfig {
@@ -46,12 +54,16 @@ struct StackConfig {
     std::string architecture;
     int vocab = 0, width = 0;
     float embed_scale = 1.f;
+    int max_positions = 0;   // rows of the table of learned position vectors (0: there is none)
+    float logit_scale = 1.f;
     NormKind norm = NormKind::DynamicTanh;
+    bool post_norm = false;  // the result of a sublayer is normed before it is added to the residual stream
     float eps = 1e-5f;
     int loop_start = 0, loop_stop = 0, loop_times = 0;  // layers start .. stop-1 run `times` times in a row (0 times: no loop)
     int side_dim = 0;                                   // per-layer token input (0: none)
     std::vector<StackLayerConfig> layers;
     bool has_loop() const { return loop_times > 0; }
+    bool recurrent() const;              // some layer carries a state from position to position
     std::vector<LayerRun> runs() const;  // the layers in the order they run; every run has a cache of its own
 };
 

@@ -6,15 +6,31 @@
 
 namespace l2b {
 
-// x[t] = scale * table[tokens[t]]; a token id outside [0, vocab) gives a row of zeros (the table is never read out of bounds).
-// Grid (blocks per row, rows).
-__global__ void scaled_embed_kernel(const bf16* __restrict__ table, const int* tokens, int width, int vocab, float scale, float* __restrict__ x) {
+// x[t] = scale * table[tokens[t]] + pos_table[position of t]; a token id outside [0, vocab) gives a table row of zeros (no table is
+// read out of bounds).  Grid (blocks per row, rows).
+struct EmbedParams {
+    const bf16* table;
+    const int* tokens;
+    int width, vocab;
+    float scale;
+    const bf16* pos_table;  // learned position vectors (null: none)
+    int max_positions;
+    const int* pos;         // decode: device scalar
+    const int* pos_list;    // batched decode: position of every row
+    int pos0;               // otherwise row r sits at pos0 + r
+    float* x;
+};
+__global__ void embed_positions_kernel(const __grid_constant__ EmbedParams p) {
     pdl_launch_dependents();
     pdl_wait();
-    const int tok = __ldcg(tokens + blockIdx.y);
-    const bool valid = tok >= 0 && tok < vocab;
-    for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < width; i += gridDim.x * blockDim.x)
-        x[(size_t)blockIdx.y * width + i] = valid ? scale * __bfloat162float(table[(size_t)tok * width + i]) : 0.f;
+    const int row = (int)blockIdx.y, tok = __ldcg(p.tokens + row);
+    const bool valid = tok >= 0 && tok < p.vocab;
+    const int pos = p.pos ? __ldcg(p.pos) : p.pos_list ? __ldcg(p.pos_list + row) : p.pos0 + row;
+    const bf16* const pv = p.pos_table && pos >= 0 && pos < p.max_positions ? p.pos_table + (size_t)pos * p.width : nullptr;
+    for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < p.width; i += gridDim.x * blockDim.x) {
+        const float e = valid ? p.scale * __bfloat162float(p.table[(size_t)tok * p.width + i]) : 0.f;
+        p.x[(size_t)row * p.width + i] = pv ? e + __bfloat162float(pv[i]) : e;
+    }
 }
 
 struct RowsParams {
@@ -30,7 +46,7 @@ struct RowsParams {
 // V: values a thread takes at a time (4 when width and lda allow 16-byte accesses, else 1)
 template <typename AT, int V>
 __global__ void __launch_bounds__(256) residual_rows_kernel(const __grid_constant__ RowsParams p) {
-    __shared__ float s_red[8];
+    __shared__ float s_red[8], s_red2[8];
     struct alignas(4 * V) F { float v[V]; };
     struct alignas(sizeof(AT) * V) A { AT v[V]; };
     const int src = p.index ? __ldg(p.index + blockIdx.x) : (int)blockIdx.x;
@@ -48,21 +64,35 @@ __global__ void __launch_bounds__(256) residual_rows_kernel(const __grid_constan
         scale = 1.f / sqrtf(block_sum_all<8>(ss, s_red) / (float)p.width + p.upd.eps);
     }
     A* const act = p.act ? reinterpret_cast<A*>(static_cast<AT*>(p.act) + (size_t)blockIdx.x * p.lda) : nullptr;
-    for (int i = threadIdx.x; i < n; i += 256) {
+    auto updated = [&](int i) {
         F t = x[i];
         if (y) {
             const F b = y[i];
 #pragma unroll
-            for (int k = 0; k < V; ++k) t.v[k] = fmaf(b.v[k] * scale, __ldg(p.upd.side_w + i * V + k), t.v[k]);
+            for (int k = 0; k < V; ++k) t.v[k] = fmaf(b.v[k] * scale, __ldg(p.upd.w + i * V + k), t.v[k]);
         }
         if (p.upd.step)
 #pragma unroll
             for (int k = 0; k < V; ++k) t.v[k] += __ldg(p.upd.step + i * V + k);
+        return t;
+    };
+    float rms_scale = 1.f;
+    if (act && p.norm.kind == NORM_RMS) {  // (the second pass finds its inputs in the first-level cache)
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < n; i += 256) {
+            const F t = updated(i);
+#pragma unroll
+            for (int k = 0; k < V; ++k) ss = fmaf(t.v[k], t.v[k], ss);
+        }
+        rms_scale = 1.f / sqrtf(block_sum_all<8>(ss, s_red2) / (float)p.width + p.norm.eps);
+    }
+    for (int i = threadIdx.x; i < n; i += 256) {
+        const F t = updated(i);
         if (p.store_x) x[i] = t;
         if (act) {
             A o;
 #pragma unroll
-            for (int k = 0; k < V; ++k) put(&o.v[k], apply_norm(p.norm, t.v[k], i * V + k));
+            for (int k = 0; k < V; ++k) put(&o.v[k], apply_norm(p.norm, t.v[k], i * V + k) * rms_scale);
             act[i] = o;
         }
     }

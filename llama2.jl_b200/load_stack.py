@@ -7,7 +7,7 @@ from .model import LanguageModel, StackConfig, _DeviceModel
 
 # config.json "architecture" -> configuration class.  The library has its own table of the same names (csrc/stack_config.cpp),
 # which knows the designs themselves.
-ARCHITECTURES = {"Savozen": StackConfig}
+ARCHITECTURES = {"Savozen": StackConfig, "Perezen": StackConfig}
 
 
 def load_stack_model(path: str, seq_len: int, compute: str = "bfloat16", device: int = -1, stream=None) -> LanguageModel:

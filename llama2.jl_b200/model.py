@@ -104,6 +104,10 @@ class StackConfig:
     seq_len: int
     compute: str = "bfloat16"
 
+    def __post_init__(self):
+        if self.raw.get("max_positions"):  # learned position vectors: there are none beyond
+            self.seq_len = min(self.seq_len, int(self.raw["max_positions"]))
+
     @property
     def architecture(self):
         return self.raw["architecture"]
