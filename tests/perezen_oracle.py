@@ -82,6 +82,10 @@ def differential_attention(h, w, m, eps, keys_values, operand=exact):
     return operand(np.concatenate(heads, -1) * sigmoid(h @ w["g"].T)) @ w["o"].T
 
 
+def mlstm_denominator(nq, m):
+    return max(abs(nq), np.exp(-m)) + 1e-6
+
+
 def mlstm_recurrence(q, k, v, log_i, log_f):
     """One head, token by token: q, k [tokens, dim], v [tokens, vdim], log gates [tokens] -> [tokens, vdim]."""
     S, n, m = np.zeros((k.shape[1], v.shape[1])), np.zeros(k.shape[1]), 0.0
@@ -90,7 +94,7 @@ def mlstm_recurrence(q, k, v, log_i, log_f):
         top = max(log_f[t] + m, log_i[t])
         keep, add = np.exp(log_f[t] + m - top), np.exp(log_i[t] - top)
         S, n, m = keep * S + add * np.outer(k[t], v[t]), keep * n + add * k[t], top
-        out[t] = (S.T @ q[t]) / (max(abs(n @ q[t]), np.exp(-m)) + 1e-6)
+        out[t] = (S.T @ q[t]) / mlstm_denominator(n @ q[t], m)
     return out
 
 

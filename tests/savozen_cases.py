@@ -1,13 +1,7 @@
 """Small Savozen configurations with random weights for the tests (nothing of a published model)."""
-import json
-import struct
-
 import numpy as np
 
-
-def bf16_round(a):
-    u = np.ascontiguousarray(a, dtype=np.float32).view(np.uint32)
-    return (((u + 0x7FFF + ((u >> 16) & 1)) >> 16) << 16).astype(np.uint32).view(np.float32).reshape(np.shape(a))
+from stack_common import bf16_round, tokens, write_folder  # noqa: F401
 
 
 def mixer(heads=3, dim=24, rot_dim=16, vdim=40, kv_rank=56, scale=0.4, base=10000.0):
@@ -68,25 +62,6 @@ def weights(cfg, seed, sharp=3.0):
             mat(p + "side.proj", D, side["dim"])
             w[p + "side.norm"] = bf16_round(0.5 + 0.2 * rng.standard_normal(D))
     return w
-
-
-def tokens(cfg, n, seed):
-    return np.random.default_rng(seed).integers(0, cfg["vocab"], n).astype(np.int32)
-
-
-def write_folder(path, cfg, w):
-    """config.json and model.safetensors (bf16) in folder `path`."""
-    with open(path / "config.json", "w") as f:
-        json.dump(cfg, f)
-    head, blobs, at = {}, [], 0
-    for name, a in w.items():
-        b = (np.ascontiguousarray(a, dtype=np.float32).view(np.uint32) >> 16).astype("<u2").tobytes()
-        head[name] = dict(dtype="BF16", shape=list(np.shape(a)), data_offsets=[at, at + len(b)])
-        blobs.append(b)
-        at += len(b)
-    h = json.dumps(head).encode()
-    with open(path / "model.safetensors", "wb") as f:
-        f.write(struct.pack("<Q", len(h)) + h + b"".join(blobs))
 
 
 M = mixer

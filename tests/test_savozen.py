@@ -10,42 +10,15 @@ import pytest
 
 import savozen_cases as sc
 import savozen_oracle as so
+from stack_common import COMPUTE, bf16, build, check, err, feed
 
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
-LIMIT32 = 3e-5  # of the logits' root mean square
-COMPUTE = ["float32", "bfloat16"]
-
-
-def err(got, want):
-    """Per position: rms over the vocabulary of the difference (mean taken off), relative to the rms of the expected logits."""
-    d = np.asarray(got, np.float64) - want
-    d -= d.mean(-1, keepdims=True)
-    return np.sqrt((d * d).mean(-1)) / np.sqrt((want * want).mean())
-
-
-def bf16(x):
-    return sc.bf16_round(x).astype(np.float64)
 
 
 def expected(cfg, w, toks):
     """(exact logits, error of every position when operands are rounded to bf16)."""
     want = so.forward(cfg, w, toks)
     return want, err(so.forward(cfg, w, toks, operand=bf16), want)
-
-
-def check(got, want, compute, rows=slice(None)):
-    """32-bit: within LIMIT32 everywhere.  16-bit: no more than a few times what rounding the operands alone costs, in the median and
-    at the worst position."""
-    want, rounding = want
-    e = err(got, want[rows])
-    assert np.isfinite(e).all()
-    worst = (compute, int(e.argmax()), float(e.max()), float(np.median(e)), None if rounding is None else (float(rounding.max()), float(np.median(rounding))))
-    if compute == "float32":
-        assert e.max() <= LIMIT32, worst
-    else:
-        assert e.max() <= 3 * rounding.max(), worst
-        if e.size > 20:
-            assert np.median(e) <= 2 * np.median(rounding), worst
 
 
 # ---- CPU -------------------------------------------------------------------------------------------
@@ -136,20 +109,6 @@ def test_trace_run_says_what_it_takes():
 
 
 # ---- GPU -------------------------------------------------------------------------------------------
-def build(pkg, cfg, w, seq_len, compute):
-    return pkg.LanguageModel(pkg.StackConfig(cfg, seq_len, compute), None, pkg.StackWeights(w))
-
-
-def feed(pkg, state, toks, sizes):
-    """The tokens in portions of the given sizes (the last one repeated); logits of every position."""
-    out, at, i = [], 0, 0
-    while at < len(toks):
-        n = min(sizes[min(i, len(sizes) - 1)], len(toks) - at)
-        out.append(pkg.extend(state, toks[at:at + n], at, range(n)))
-        at, i = at + n, i + 1
-    return np.concatenate(out)
-
-
 @pytest.mark.gpu
 @pytest.mark.parametrize("compute", COMPUTE)
 @pytest.mark.parametrize("case", list(sc.CASES))
