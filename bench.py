@@ -17,7 +17,7 @@ What the printed line says:
 On N > 1 GPUs every rank runs an independent replica of the 8B shape (it fits one GPU and has no exchange step), `value` is
 the sum over ranks, and the key `tp_70b` carries the Llama-2-70B shape run tensor-parallel over the same N GPUs.
 
-    python bench.py [--gpus N] [--steps K] [--warmup W] [--impl ours|reference] [--workload 8b|tiny|phi3|70b-tp|matvec-q4k|savozen|...]
+    python bench.py [--gpus N] [--steps K] [--warmup W] [--impl ours|reference] [--workload 8b|tiny|phi3|70b-tp|matvec-q4k|savozen|perezen|...]
 """
 import argparse
 import ctypes as C
@@ -307,9 +307,10 @@ def run_tp_70b(args, pkg, synth, L, torch, dist, world, rank, local, steps, posi
     return out, [int(x) for x in toks]
 
 
-def run_savozen(args):
-    """Prefill and decode of the Savozen design at the layer sizes of synth.SAVOZEN_SIZES (random weights, reduced depth), each beside
-    the llama shape of equal width, feed-forward, head count and depth in q4_K.  One line per size."""
+def run_stack(args):
+    """Prefill and decode of a layer-stack design at the sizes of synth (random weights, reduced depth), each beside the closest other
+    model of equal size: Savozen beside the llama shape of equal width, feed-forward, head count and depth in q4_K, Perezen beside
+    Savozen's layers.  One line per size."""
     import torch
     import __graft_entry__ as g
     pkg = g.load_package()
@@ -321,6 +322,12 @@ def run_savozen(args):
             tflops = float(json.load(f)["bf16_tflops"])
     except Exception:
         tflops = 1590.0
+    designs = {
+        "savozen": dict(raw=lambda n: synth.SAVOZEN_SIZES[n]["raw"], weights=synth.savozen_weights, flops=synth.savozen_flops_per_token, cache=synth.savozen_cache_bytes,
+                        dtype="bf16 weights and latent cache, f32 elsewhere"),
+        "perezen": dict(raw=lambda n: synth.PEREZEN_SIZES[n], weights=synth.perezen_weights, flops=synth.perezen_flops_per_token, cache=synth.perezen_cache_bytes,
+                        dtype="bf16 weights and keys / values, f32 elsewhere (states included)"),
+    }
 
     def timed(model, prompt, n_pos):
         for _ in range(args.warmup):
@@ -331,10 +338,23 @@ def run_savozen(args):
             a, b = model.last_phase_ms()
             pm, dm = pm + a, dm + b
         return pm / args.steps, dm / args.steps, model.last_launches()
-    for name, size in synth.SAVOZEN_SIZES.items():
+
+    def measure(design, raw, prompt, n_prompt, n_pos):
+        d, n_dec = designs[design], max(n_pos - n_prompt, 1)
+        model = pkg.LanguageModel(pkg.StackConfig(raw, 2048), None, d["weights"](raw, 5))
+        wbytes, kpt = model.weight_bytes_per_token(), model.kernels_per_token()
+        pm, dm, launches = timed(model, prompt[:n_pos], n_pos)
+        model.close()
+        nbytes = wbytes + d["cache"](raw, n_prompt + n_dec / 2)
+        flops = sum(d["flops"](raw, n_prompt / 2)) * n_prompt
+        return dict(pm=pm, dm=dm, launches=launches, kernels=kpt, bytes=int(nbytes), decode=round(n_dec / dm * 1e3, 1), gbs=round(nbytes * n_dec / dm / 1e6, 1),
+                    hbm=round(nbytes * n_dec / dm / 1e6 / peak, 4), us=round(dm * 1e3 / n_dec, 2), prefill=round(n_prompt / pm * 1e3, 1),
+                    tflops=round(flops / pm / 1e9, 1), bf16=round(flops / pm / 1e9 / tflops, 4))
+
+    for name in ("2k", "4k"):
         if args.size and name != args.size:
             continue
-        raw, ll = json.loads(json.dumps(size["raw"])), size["llama"]
+        raw = json.loads(json.dumps(designs[args.workload]["raw"](name)))
         if args.layers:
             raw["layers"] = raw["layers"][:args.layers]
         n_layers, n_prompt = len(raw["layers"]), args.prompt_len or 1024
@@ -342,26 +362,24 @@ def run_savozen(args):
         prompt = synth.tokens(n_prompt, 77, 0, raw["vocab"])
         sampler = ClockSampler(0)
         sampler.start()
-        model = pkg.LanguageModel(pkg.StackConfig(raw, 2048), None, synth.savozen_weights(raw, 5))
-        wbytes, kpt = model.weight_bytes_per_token(), model.kernels_per_token()
-        pm, dm, launches = timed(model, prompt[:n_pos], n_pos)
-        model.close()
-        n_dec = max(n_pos - n_prompt, 1)
-        m = raw["layers"][0]["mixer"]
-        cache = 2 * (m["kv_rank"] + m["rot_dim"]) * n_layers * (n_prompt + n_dec / 2)  # bf16 rows read per position, on average
-        dense, att = synth.savozen_flops_per_token(raw, n_prompt / 2)
-        achieved = (wbytes + cache) * n_dec / dm / 1e6
-        line = {"metric": "Savozen layers, prefill and decode tok/s", "value": round(n_dec / dm * 1e3, 1), "unit": "decode tok/s", "n_gpus": 1, "steps": args.steps,
-                "warmup": args.warmup, "ms_per_step": round(pm + dm, 4), "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
-                "dtype": "bf16 weights and latent cache, f32 elsewhere", "data": "synthetic (seeded random weights and token ids)",
-                "config": {"workload": f"savozen-{name}: width {raw['width']}, ff {raw['layers'][0]['mlp']['ff']}, {m['heads']} heads, {n_layers} layers, vocab {raw['vocab']}, "
+        r = measure(args.workload, raw, prompt, n_prompt, n_pos)
+        n_dec, m = max(n_pos - n_prompt, 1), raw["layers"][0]["mixer"]
+        line = {"metric": f"{raw['architecture']} layers, prefill and decode tok/s", "value": r["decode"], "unit": "decode tok/s", "n_gpus": 1, "steps": args.steps,
+                "warmup": args.warmup, "ms_per_step": round(r["pm"] + r["dm"], 4), "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+                "dtype": designs[args.workload]["dtype"], "data": "synthetic (seeded random weights and token ids)",
+                "config": {"workload": f"{args.workload}-{name}: width {raw['width']}, ff {raw['layers'][0]['mlp']['ff']}, {m['heads']} heads, {n_layers} layers, vocab {raw['vocab']}, "
                                        f"{n_prompt} prompt ids + {n_dec} greedy tokens, batch 1", "l2": "inputs larger than L2 (the weights streamed per position)"},
-                "prefill": {"value": round(n_prompt / pm * 1e3, 1), "unit": "tok/s", "ms": round(pm, 3), "tflops": round((dense + att) * n_prompt / pm / 1e9, 1),
-                            "frac_of_measured_bf16": round((dense + att) * n_prompt / pm / 1e9 / tflops, 4)},
-                "us_per_decode_token": round(dm * 1e3 / n_dec, 2), "kernels_per_token": kpt, "gpu_launches": launches * args.steps,
-                "roofline": {"bound": "hbm", "achieved": round(achieved, 1), "peak": peak, "unit": "GB/s", "frac": round(achieved / peak, 4), "peak_kind": kind,
-                             "bytes_per_position": int(wbytes + cache)}}
-        if not args.no_closest:
+                "prefill": {"value": r["prefill"], "unit": "tok/s", "ms": round(r["pm"], 3), "tflops": r["tflops"], "frac_of_measured_bf16": r["bf16"]},
+                "us_per_decode_token": r["us"], "kernels_per_token": r["kernels"], "gpu_launches": r["launches"] * args.steps,
+                "roofline": {"bound": "hbm", "achieved": r["gbs"], "peak": peak, "unit": "GB/s", "frac": r["hbm"], "peak_kind": kind, "bytes_per_position": r["bytes"]}}
+        if not args.no_closest and args.workload == "perezen":
+            sraw = json.loads(json.dumps(designs["savozen"]["raw"](name)))
+            sraw["layers"] = sraw["layers"][:n_layers]
+            o = measure("savozen", sraw, prompt, n_prompt, n_pos)
+            line["closest_model"] = {"workload": "Savozen layers of equal width, ff, heads and depth, bf16", "decode_tok_s": o["decode"], "us_per_decode_token": o["us"], "hbm_frac": o["hbm"],
+                                     "achieved_gbs": o["gbs"], "prefill_tok_s": o["prefill"], "prefill_tflops": o["tflops"], "prefill_frac_of_measured_bf16": o["bf16"]}
+        elif not args.no_closest:
+            ll = synth.SAVOZEN_SIZES[name]["llama"]
             spec = synth.scaled(dict(config=ll, types=synth.ALL(synth.Q4), tied=False), n_layers=n_layers)
             cfg = spec["config"]
             other = pkg.LanguageModel(cfg, None, synth.model_weights(cfg, spec["types"], seed=6, distinct_layers=1))
@@ -382,8 +400,8 @@ def run_savozen(args):
 def run_ours(args):
     if args.workload.startswith("matvec"):
         return run_matvec(args)
-    if args.workload == "savozen":
-        return run_savozen(args)
+    if args.workload in ("savozen", "perezen"):
+        return run_stack(args)
     import torch
     import torch.distributed as dist
     import __graft_entry__ as g
@@ -628,7 +646,7 @@ def main():
     ap.add_argument("--steps", type=int, default=3)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="8b", choices=["8b", "tiny", "phi3", "70b-tp", "matvec-q4k", "matvec-q5k", "matvec-q6k", "savozen"])
+    ap.add_argument("--workload", default="8b", choices=["8b", "tiny", "phi3", "70b-tp", "matvec-q4k", "matvec-q5k", "matvec-q6k", "savozen", "perezen"])
     ap.add_argument("--layers", type=int, default=0, help="run the workload's shape with this many layers (0 = all)")
     ap.add_argument("--matvec-in", type=int, default=4096)
     ap.add_argument("--matvec-out", type=int, default=14336)
@@ -640,8 +658,8 @@ def main():
     ap.add_argument("--no-cpu-baseline", action="store_true", help="skip the oracle run (parity and cpu_baseline keys)")
     ap.add_argument("--no-tp", action="store_true", help="skip the 70B-shape leg (one GPU: the base figure; several: the tensor-parallel run)")
     ap.add_argument("--tp-positions", type=int, default=576, help="positions of the tensor-parallel 70B leg (512 prompt ids, then decode)")
-    ap.add_argument("--size", default="", help="savozen workload: only this size (2k or 4k)")
-    ap.add_argument("--no-closest", action="store_true", help="savozen workload: skip the llama shape of equal size")
+    ap.add_argument("--size", default="", help="savozen and perezen workloads: only this size (2k or 4k)")
+    ap.add_argument("--no-closest", action="store_true", help="savozen and perezen workloads: skip the other model of equal size")
     ap.add_argument("--positions", type=int, default=0, help="run only this many positions per step (for profiler captures)")
     args = ap.parse_args()
     args.warmup = max(args.warmup, 3) if args.impl == "ours" else args.warmup

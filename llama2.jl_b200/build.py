@@ -12,7 +12,7 @@ HEADERS = ["csrc/common.cuh", "csrc/kquants.cuh", "csrc/fused_matvec.cuh", "csrc
            "csrc/small_ops.cuh", "csrc/token_kernel.cuh", "csrc/kq_gemm.cuh", "csrc/prefill_ops.cuh", "csrc/gguf_reader.h", "csrc/host_common.h",
            "csrc/tcgen05.cuh", "csrc/json.h", "csrc/safetensors.h", "csrc/stack_config.h", "csrc/stack.h", "csrc/dense_ops.cuh",
            "csrc/dense_matvec.cuh", "csrc/dense_gemm.cuh", "csrc/stack_rows.cuh", "csrc/cache_scan.cuh", "csrc/latent_attention.cuh",
-           "csrc/head_attention.cuh", "csrc/mlstm.cuh", "csrc/latent_prefill.cuh",
+           "csrc/head_attention.cuh", "csrc/head_prefill.cuh", "csrc/mlstm.cuh", "csrc/mlstm_prefill.cuh", "csrc/latent_prefill.cuh",
            "../include/llama2_b200.h"]
 OUTPUT = os.path.join(_HERE, "libllama2_b200.so")
 SYNTH_OUTPUT = os.path.join(_HERE, "libl2b_synth.so")  # test support: seeded synthetic data, plain C++

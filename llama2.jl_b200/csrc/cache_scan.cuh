@@ -60,15 +60,6 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], 
 __device__ __forceinline__ void ldmatrix4_trans(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
-// x = hi + lo with both bf16: two values -> two packed words
-__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-    const float2 f = __bfloat1622float2(h);
-    const __nv_bfloat162 l = __floats2bfloat162_rn(x - f.x, y - f.y);
-    hi = *reinterpret_cast<const uint32_t*>(&h);
-    lo = *reinterpret_cast<const uint32_t*>(&l);
-}
-
 // Grid (nsplit * blocks of 16 heads, rows).  N: K = 16 steps of a cache row, and pairs of 8-column tiles of the summed columns, per warp at most.
 template <int N>
 __global__ void __launch_bounds__(CS_SCAN_THREADS) cache_scan_mma_kernel(const __grid_constant__ CacheScan p) {

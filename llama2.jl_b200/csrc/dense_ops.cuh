@@ -215,6 +215,16 @@ __device__ __forceinline__ float fast_exp2(float x) {
     return r;
 }
 
+__device__ __forceinline__ uint32_t pack_bf16(float x, float y) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
+    return *reinterpret_cast<const uint32_t*>(&h);
+}
+// x = hi + lo with both bf16: two values -> two packed words
+__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
+    hi = pack_bf16(x, y);
+    lo = pack_bf16(x - __uint_as_float(hi << 16), y - __uint_as_float(hi & 0xFFFF0000u));
+}
+
 // Sum over the first NW warps of a block; each of their threads gets it.  s holds NW floats and may be reused after the next barrier.
 template <int NW>
 __device__ __forceinline__ float block_sum_all(float v, float* s) {

@@ -9,10 +9,10 @@
 
 #include "dense_gemm.cuh"
 #include "dense_matvec.cuh"
-#include "head_attention.cuh"
+#include "head_prefill.cuh"
 #include "latent_attention.cuh"
 #include "latent_prefill.cuh"
-#include "mlstm.cuh"
+#include "mlstm_prefill.cuh"
 #include "stack_rows.cuh"
 
 using namespace l2b;
@@ -404,15 +404,18 @@ struct StackSession {
     // many positions
     float *xr = nullptr, *in = nullptr, *y = nullptr;
     void *act = nullptr, *act2 = nullptr;        // operands of the products, [max_rows][k rounded up to 8]
-    bf16 *pq = nullptr, *pk = nullptr, *pv = nullptr;  // expanded attention: queries, keys, transposed values
+    bf16 *pq = nullptr, *pk = nullptr, *pv = nullptr;  // prompt attention: queries; latent attention: expanded keys, transposed values
     int pv_ld = 0;
+    float* aside = nullptr;                      // differential attention with many value dimensions: the first map's result
+    MlstmPrefillParams mp = {};                  // mLSTM in chunks: buffers (q null: there are none)
 };
 
 static size_t act_bytes(const StackModel* m) { return m->f32 ? 4 : 2; }
 
 constexpr int ABSORB_ROWS = 64;  // rows per pass of the absorbed form of the attention (bounds its scratch)
-// The expanded form of the attention (latent_prefill.cuh) is for portions of at least this many rows.
-constexpr int EXPAND_MIN_ROWS = 48;
+// The tiled forms of the attention (latent_prefill.cuh, head_prefill.cuh) and the chunked form of the recurrence (mlstm_prefill.cuh)
+// are for portions of at least this many rows.
+constexpr int EXPAND_MIN_ROWS = 48, MLSTM_MIN_ROWS = 32;
 
 // Blocks of query vectors and ranges of positions of the scan kernel: about one block per SM in a decode step, two for several rows.
 static int scan_blocks(const CacheScan& c, bool f32) {
@@ -427,6 +430,20 @@ static int prefill_kstages(const LatentShape& s, const DeviceInfo& di) {
     if (s.vp > 256) return 0;
     for (int k = 2; k >= 1; --k)
         if (lp_smem_layout(s.dim, s.rot, s.vp, k).total + 1024 <= di.max_smem_optin - 1024) return k;
+    return 0;
+}
+
+static int head_prefill_kstages(const HeadShape& s, const DeviceInfo& di) {
+    const int vn = up(s.vdim, 16);
+    if (vn > 256 || !(s.scale2 > 0.f)) return 0;
+    for (int k = 2; k >= 1; --k)
+        if (hp_smem_layout(s.dim, vn, k).total + 1024 <= di.max_smem_optin - 4096) return k;
+    return 0;
+}
+// Ring slots of the chunk kernel (0: the heads do not fit the chunked form).
+static int mlstm_prefill_stages(const MlstmShape& s, const DeviceInfo& di) {
+    for (int k = 2; k >= 1; --k)
+        if (mc_smem_layout(up(s.dim, 16), k).total + 1024 <= di.max_smem_optin - 8192) return k;
     return 0;
 }
 
@@ -445,6 +462,9 @@ static int32_t set_stack_kernel_attrs() {
         };
         set((const void*)dense_matvec_kernel);
         set((const void*)latent_prefill_kernel);
+        set((const void*)head_prefill_kernel);
+        set((const void*)mlstm_state_kernel);
+        set((const void*)mlstm_chunk_kernel);
         set((const void*)bf16_gemm_kernel<32, 1>); set((const void*)bf16_gemm_kernel<32, 2>);
         set((const void*)bf16_gemm_kernel<64, 1>); set((const void*)bf16_gemm_kernel<64, 2>);
         set((const void*)bf16_gemm_kernel<128, 1>); set((const void*)bf16_gemm_kernel<128, 2>);
@@ -492,12 +512,23 @@ int32_t stack_session_create(const StackModel* m, const StackSessionInfo& info, 
     s->di = di;
     const StackConfig& c = m->cfg;
     int max_in = 1, max_k = c.width, max_k2 = 1;
-    size_t pq = 0, pk = 0, pv = 0;
+    size_t pq = 0, pk = 0, pv = 0, aside = 0, mh = 0, mk = 0, mv = 0, ms = 0;
     s->pv_ld = up(info.seq_len, 8);
     for (size_t i = 0; i < m->layers.size(); ++i) {
         const StackLayerW& w = m->layers[i];
         max_in = std::max(max_in, w.in.rows);
         max_k2 = std::max(std::max(max_k2, w.o.k), std::max(w.down.k, w.side_proj.k));
+        if (w.head.heads && head_prefill_kstages(w.head, di)) {
+            pq = std::max(pq, (size_t)2 * w.head.heads * up(w.head.dim, 16));
+            if (up(w.head.vdim, 16) > HP_OWN_COLS) aside = std::max(aside, (size_t)w.head.heads * w.head.vdim);
+        }
+        if (w.mlstm.heads && mlstm_prefill_stages(w.mlstm, di)) {
+            const MlstmShape& sh = w.mlstm;
+            mh = std::max(mh, (size_t)sh.heads);
+            mk = std::max(mk, (size_t)sh.heads * up(sh.dim, 16));
+            mv = std::max(mv, (size_t)sh.heads * up(sh.vdim, 8));
+            ms = std::max(ms, (size_t)sh.heads * up(sh.dim, 16) * up(sh.vdim, 8));
+        }
         if (c.layers[i].mix.kind != MixerKind::LatentAttention) continue;
         pq = std::max(pq, (size_t)w.latent.heads * (w.latent.dp + up(w.latent.rot, 16)));
         pk = std::max(pk, (size_t)w.latent.heads * w.latent.dp);
@@ -548,8 +579,19 @@ int32_t stack_session_create(const StackModel* m, const StackSessionInfo& info, 
     L2B_TRY(alloc(s->act2, T * up(max_k2, 8) * act_bytes(m)));
     if (!m->f32 && info.n_seq == 1 && info.max_rows >= EXPAND_MIN_ROWS && pq) {
         L2B_TRY(alloc(s->pq, T * pq * 2));
-        L2B_TRY(alloc(s->pk, (size_t)info.seq_len * pk * 2));
-        L2B_TRY(alloc(s->pv, pv * s->pv_ld * 2));
+        if (pk) L2B_TRY(alloc(s->pk, (size_t)info.seq_len * pk * 2));
+        if (pv) L2B_TRY(alloc(s->pv, pv * s->pv_ld * 2));
+        if (aside) L2B_TRY(alloc(s->aside, T * aside * 4));
+    }
+    const size_t nchunk = (T + MP_L - 1) / MP_L;
+    if (!m->f32 && info.n_seq == 1 && info.max_rows >= MLSTM_MIN_ROWS && mh && nchunk <= MP_MAX_CHUNKS) {
+        MlstmPrefillParams& p = s->mp;
+        for (bf16** b : {&p.q, &p.k}) L2B_TRY(alloc(*b, T * mk * 2));
+        L2B_TRY(alloc(p.v, T * mv * 2));
+        for (float** f : {&p.a, &p.mx, &p.w, &p.floor, &p.u}) L2B_TRY(alloc(*f, mh * nchunk * MP_L * 4));
+        L2B_TRY(alloc(p.decay, mh * nchunk * 4));
+        for (bf16** b : {&p.sh, &p.sl}) L2B_TRY(alloc(*b, nchunk * ms * 2));
+        L2B_TRY(alloc(p.sn, nchunk * mk * 4));
     }
     CU(cudaStreamSynchronize(st));
     CU(cudaDeviceSynchronize());
@@ -827,12 +869,14 @@ int32_t stack_enqueue_token(StackSession* s, const int* token, const int* pos, f
 }
 
 // ---- many positions ----------------------------------------------------------------------------
-static int32_t bf16_map(CUtensorMap& map, const bf16* base, int64_t inner, int64_t rows, int64_t stride_elems, int box_rows) {
+// A tile of 64 values x box_rows rows; depth > 1: of one of `depth` matrices (the tile does not reach into the next one).
+static int32_t bf16_map(CUtensorMap& map, const bf16* base, int64_t inner, int64_t rows, int64_t stride_elems, int box_rows, int64_t depth = 1, int64_t depth_stride = 0) {
     EncodeTiledFn enc = encode_tiled_fn();
     if (!enc) return fail(L2B_ERR_CUDA, "cuTensorMapEncodeTiled is not available from this driver");
-    const cuuint64_t dims[2] = {(cuuint64_t)inner, (cuuint64_t)rows}, strides[1] = {(cuuint64_t)stride_elems * 2};
-    const cuuint32_t box[2] = {64u, (cuuint32_t)box_rows}, estr[2] = {1u, 1u};
-    const CUresult r = enc(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<bf16*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+    const int rank = depth_stride ? 3 : 2;
+    const cuuint64_t dims[3] = {(cuuint64_t)inner, (cuuint64_t)rows, (cuuint64_t)depth}, strides[2] = {(cuuint64_t)stride_elems * 2, (cuuint64_t)depth_stride * 2};
+    const cuuint32_t box[3] = {64u, (cuuint32_t)box_rows, 1u}, estr[3] = {1u, 1u, 1u};
+    const CUresult r = enc(&map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, rank, const_cast<bf16*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
                            CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     if (r != CUDA_SUCCESS) return fail(L2B_ERR_CUDA, "cuTensorMapEncodeTiled failed with code " + std::to_string((int)r));
     return L2B_OK;
@@ -951,7 +995,8 @@ static int32_t enqueue_latent_rows(StackSession* s, int run, int n, int pos0, co
     return L2B_OK;
 }
 
-// Differential attention of n rows.  Result (gated) in act2 [n][ldo].
+// Differential attention of n rows: the tiled form (long portions of one sequence, bf16), or the scan over rows.  Result (gated) in
+// act2 [n][ldo].
 static int32_t enqueue_head_rows(StackSession* s, int run, int n, int pos0, const int* pos_list, int ldo, int* status, cudaStream_t st, long long* launches) {
     const StackModel* m = s->m;
     HeadAttnParams a = head_params(s, run, s->in);
@@ -961,15 +1006,33 @@ static int32_t enqueue_head_rows(StackSession* s, int run, int n, int pos0, cons
     a.c.status = status;
     a.out = s->act2;
     a.ldo = ldo;
-    return rows_in_parts(s, a, n, [&](HeadAttnParams& b, int r, int k) {
-        b.in += (size_t)r * a.ld;
-        *launches += 3;
-        return m->f32 ? (launch_head_attention<float, float>(b, k, false, s->di, st)) : (launch_head_attention<bf16, bf16>(b, k, false, s->di, st));
-    });
+    const HeadShape& sh = a.s;
+    const int kstages = head_prefill_kstages(sh, s->di);
+    if (!s->pq || pos_list || n < EXPAND_MIN_ROWS || kstages == 0)
+        return rows_in_parts(s, a, n, [&](HeadAttnParams& b, int r, int k) {
+            b.in += (size_t)r * a.ld;
+            *launches += 3;
+            return m->f32 ? (launch_head_attention<float, float>(b, k, false, s->di, st)) : (launch_head_attention<bf16, bf16>(b, k, false, s->di, st));
+        });
+    a.pq = s->pq;
+    a.dq = up(sh.dim, 16);
+    CU(launch_head_rows<bf16>(a, n, false, st));
+    HeadPrefillParams f;
+    memset(&f, 0, sizeof(f));
+    f.s = sh; f.n = n; f.pos0 = pos0; f.chunk = a.c.chunk; f.dq = a.dq; f.vn = up(sh.vdim, 16); f.kstages = kstages;
+    f.gate = a.in + a.off_g; f.ld = a.ld; f.aside = s->aside; f.out = static_cast<bf16*>(s->act2); f.ldo = ldo; f.status = status;
+    CUtensorMap mq, mkv;
+    L2B_TRY(bf16_map(mq, s->pq, (int64_t)2 * sh.heads * a.dq, n, (int64_t)2 * sh.heads * a.dq, HP_TILE));
+    L2B_TRY(bf16_map(mkv, static_cast<const bf16*>(a.c.cache), sh.row, pos0 + n, sh.row, HP_TILE, sh.kv_heads, (int64_t)a.c.group_stride));
+    const size_t smem = (size_t)hp_smem_layout(sh.dim, f.vn, kstages).total + 1024;
+    CU(launch_kernel_args(head_prefill_kernel, dim3((n + HP_TILE - 1) / HP_TILE, sh.heads), dim3(HP_THREADS), smem, st, false, 1, f, mq, mkv));
+    *launches += 2;
+    return L2B_OK;
 }
 
-// mLSTM of n rows: n tokens of one sequence, or one of every sequence.  Result (gated) in act2 [n][ldo].
-static int32_t enqueue_mlstm_rows(StackSession* s, int run, int n, int pos0, const int* pos_list, int ldo, cudaStream_t st, long long* launches) {
+// mLSTM of n rows: n tokens of one sequence (in chunks, when there are many; bf16), or one of every sequence.  Result (gated) in act2
+// [n][ldo].
+static int32_t enqueue_mlstm_rows(StackSession* s, int run, int n, int pos0, const int* pos_list, int ldo, int* status, cudaStream_t st, long long* launches) {
     const StackModel* m = s->m;
     MlstmParams a = mlstm_params(s, run, s->in);
     a.pos0 = pos0;
@@ -978,6 +1041,35 @@ static int32_t enqueue_mlstm_rows(StackSession* s, int run, int n, int pos0, con
     a.tokens = pos_list ? 1 : n;
     a.out = s->act2;
     a.ldo = ldo;
+    const MlstmShape& sh = a.s;
+    const int stages = mlstm_prefill_stages(sh, s->di);
+    if (s->mp.q && !pos_list && n >= MLSTM_MIN_ROWS && stages) {
+        MlstmPrefillParams p = s->mp;
+        p.m = a;
+        p.n = n;
+        p.nchunk = (n + MP_L - 1) / MP_L;
+        p.dp = up(sh.dim, 16);
+        p.vp = p.vs = up(sh.vdim, 8);
+        p.sstages = stages;
+        p.status = status;
+        for (p.vt = 1; p.vt * MP_COLS < sh.vdim;) p.vt *= 2;
+        CUtensorMap mq, mk, mv, msh, msl;
+        const int64_t nk = (int64_t)sh.heads * p.dp, nv = (int64_t)sh.heads * p.vp, rows = (int64_t)p.nchunk * sh.heads * p.dp;
+        L2B_TRY(bf16_map(mq, p.q, nk, n, nk, MP_L));
+        L2B_TRY(bf16_map(mk, p.k, nk, n, nk, MP_L));
+        L2B_TRY(bf16_map(mv, p.v, nv, n, nv, MP_L));
+        L2B_TRY(bf16_map(msh, p.sh, p.vs, rows, p.vs, 64));
+        L2B_TRY(bf16_map(msl, p.sl, p.vs, rows, p.vs, 64));
+        mlstm_operands_kernel<<<n, 256, 0, st>>>(p);
+        CU(cudaGetLastError());
+        mlstm_gates_kernel<<<sh.heads, 32 * p.nchunk, 0, st>>>(p);
+        CU(cudaGetLastError());
+        const dim3 sgrid((sh.vdim + MP_STATE_COLS - 1) / MP_STATE_COLS, (sh.dim + 127) / 128, sh.heads), cgrid(p.vt, p.nchunk, sh.heads);
+        CU(launch_kernel_args(mlstm_state_kernel, sgrid, dim3(MP_THREADS), (size_t)MsSmem::total + 1024, st, false, 1, p, mk));
+        CU(launch_kernel_args(mlstm_chunk_kernel, cgrid, dim3(MP_THREADS), (size_t)mc_smem_layout(p.dp, stages).total + 1024, st, false, p.vt, p, mq, mk, mv, msh, msl));
+        *launches += 4;
+        return L2B_OK;
+    }
     const int rows = pos_list ? n : 1;
     CU(m->f32 ? launch_mlstm_step<float>(a, rows, false, st) : launch_mlstm_step<bf16>(a, rows, false, st));
     ++*launches;
@@ -1039,7 +1131,7 @@ int32_t stack_enqueue_rows(StackSession* s, const int* dev_tokens, int n, int po
         switch (c.layers[l].mix.kind) {
             case MixerKind::LatentAttention: L2B_TRY(enqueue_latent_rows(s, (int)r, n, pos0, pos_list, up(w.o.k, 8), status, st, &count)); break;
             case MixerKind::DifferentialAttention: L2B_TRY(enqueue_head_rows(s, (int)r, n, pos0, pos_list, up(w.o.k, 8), status, st, &count)); break;
-            case MixerKind::Mlstm: L2B_TRY(enqueue_mlstm_rows(s, (int)r, n, pos0, pos_list, up(w.o.k, 8), st, &count)); break;
+            case MixerKind::Mlstm: L2B_TRY(enqueue_mlstm_rows(s, (int)r, n, pos0, pos_list, up(w.o.k, 8), status, st, &count)); break;
         }
         L2B_TRY(result(w.o, w.norm1b));
         if (w.gu.w) {

@@ -90,9 +90,33 @@ __device__ __forceinline__ uint64_t umma_desc_sw128(const void* smem_ptr, uint32
     d |= (uint64_t)2 << 61;                     // layout type: 128-byte swizzle
     return d;
 }
-// Instruction descriptor: f32 accumulators, A and B bf16, both K-major.
-__host__ __device__ constexpr uint32_t umma_idesc_bf16(int M, int N) {
-    return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(N >> 3) << 17) | ((uint32_t)(M >> 4) << 24);
+// The same for an operand whose rows run along K: tiles of 64 bf16 (128 bytes) of M or N per K row, 128-byte swizzle as TMA writes it;
+// groups of 8 K rows are 1024 bytes apart, the next 64 of M or N `piece` bytes further.  16 K rows are 2048 bytes.
+__device__ __forceinline__ uint64_t umma_desc_sw128_mn(const void* smem_ptr, uint32_t k_bytes, uint32_t piece) {
+    uint64_t d = 0;
+    d |= (uint64_t)(((smem_u32(smem_ptr) + k_bytes) >> 4) & 0x3FFFu);
+    d |= (uint64_t)((piece >> 4) & 0x3FFFu) << 16;
+    d |= (uint64_t)(1024u >> 4) << 32;
+    d |= (uint64_t)1 << 46;
+    d |= (uint64_t)2 << 61;
+    return d;
+}
+// Instruction descriptor: f32 accumulators, A and B bf16, each K-major (0) or with rows along K (1).
+__host__ __device__ constexpr uint32_t umma_idesc_bf16(int M, int N, int a_mn = 0, int b_mn = 0) {
+    return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)a_mn << 15) | ((uint32_t)b_mn << 16) | ((uint32_t)(N >> 3) << 17) | ((uint32_t)(M >> 4) << 24);
+}
+// Byte offset of the 16-byte chunk `chunk` (0 .. 7) of a 128-byte row under that swizzle.
+__device__ __forceinline__ int sw128_chunk(int row, int chunk) { return row * 128 + ((chunk ^ (row & 7)) << 4); }
+// One column of this thread's tensor-memory lane: load and store
+__device__ __forceinline__ float tmem_ld1f(uint32_t taddr) {
+    int r;
+    asm volatile("tcgen05.ld.sync.aligned.32x32b.x1.b32 {%0}, [%1];" : "=r"(r) : "r"(taddr) : "memory");
+    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+    return __int_as_float(r);
+}
+__device__ __forceinline__ void tmem_st1f(uint32_t taddr, float v) {
+    asm volatile("tcgen05.st.sync.aligned.32x32b.x1.b32 [%0], {%1};" ::"r"(taddr), "f"(v) : "memory");
+    asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
 }
 // 32 consecutive columns of this thread's tensor-memory lane: load and store
 __device__ __forceinline__ void tmem_ld32f(uint32_t taddr, float (&v)[32]) {

@@ -156,3 +156,86 @@ def savozen_flops_per_token(raw, npos):
         dense += D * (H * (d + r) + R + r + H * dv) + H * (d + dv) * R + H * dv * D + 3 * D * (l["mlp"]["ff"] if l["mlp"] else 0) + 2 * D * side
         att += H * npos * (d + r + dv)
     return 2 * dense, 2 * att
+
+
+def _perezen(width, ff, heads, kv_heads, dim, vdim, mheads, mdim, mvdim, layers, vocab, chunk=8192):
+    """Layers in threes: attention, mLSTM (no feed-forward), attention on the keys and values of the first."""
+    att = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=dim ** -0.5, diff=0.4, rot=dict(base=500000.0, dims=dim), mask=dict(size=chunk))
+    rec = dict(heads=mheads, dim=mdim, vdim=mvdim, gate_cap=15.0)
+    mlp = dict(kind="dense", ff=ff)
+    return dict(architecture="Perezen", norm=dict(eps=1e-5), vocab=vocab, width=width, max_positions=2048, logit_scale=1.0,
+                layers=[dict(type="mlstm", mixer=rec, mlp=None) if i % 3 == 1 else dict(type="attention", mixer=dict(att, kv_from=i - 2) if i % 3 == 2 else att, mlp=mlp)
+                        for i in range(layers)])
+
+
+# Layers of the size of a real model's; each is measured beside the Savozen layers of the same name (equal width, feed-forward and heads).
+PEREZEN_SIZES = {
+    "2k": _perezen(2048, 8192, 16, 4, 64, 128, 4, 256, 512, 8, 32768),
+    "4k": _perezen(4096, 14336, 32, 8, 64, 128, 8, 256, 512, 8, 32768),
+}
+
+
+def perezen_weights(raw, seed):
+    """Weights of a Perezen configuration by tensor name; layers of one size share their host arrays."""
+    D, V, shared = raw["width"], raw["vocab"], {}
+
+    def mat(out, inn):
+        if (out, inn) not in shared:
+            shared[(out, inn)] = bf16_matrix(out, inn, seed + len(shared))
+        return shared[(out, inn)]
+    w = StackWeights({"embed": mat(V, D), "head": mat(V, D), "pos": mat(raw["max_positions"], D), "final.norm": np.ones(D, np.float32)})
+    for i, l in enumerate(raw["layers"]):
+        p, m = f"l{i}.", l["mixer"]
+        H, d, dv = m["heads"], m["dim"], m["vdim"]
+        w[p + "norm1"], w[p + "norm1b"] = np.ones(D, np.float32), np.full(D, 0.5, np.float32)
+        w[p + "mix.g"], w[p + "mix.o"] = mat(H * dv, D), mat(D, H * dv)
+        if l["type"] == "mlstm":
+            w[p + "mix.q"], w[p + "mix.k"], w[p + "mix.v"], w[p + "mix.norm"] = mat(H * d, D), mat(H * d, D), mat(H * dv, D), np.ones(H * dv, np.float32)
+            w[p + "mix.i"], w[p + "mix.f"] = mat(H, D), mat(H, D)
+            w[p + "mix.i.b"], w[p + "mix.f.b"] = np.zeros(H, np.float32), np.linspace(2.0, 8.0, H, dtype=np.float32)
+        else:
+            G = m["kv_heads"]
+            parts = [("q", H * 2 * d)] + ([("k", G * 2 * d), ("v", G * dv)] if m.get("kv_from") is None else [])
+            for n, rows in parts:
+                w[p + "mix." + n], w[p + "mix." + n + ".b"] = mat(rows, D), np.zeros(rows, np.float32)
+                if n != "v":
+                    w[p + "mix." + n + ".norm"] = np.ones(d, np.float32)
+            for n in ("lq1", "lk1", "lq2", "lk2"):
+                w[p + "mix." + n] = normal_f32(d, seed, 0.1)
+        if l["mlp"]:
+            ff = l["mlp"]["ff"]
+            w[p + "norm2"], w[p + "norm2b"] = np.ones(D, np.float32), np.full(D, 0.5, np.float32)
+            w[p + "mlp.gate"], w[p + "mlp.up"], w[p + "mlp.down"] = mat(ff, D), mat(ff, D), mat(D, ff)
+    return w
+
+
+def perezen_flops_per_token(raw, npos):
+    """Multiply-adds x 2 of one prompt token's matrix products, and of its mixers: attention over npos positions (within the chunk), the
+    recurrence's update and read of the state."""
+    D = raw["width"]
+    dense = mix = 0
+    for l in raw["layers"]:
+        m = l["mixer"]
+        H, d, dv = m["heads"], m["dim"], m["vdim"]
+        if l["type"] == "mlstm":
+            dense += D * (H * (2 * d + 2 * dv + 2) + H * dv)
+            mix += 2 * H * d * dv
+        else:
+            G = m["kv_heads"] if m.get("kv_from") is None else 0
+            dense += D * (2 * H * d + G * (2 * d + dv) + 2 * H * dv)
+            mix += 2 * H * min(npos, m["mask"]["size"]) * (d + dv)
+        dense += 3 * D * (l["mlp"]["ff"] if l["mlp"] else 0)
+    return 2 * dense, 2 * mix
+
+
+def perezen_cache_bytes(raw, npos):
+    """Bytes of cache and state a decode step at position npos reads and writes (bf16 rows; f32 states)."""
+    b = 0
+    for l in raw["layers"]:
+        m = l["mixer"]
+        b += 8 * m["heads"] * m["dim"] * m["vdim"] if l["type"] == "mlstm" else 2 * m["kv_heads"] * (2 * m["dim"] + m["vdim"]) * min(npos, m["mask"]["size"])
+    return b
+
+
+def savozen_cache_bytes(raw, npos):
+    return sum(2 * (l["mixer"]["kv_rank"] + l["mixer"]["rot_dim"]) * npos for l in raw["layers"])
