@@ -35,16 +35,98 @@ struct HeadAttnParams {
 
 constexpr int HA_WARPS = 8;
 
-// Element d of a vector of `dim` values at src after its norm (inv = 1 / rms) and the rotation.
-__device__ __forceinline__ float normed_rotated(const float* src, float inv, const float* w, int d, int rdims, const float2* cs) {
-    const float v = __ldcg(src + d) * inv * __ldg(w + d);
-    const int half = rdims >> 1;
-    if (d >= rdims) return v;
-    const bool second = d >= half;
-    const int i = second ? d - half : d, o = second ? i : i + half;
-    const float2 t = __ldg(cs + i);
-    const float u = __ldcg(src + o) * inv * __ldg(w + o);
-    return second ? v * t.x + u * t.y : v * t.x - u * t.y;
+constexpr int HA_REGS = 4;  // values of a vector a lane holds (a longer vector is read again)
+
+// A vector of `dim` values at src after its norm and the rotation, by a warp: lane l makes elements l, l + 32, ...; put_at(d, value) takes
+// them, zeros from dim to `pad` included.
+template <class PutAt>
+__device__ __forceinline__ void normed_rotated(const float* src, const float* w, int dim, int rdims, float eps, const float2* cs, int pad, const PutAt& put_at) {
+    const int lane = threadIdx.x & 31, half = rdims >> 1;
+    float v[HA_REGS];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < HA_REGS; ++i) {
+        v[i] = lane + 32 * i < dim ? __ldcg(src + lane + 32 * i) : 0.f;
+        ss = fmaf(v[i], v[i], ss);
+    }
+    for (int d = lane + 32 * HA_REGS; d < dim; d += 32) {
+        const float x = __ldcg(src + d);
+        ss = fmaf(x, x, ss);
+    }
+    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)dim + eps);
+    auto partner = [&](int d) { return d >= rdims ? d : d >= half ? d - half : d + half; };
+    auto turned = [&](int d, float x, float y) {  // x: element d, y: its partner, both without weight
+        const float a = x * inv * __ldg(w + d);
+        if (d >= rdims) return a;
+        const bool second = d >= half;
+        const float2 t = __ldg(cs + (second ? d - half : d));
+        const float u = y * inv * __ldg(w + partner(d));
+        return second ? a * t.x + u * t.y : a * t.x - u * t.y;
+    };
+#pragma unroll
+    for (int i = 0; i < HA_REGS; ++i) {
+        const int d = lane + 32 * i, o = partner(d);
+        float y = 0.f;
+        if (rdims <= 32 * HA_REGS) {
+#pragma unroll
+            for (int j = 0; j < HA_REGS; ++j) {
+                if (32 * j < rdims && 32 * i < rdims) {  // (uniform)
+                    const float x = __shfl_sync(0xffffffffu, v[j], o & 31);
+                    if (o >> 5 == j) y = x;
+                }
+            }
+        } else if (d < rdims) {
+            y = __ldcg(src + o);
+        }
+        if (d < pad) put_at(d, d < dim ? turned(d, v[i], y) : 0.f);
+    }
+    for (int d = lane + 32 * HA_REGS; d < pad; d += 32) put_at(d, d < dim ? turned(d, __ldcg(src + d), __ldcg(src + partner(d))) : 0.f);
+}
+
+// The same by half / 4 lanes (a power of two) that hold both values of their pairs, four pairs each and four values at a time of the
+// unrotated rest; for the portions of a prompt.  Everything is aligned to four values.
+__device__ __forceinline__ void put4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void put4(bf16* p, float4 v) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w)); }
+template <typename T>
+__device__ __forceinline__ void normed_rotated_quads(const float* src, const float* w, int dim, int rdims, float eps, const float2* cs, int lanes, T* dst) {
+    const int l = (threadIdx.x & 31) & (lanes - 1), half = rdims >> 1;
+    const float4 a = __ldcg(reinterpret_cast<const float4*>(src) + l), b = __ldcg(reinterpret_cast<const float4*>(src + half) + l);
+    float ss = a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w + b.x * b.x + b.y * b.y + b.z * b.z + b.w * b.w;
+    for (int d = rdims + 4 * l; d < dim; d += 4 * lanes) {
+        const float4 c = __ldcg(reinterpret_cast<const float4*>(src + d));
+        ss += c.x * c.x + c.y * c.y + c.z * c.z + c.w * c.w;
+    }
+    for (int o = 1; o < lanes; o <<= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float inv = 1.f / sqrtf(ss / (float)dim + eps);
+    const float4 wa = __ldg(reinterpret_cast<const float4*>(w) + l), wb = __ldg(reinterpret_cast<const float4*>(w + half) + l);
+    const float4 t = __ldg(reinterpret_cast<const float4*>(cs) + 2 * l), u = __ldg(reinterpret_cast<const float4*>(cs) + 2 * l + 1);
+    const float4 p = make_float4(a.x * inv * wa.x, a.y * inv * wa.y, a.z * inv * wa.z, a.w * inv * wa.w);
+    const float4 q = make_float4(b.x * inv * wb.x, b.y * inv * wb.y, b.z * inv * wb.z, b.w * inv * wb.w);
+    put4(dst + 4 * l, make_float4(p.x * t.x - q.x * t.y, p.y * t.z - q.y * t.w, p.z * u.x - q.z * u.y, p.w * u.z - q.w * u.w));
+    put4(dst + half + 4 * l, make_float4(q.x * t.x + p.x * t.y, q.y * t.z + p.y * t.w, q.z * u.x + p.z * u.y, q.w * u.z + p.w * u.w));
+    for (int d = rdims + 4 * l; d < dim; d += 4 * lanes) {
+        const float4 c = __ldcg(reinterpret_cast<const float4*>(src + d)), wc = __ldg(reinterpret_cast<const float4*>(w + d));
+        put4(dst + d, make_float4(c.x * inv * wc.x, c.y * inv * wc.y, c.z * inv * wc.z, c.w * inv * wc.w));
+    }
+}
+// Grid (parts of the items, rows): the operands of a prompt portion.  Needs dim a multiple of 8 that is its own stored size, vdim a
+// multiple of 8, `lanes` = rdims / 8 a power of two up to 32, ld and offsets multiples of 4.
+__global__ void __launch_bounds__(HA_WARPS * 32) head_rows_quads_kernel(const __grid_constant__ HeadAttnParams p, int lanes) {
+    const HeadShape& S = p.s;
+    const int row = (int)blockIdx.y, pos = scan_position(p.c, row), per = HA_WARPS * 32 / lanes;  // vectors at a time
+    const float2* const cs = p.rope + (size_t)pos * (S.rdims >> 1);
+    const float* const in = p.in + (size_t)row * p.ld;
+    bf16* const cache = static_cast<bf16*>(p.c.cache) + (size_t)pos * S.row;
+    const int nq = 2 * S.heads, n = nq + (p.own_kv ? 2 * S.kv_heads : 0);
+    for (int i0 = (int)blockIdx.x * per; i0 < n; i0 += (int)gridDim.x * per) {
+        const int i = min(i0 + (int)threadIdx.x / lanes, n - 1);  // (the last ones may do the same work twice: shuffles need whole warps)
+        if (i < nq) normed_rotated_quads(in + (size_t)i * S.dim, p.qnorm, S.dim, S.rdims, S.eps, cs, lanes, p.pq + ((size_t)row * nq + i) * p.dq);
+        else normed_rotated_quads(in + p.off_k + (size_t)(i - nq) * S.dim, p.knorm, S.dim, S.rdims, S.eps, cs, lanes,
+                                  cache + (size_t)((i - nq) >> 1) * p.c.group_stride + S.vp + ((i - nq) & 1) * S.dp);
+    }
+    if (!p.own_kv) return;
+    for (int i = ((int)blockIdx.x * HA_WARPS * 32 + (int)threadIdx.x) * 4; i < S.kv_heads * S.vdim; i += (int)gridDim.x * HA_WARPS * 128)
+        put4(cache + (size_t)(i / S.vdim) * p.c.group_stride + i % S.vdim, __ldcg(reinterpret_cast<const float4*>(in + p.off_v + i)));
 }
 
 // Grid (ceil(items / HA_WARPS), rows); a warp makes one item: the query of a (head, map), the key of a (kv head, map), a value.
@@ -64,25 +146,18 @@ __global__ void __launch_bounds__(HA_WARPS * 32) head_rows_kernel(const __grid_c
         const int sub = query ? item : item - nq;
         const float* const src = in + (query ? 0 : p.off_k) + (size_t)sub * S.dim;
         const float* const w = query ? p.qnorm : p.knorm;
-        float ss = 0.f;
-        for (int d = lane; d < S.dim; d += 32) {
-            const float v = __ldcg(src + d);
-            ss = fmaf(v, v, ss);
-        }
-        const float inv = 1.f / sqrtf(warp_sum(ss) / (float)S.dim + S.eps);
         if (!query) {
             CT* const dst = static_cast<CT*>(p.c.cache) + (size_t)row * p.c.cache_stride + (size_t)(sub >> 1) * p.c.group_stride + (size_t)pos * S.row + S.vp + (sub & 1) * S.dp;
-            for (int d = lane; d < S.dp; d += 32) put(dst + d, d < S.dim ? normed_rotated(src, inv, w, d, S.rdims, cs) : 0.f);
+            normed_rotated(src, w, S.dim, S.rdims, S.eps, cs, S.dp, [&](int d, float v) { put(dst + d, v); });
         } else if (p.pq) {
             bf16* const dst = p.pq + ((size_t)row * nq + sub) * p.dq;
-            for (int d = lane; d < p.dq; d += 32) put(dst + d, d < S.dim ? normed_rotated(src, inv, w, d, S.rdims, cs) : 0.f);
+            normed_rotated(src, w, S.dim, S.rdims, S.eps, cs, p.dq, [&](int d, float v) { put(dst + d, v); });
         } else {
             float* const dst = p.c.qp + ((size_t)row * nq + sub) * S.row;
-            const int k0 = S.vp + (sub & 1) * S.dp;
-            for (int e = lane; e < S.row; e += 32) {
-                const int d = e - k0;
-                dst[e] = d >= 0 && d < S.dim ? S.scale2 * normed_rotated(src, inv, w, d, S.rdims, cs) : 0.f;
-            }
+            const int k0 = S.vp + (sub & 1) * S.dp, k1 = k0 + S.dp;
+            for (int e = lane; e < S.row; e += 32)
+                if (e < k0 || e >= k1) dst[e] = 0.f;
+            normed_rotated(src, w, S.dim, S.rdims, S.eps, cs, S.dp, [&](int d, float v) { dst[k0 + d] = S.scale2 * v; });
         }
         return;
     }

@@ -277,7 +277,8 @@ __global__ void __launch_bounds__(MP_THREADS) mlstm_state_kernel(const __grid_co
 }
 
 // Grid (vt, chunks, heads), clusters of vt blocks.
-struct McSmem {  // Q, K (later A high and low), V, ring of [64 rows of S][128 columns] high and low
+constexpr int MC_ROWS = 32, MC_BOX = MC_ROWS * 128, MC_SLOT = 4 * MC_BOX, MC_MAX_SLOTS = 4;  // a ring slot: 32 rows of S x 128 columns, both terms
+struct McSmem {  // Q, K (later A high and low), V, ring of S
     int q, k, v, s, total, qbytes;
 };
 __host__ __device__ inline McSmem mc_smem_layout(int dp, int sstages) {
@@ -287,14 +288,14 @@ __host__ __device__ inline McSmem mc_smem_layout(int dp, int sstages) {
     L.k = L.qbytes;
     L.v = L.k + (L.qbytes > 4 * MP_SUB ? L.qbytes : 4 * MP_SUB);
     L.s = L.v + 2 * MP_SUB;
-    L.total = L.s + sstages * 2 * MP_SUB;
+    L.total = L.s + sstages * MC_SLOT;
     return L;
 }
-__global__ void __launch_bounds__(MP_THREADS) mlstm_chunk_kernel(const __grid_constant__ MlstmPrefillParams p, const __grid_constant__ CUtensorMap map_q,
+__global__ void __launch_bounds__(MP_THREADS, 1) mlstm_chunk_kernel(const __grid_constant__ MlstmPrefillParams p, const __grid_constant__ CUtensorMap map_q,
                                                                  const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                                                                  const __grid_constant__ CUtensorMap map_sh, const __grid_constant__ CUtensorMap map_sl) {
     extern __shared__ __align__(1024) uint8_t mc_raw[];
-    __shared__ __align__(8) uint64_t s_qk, s_v, s_s[2], s_sfree[2], s_a, s_p, s_o;
+    __shared__ __align__(8) uint64_t s_qk, s_v, s_s[MC_MAX_SLOTS], s_sfree[MC_MAX_SLOTS], s_a, s_p, s_o;
     __shared__ uint32_t s_tmem;
     __shared__ float s_g[MP_L];                     // a of the chunk's tokens
     __shared__ float s_den[2][MP_L];                // halves' shares of n . q
@@ -305,7 +306,7 @@ __global__ void __launch_bounds__(MP_THREADS) mlstm_chunk_kernel(const __grid_co
     const McSmem L = mc_smem_layout(p.dp, p.sstages);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int rank = (int)blockIdx.x, c0 = rank * MP_COLS, c = (int)blockIdx.y, h = (int)blockIdx.z;
-    const int nd = (p.dp + 63) / 64, t0 = c * MP_L;
+    const int nd = (p.dp + 63) / 64, ns = (p.dp + MC_ROWS - 1) / MC_ROWS, t0 = c * MP_L;
     const bool state = c > 0 || p.m.pos0 > 0;       // (a sequence's first chunk has none)
     if (threadIdx.x == 0) {
         mbar_init(&s_qk, 1);
@@ -313,7 +314,7 @@ __global__ void __launch_bounds__(MP_THREADS) mlstm_chunk_kernel(const __grid_co
         mbar_init(&s_a, 1);
         mbar_init(&s_p, MP_WARPS);
         mbar_init(&s_o, 1);
-        for (int i = 0; i < 2; ++i) {
+        for (int i = 0; i < p.sstages; ++i) {
             mbar_init(s_s + i, 1);
             mbar_init(s_sfree + i, 1);
         }
@@ -338,18 +339,18 @@ __global__ void __launch_bounds__(MP_THREADS) mlstm_chunk_kernel(const __grid_co
             }
             mbar_arrive_expect_tx(&s_v, 2 * MP_SUB);
             for (int i = 0; i < 2; ++i) tma_load_2d(smem + L.v + i * MP_SUB, &map_v, h * p.vp + c0 + 64 * i, t0, &s_v);
-            for (int j = 0; state && j < nd && ok; ++j) {
-                const int s = p.sstages == 2 ? j & 1 : 0, use = p.sstages == 2 ? j >> 1 : j;
+            for (int j = 0; state && j < ns && ok; ++j) {
+                const int s = j % p.sstages, use = j / p.sstages;
                 if (use > 0 && !mbar_wait_bounded(s_sfree + s, (uint32_t)((use - 1) & 1))) {
                     ok = false;
                     break;
                 }
-                uint8_t* const dst = smem + L.s + s * 2 * MP_SUB;  // high: 2 x [64 rows][64 columns], then low
-                mbar_arrive_expect_tx(s_s + s, 2 * MP_SUB);
-                const int row = (c * S.heads + h) * p.dp + 64 * j;
+                uint8_t* const dst = smem + L.s + s * MC_SLOT;  // high: 2 x [32 rows][64 columns], then low
+                mbar_arrive_expect_tx(s_s + s, MC_SLOT);
+                const int row = (c * S.heads + h) * p.dp + MC_ROWS * j;
                 for (int i = 0; i < 2; ++i) {
-                    tma_load_2d(dst + i * (MP_SUB / 2), &map_sh, c0 + 64 * i, row, s_s + s);
-                    tma_load_2d(dst + MP_SUB + i * (MP_SUB / 2), &map_sl, c0 + 64 * i, row, s_s + s);
+                    tma_load_2d(dst + i * MC_BOX, &map_sh, c0 + 64 * i, row, s_s + s);
+                    tma_load_2d(dst + (2 + i) * MC_BOX, &map_sl, c0 + 64 * i, row, s_s + s);
                 }
             }
             if (!ok) {
@@ -369,18 +370,18 @@ __global__ void __launch_bounds__(MP_THREADS) mlstm_chunk_kernel(const __grid_co
                               kk ? 1u : 0u);
                 umma_commit(&s_a);
             }
-            for (int j = 0; state && j < nd && ok; ++j) {
-                const int s = p.sstages == 2 ? j & 1 : 0, use = p.sstages == 2 ? j >> 1 : j;
+            for (int j = 0; state && j < ns && ok; ++j) {
+                const int s = j % p.sstages, use = j / p.sstages;
                 if (!mbar_wait_bounded(s_s + s, (uint32_t)(use & 1))) {
                     ok = false;
                     break;
                 }
                 tc_fence_after();
-                const uint8_t* const src = smem + L.s + s * 2 * MP_SUB;
+                const uint8_t* const src = smem + L.s + s * MC_SLOT;
                 for (int term = 0; term < 2; ++term)
-                    for (int kk = 0; kk < 4 && 64 * j + 16 * kk < p.dp; ++kk)
-                        umma_bf16(tmem_r, umma_desc_sw128(smem + L.q + j * MP_SUB, kk * 32), umma_desc_sw128_mn(src + term * MP_SUB, kk * 2048, MP_SUB / 2), idesc_v,
-                                  j | term | kk ? 1u : 0u);
+                    for (int kk = 0; kk < MC_ROWS / 16 && MC_ROWS * j + 16 * kk < p.dp; ++kk)
+                        umma_bf16(tmem_r, umma_desc_sw128(smem + L.q + (j >> 1) * MP_SUB, (j & 1) * 64 + kk * 32), umma_desc_sw128_mn(src + 2 * term * MC_BOX, kk * 2048, MC_BOX),
+                                  idesc_v, j | term | kk ? 1u : 0u);
                 umma_commit(s_sfree + s);
             }
             if (ok && (!mbar_wait_bounded(&s_v, 0u) || !mbar_wait_bounded(&s_p, 0u))) ok = false;

@@ -406,7 +406,7 @@ struct StackSession {
     void *act = nullptr, *act2 = nullptr;        // operands of the products, [max_rows][k rounded up to 8]
     bf16 *pq = nullptr, *pk = nullptr, *pv = nullptr;  // prompt attention: queries; latent attention: expanded keys, transposed values
     int pv_ld = 0;
-    float* aside = nullptr;                      // differential attention with many value dimensions: the first map's result
+    float* aside = nullptr;                      // differential attention: the first map's result
     MlstmPrefillParams mp = {};                  // mLSTM in chunks: buffers (q null: there are none)
 };
 
@@ -433,16 +433,23 @@ static int prefill_kstages(const LatentShape& s, const DeviceInfo& di) {
     return 0;
 }
 
-static int head_prefill_kstages(const HeadShape& s, const DeviceInfo& di) {
-    const int vn = up(s.vdim, 16);
+// Key stages of the tiled differential attention (0: the heads do not fit it), and whether two of its blocks share an SM.
+static int head_prefill_kstages(const HeadShape& s, const DeviceInfo& di, bool* two = nullptr) {
+    const int vn = up(s.vdim, 16), sm_bytes = di.max_smem_optin + 1024;                       // (1 KiB of an SM's shared memory goes to every block)
+    auto bytes = [&](int k) { return hp_smem_layout(s.dim, vn, k).total + 1024 + 5 * 1024; };  // (static shared memory included)
+    if (two) *two = false;
     if (vn > 256 || !(s.scale2 > 0.f)) return 0;
+    if (vn <= HP_HALF_COLS && 2 * (bytes(1) + 1024) <= sm_bytes) {
+        if (two) *two = true;
+        return 2 * (bytes(2) + 1024) <= sm_bytes ? 2 : 1;
+    }
     for (int k = 2; k >= 1; --k)
-        if (hp_smem_layout(s.dim, vn, k).total + 1024 <= di.max_smem_optin - 4096) return k;
+        if (bytes(k) <= di.max_smem_optin) return k;
     return 0;
 }
 // Ring slots of the chunk kernel (0: the heads do not fit the chunked form).
 static int mlstm_prefill_stages(const MlstmShape& s, const DeviceInfo& di) {
-    for (int k = 2; k >= 1; --k)
+    for (int k = MC_MAX_SLOTS; k >= 1; --k)
         if (mc_smem_layout(up(s.dim, 16), k).total + 1024 <= di.max_smem_optin - 8192) return k;
     return 0;
 }
@@ -520,7 +527,7 @@ int32_t stack_session_create(const StackModel* m, const StackSessionInfo& info, 
         max_k2 = std::max(std::max(max_k2, w.o.k), std::max(w.down.k, w.side_proj.k));
         if (w.head.heads && head_prefill_kstages(w.head, di)) {
             pq = std::max(pq, (size_t)2 * w.head.heads * up(w.head.dim, 16));
-            if (up(w.head.vdim, 16) > HP_OWN_COLS) aside = std::max(aside, (size_t)w.head.heads * w.head.vdim);
+            aside = std::max(aside, (size_t)w.head.heads * w.head.vdim);
         }
         if (w.mlstm.heads && mlstm_prefill_stages(w.mlstm, di)) {
             const MlstmShape& sh = w.mlstm;
@@ -1007,7 +1014,8 @@ static int32_t enqueue_head_rows(StackSession* s, int run, int n, int pos0, cons
     a.out = s->act2;
     a.ldo = ldo;
     const HeadShape& sh = a.s;
-    const int kstages = head_prefill_kstages(sh, s->di);
+    bool two;
+    const int kstages = head_prefill_kstages(sh, s->di, &two), blocks = (n + HP_TILE - 1) / HP_TILE * sh.heads;
     if (!s->pq || pos_list || n < EXPAND_MIN_ROWS || kstages == 0)
         return rows_in_parts(s, a, n, [&](HeadAttnParams& b, int r, int k) {
             b.in += (size_t)r * a.ld;
@@ -1016,16 +1024,21 @@ static int32_t enqueue_head_rows(StackSession* s, int run, int n, int pos0, cons
         });
     a.pq = s->pq;
     a.dq = up(sh.dim, 16);
-    CU(launch_head_rows<bf16>(a, n, false, st));
+    const int lanes = sh.rdims / 8, vectors = 2 * sh.heads + (a.own_kv ? 2 * sh.kv_heads : 0), per = lanes ? HA_WARPS * 32 / lanes : 1;
+    if (sh.rdims % 8 == 0 && lanes && (lanes & (lanes - 1)) == 0 && lanes <= 32 && sh.dim % 16 == 0 && sh.vdim % 8 == 0)
+        head_rows_quads_kernel<<<dim3((vectors + per - 1) / per, n), HA_WARPS * 32, 0, st>>>(a, lanes);
+    else launch_head_rows<bf16>(a, n, false, st);
+    CU(cudaGetLastError());
     HeadPrefillParams f;
     memset(&f, 0, sizeof(f));
     f.s = sh; f.n = n; f.pos0 = pos0; f.chunk = a.c.chunk; f.dq = a.dq; f.vn = up(sh.vdim, 16); f.kstages = kstages;
+    f.paired = two && blocks > s->di.sms && blocks <= 2 * s->di.sms ? s->di.sms : 0;
     f.gate = a.in + a.off_g; f.ld = a.ld; f.aside = s->aside; f.out = static_cast<bf16*>(s->act2); f.ldo = ldo; f.status = status;
     CUtensorMap mq, mkv;
     L2B_TRY(bf16_map(mq, s->pq, (int64_t)2 * sh.heads * a.dq, n, (int64_t)2 * sh.heads * a.dq, HP_TILE));
     L2B_TRY(bf16_map(mkv, static_cast<const bf16*>(a.c.cache), sh.row, pos0 + n, sh.row, HP_TILE, sh.kv_heads, (int64_t)a.c.group_stride));
     const size_t smem = (size_t)hp_smem_layout(sh.dim, f.vn, kstages).total + 1024;
-    CU(launch_kernel_args(head_prefill_kernel, dim3((n + HP_TILE - 1) / HP_TILE, sh.heads), dim3(HP_THREADS), smem, st, false, 1, f, mq, mkv));
+    CU(launch_kernel_args(head_prefill_kernel, dim3(blocks), dim3(HP_THREADS), smem, st, false, 1, f, mq, mkv));
     *launches += 2;
     return L2B_OK;
 }
@@ -1058,8 +1071,8 @@ static int32_t enqueue_mlstm_rows(StackSession* s, int run, int n, int pos0, con
         L2B_TRY(bf16_map(mq, p.q, nk, n, nk, MP_L));
         L2B_TRY(bf16_map(mk, p.k, nk, n, nk, MP_L));
         L2B_TRY(bf16_map(mv, p.v, nv, n, nv, MP_L));
-        L2B_TRY(bf16_map(msh, p.sh, p.vs, rows, p.vs, 64));
-        L2B_TRY(bf16_map(msl, p.sl, p.vs, rows, p.vs, 64));
+        L2B_TRY(bf16_map(msh, p.sh, p.vs, rows, p.vs, MC_ROWS));
+        L2B_TRY(bf16_map(msl, p.sl, p.vs, rows, p.vs, MC_ROWS));
         mlstm_operands_kernel<<<n, 256, 0, st>>>(p);
         CU(cudaGetLastError());
         mlstm_gates_kernel<<<sh.heads, 32 * p.nchunk, 0, st>>>(p);
