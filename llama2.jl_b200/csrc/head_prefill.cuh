@@ -304,7 +304,7 @@ __global__ void __launch_bounds__(HP_THREADS) head_prefill_kernel(const __grid_c
                     o[i] = t < p.n && c + lane < p.s.vdim ? __ldg(p.gate + (size_t)t * p.ld + h * p.s.vdim + c + lane) : 0.f;
                 }
 #pragma unroll
-                for (int i = 0; i < 32; ++i) sg[i * 33 + lane] = sigmoid(o[i]);
+                for (int i = 0; i < 32; ++i) sg[i * 33 + lane] = fast_sigmoid(o[i]);
                 __syncwarp();
                 difference(c, o);
                 const int n = qi < p.n ? p.s.vdim - c : 0;  // values of this query to store

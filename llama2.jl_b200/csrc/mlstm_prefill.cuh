@@ -125,8 +125,8 @@ __global__ void __launch_bounds__(MP_MAX_CHUNKS * 32) mlstm_gates_kernel(const _
 }
 
 // Grid (blocks of 64 columns, blocks of 128 rows, heads).
-struct MsSmem {  // K [2 stages][2 pieces of 64 dims], u V high and low [2 pieces each: 64 columns; u]
-    static constexpr int k = 0, w = 4 * MP_SUB, total = 8 * MP_SUB;
+struct MsSmem {  // K [2 stages][2 pieces of 64 dims], u V [2 stages] high and low [2 pieces each: 64 columns; u]
+    static constexpr int k = 0, w = 4 * MP_SUB, wbytes = 4 * MP_SUB, total = 12 * MP_SUB;
 };
 __global__ void __launch_bounds__(MP_THREADS) mlstm_state_kernel(const __grid_constant__ MlstmPrefillParams p, const __grid_constant__ CUtensorMap map_k) {
     extern __shared__ __align__(1024) uint8_t ms_raw[];
@@ -178,7 +178,7 @@ __global__ void __launch_bounds__(MP_THREADS) mlstm_state_kernel(const __grid_co
                 for (int term = 0; term < 2; ++term)
                     for (int kk = 0; kk < 8; ++kk)
                         umma_bf16(tmem, umma_desc_sw128_mn(smem + MsSmem::k + 2 * s * MP_SUB, kk * 2048, MP_SUB),
-                                  umma_desc_sw128_mn(smem + MsSmem::w + 2 * term * MP_SUB, kk * 2048, MP_SUB), idesc, 1u);
+                                  umma_desc_sw128_mn(smem + MsSmem::w + s * MsSmem::wbytes + 2 * term * MP_SUB, kk * 2048, MP_SUB), idesc, 1u);
                 umma_commit(s_kfree + s);
                 umma_commit(&s_mma);
             }
@@ -194,16 +194,40 @@ __global__ void __launch_bounds__(MP_THREADS) mlstm_state_kernel(const __grid_co
         // u V: this thread's token of a chunk and its 32 columns
         const int tok = r;
         uint4 v[4];
+        float u = 0.f, decay = 0.f;
         auto fetch = [&](int c) {
             const bf16* src = p.v + (size_t)(c * MP_L + tok) * S.heads * p.vp + (size_t)h * p.vp + cc;
 #pragma unroll
             for (int i = 0; i < 4; ++i)
                 v[i] = c < p.nchunk && c * MP_L + tok < p.n && cc + 8 * i < p.vp ? __ldg(reinterpret_cast<const uint4*>(src) + i) : make_uint4(0u, 0u, 0u, 0u);
+            u = c < p.nchunk ? __ldg(p.u + ((size_t)h * p.nchunk + c) * MP_L + tok) : 0.f;
+        };
+        auto weigh = [&](int c) {  // u V of chunk c in two terms; rows are tokens
+            uint8_t* const wh = smem + MsSmem::w + (c & 1) * MsSmem::wbytes;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const uint32_t x[4] = {v[i].x, v[i].y, v[i].z, v[i].w};
+                uint32_t hi[4], lo[4];
+#pragma unroll
+                for (int k = 0; k < 4; ++k) split2(u * __uint_as_float(x[k] << 16), u * __uint_as_float(x[k] & 0xFFFF0000u), hi[k], lo[k]);
+                const int off = sw128_chunk(tok, 4 * half + i);
+                *reinterpret_cast<uint4*>(wh + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+                *reinterpret_cast<uint4*>(wh + 2 * MP_SUB + off) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+            }
+            // column 64: u; columns 65 .. 79: zeros
+            uint32_t hi, lo;
+            split2(u, 0.f, hi, lo);
+            const int off = MP_SUB + sw128_chunk(tok, half);
+            *reinterpret_cast<uint4*>(wh + off) = make_uint4(half ? 0u : hi, 0u, 0u, 0u);
+            *reinterpret_cast<uint4*>(wh + 2 * MP_SUB + off) = make_uint4(half ? 0u : lo, 0u, 0u, 0u);
         };
         fetch(0);
+        weigh(0);
+        fetch(1);
         bool ok = true;
         for (int c = 0; c <= p.nchunk; ++c) {
             float st[32], n = 0.f;
+            if (c < p.nchunk) decay = __ldg(p.decay + (size_t)h * p.nchunk + c);
             if (c == 0) {
 #pragma unroll
                 for (int k = 0; k < 32; ++k) st[k] = !fresh && row_in && cc + k < S.vdim ? gs[k] : 0.f;
@@ -224,28 +248,17 @@ __global__ void __launch_bounds__(MP_THREADS) mlstm_state_kernel(const __grid_co
                 }
                 break;
             }
-            const float decay = __ldg(p.decay + (size_t)h * p.nchunk + c), u = __ldg(p.u + ((size_t)h * p.nchunk + c) * MP_L + tok);
-            // u V in two terms; rows are tokens
-            uint8_t* const wh = smem + MsSmem::w;
+            float kept[32];
 #pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                const uint32_t x[4] = {v[i].x, v[i].y, v[i].z, v[i].w};
-                uint32_t hi[4], lo[4];
-#pragma unroll
-                for (int k = 0; k < 4; ++k) split2(u * __uint_as_float(x[k] << 16), u * __uint_as_float(x[k] & 0xFFFF0000u), hi[k], lo[k]);
-                const int off = sw128_chunk(tok, 4 * half + i);
-                *reinterpret_cast<uint4*>(wh + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-                *reinterpret_cast<uint4*>(wh + 2 * MP_SUB + off) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
-            }
-            {  // column 64: u; columns 65 .. 79: zeros
-                uint32_t hi, lo;
-                split2(u, 0.f, hi, lo);
-                const int off = MP_SUB + sw128_chunk(tok, half);
-                *reinterpret_cast<uint4*>(wh + off) = make_uint4(half ? 0u : hi, 0u, 0u, 0u);
-                *reinterpret_cast<uint4*>(wh + 2 * MP_SUB + off) = make_uint4(half ? 0u : lo, 0u, 0u, 0u);
-            }
-            fetch(c + 1);
-            // the state before this chunk, for the chunk kernel
+            for (int k = 0; k < 32; ++k) kept[k] = st[k] * decay;
+            tmem_st32f(at, kept);
+            if (half == 0) tmem_st1f(at_n, n * decay);
+            fence_proxy_async();
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&s_w);
+            // beside the products: the state before this chunk, for the chunk kernel, and the next chunk's operand (its place is free, as
+            // the products before these are done)
             if (d < p.dp) {
                 const size_t row = ((size_t)c * S.heads + h) * p.dp + d;
 #pragma unroll
@@ -260,14 +273,8 @@ __global__ void __launch_bounds__(MP_THREADS) mlstm_state_kernel(const __grid_co
                 }
                 if (has_n) p.sn[row] = row_in ? n : 0.f;
             }
-#pragma unroll
-            for (int k = 0; k < 32; ++k) st[k] *= decay;
-            tmem_st32f(at, st);
-            if (half == 0) tmem_st1f(at_n, n * decay);
-            fence_proxy_async();
-            tc_fence_before();
-            __syncwarp();
-            if (lane == 0) mbar_arrive(&s_w);
+            if (c + 1 < p.nchunk) weigh(c + 1);
+            fetch(c + 2);
         }
         if (!ok && lane == 0) atomicExch(p.status, DEV_ERR_TMA_TIMEOUT);
     }
@@ -505,7 +512,7 @@ __global__ void __launch_bounds__(MP_THREADS, 1) mlstm_chunk_kernel(const __grid
 #pragma unroll
             for (int k = 0; k < 32; ++k) x[k] = tw + k < p.n && col_in ? __ldg(p.m.in + (size_t)(tw + k) * p.m.ld + p.m.off_g + (size_t)h * S.vdim + cc + lane) : 0.f;
 #pragma unroll
-            for (int k = 0; k < 32; ++k) sg[k * 33 + lane] = norm * sigmoid(x[k]);
+            for (int k = 0; k < 32; ++k) sg[k * 33 + lane] = norm * fast_sigmoid(x[k]);
             __syncwarp();
             const int nv = t0 + row < p.n ? S.vdim - cc : 0;  // values of this token to store
             bf16* const dst = out + (size_t)(t0 + row) * p.m.ldo + (size_t)h * S.vdim + cc;
