@@ -228,6 +228,9 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t&
 // sigmoid for results that are rounded to bf16 next
 __device__ __forceinline__ float fast_sigmoid(float z) { return __fdividef(1.f, 1.f + fast_exp2(z * -1.4426950408889634f)); }
 
+// two packed bf16 times two f32
+__device__ __forceinline__ uint32_t mul_pack_bf16(uint32_t g, float x, float y) { return pack_bf16(__uint_as_float(g << 16) * x, __uint_as_float(g & 0xFFFF0000u) * y); }
+
 // Sum over the first NW warps of a block; each of their threads gets it.  s holds NW floats and may be reused after the next barrier.
 template <int NW>
 __device__ __forceinline__ float block_sum_all(float v, float* s) {

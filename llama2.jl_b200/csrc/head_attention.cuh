@@ -29,6 +29,7 @@ struct HeadAttnParams {
     const float2* rope;     // [positions][rdims / 2]
     bf16* pq;               // queries as operands [rows][2 heads][dq] (null: query vectors of the scan)
     int dq;
+    bf16* pg;               // beside them: sigmoid of the gates [rows][heads * vp]
     void* out;              // [rows][ldo]
     int ldo;
 };
@@ -124,12 +125,17 @@ __global__ void __launch_bounds__(HA_WARPS * 32) head_rows_quads_kernel(const __
         else normed_rotated_quads(in + p.off_k + (size_t)(i - nq) * S.dim, p.knorm, S.dim, S.rdims, S.eps, cs, lanes,
                                   cache + (size_t)((i - nq) >> 1) * p.c.group_stride + S.vp + ((i - nq) & 1) * S.dp);
     }
+    for (int i = ((int)blockIdx.x * HA_WARPS * 32 + (int)threadIdx.x) * 4; i < S.heads * S.vdim; i += (int)gridDim.x * HA_WARPS * 128) {
+        const float4 g = __ldcg(reinterpret_cast<const float4*>(in + p.off_g + i));
+        put4(p.pg + (size_t)row * S.heads * S.vdim + i, make_float4(fast_sigmoid(g.x), fast_sigmoid(g.y), fast_sigmoid(g.z), fast_sigmoid(g.w)));
+    }
     if (!p.own_kv) return;
     for (int i = ((int)blockIdx.x * HA_WARPS * 32 + (int)threadIdx.x) * 4; i < S.kv_heads * S.vdim; i += (int)gridDim.x * HA_WARPS * 128)
         put4(cache + (size_t)(i / S.vdim) * p.c.group_stride + i % S.vdim, __ldcg(reinterpret_cast<const float4*>(in + p.off_v + i)));
 }
 
-// Grid (ceil(items / HA_WARPS), rows); a warp makes one item: the query of a (head, map), the key of a (kv head, map), a value.
+// Grid (ceil(items / HA_WARPS), rows); a warp makes one item: the query of a (head, map), the key of a (kv head, map), a value, a head's
+// gates (operands only).
 template <typename CT>
 __global__ void __launch_bounds__(HA_WARPS * 32) head_rows_kernel(const __grid_constant__ HeadAttnParams p) {
     const HeadShape& S = p.s;
@@ -162,7 +168,13 @@ __global__ void __launch_bounds__(HA_WARPS * 32) head_rows_kernel(const __grid_c
         return;
     }
     item -= nq + nk;
-    if (item >= nv) return;
+    if (item >= nv) {
+        item -= nv;
+        if (!p.pq || item >= S.heads) return;
+        for (int d = lane; d < S.vp; d += 32)
+            put(p.pg + ((size_t)row * S.heads + item) * S.vp + d, d < S.vdim ? fast_sigmoid(__ldcg(in + p.off_g + (size_t)item * S.vdim + d)) : 0.f);
+        return;
+    }
     const float* const src = in + p.off_v + (size_t)item * S.vdim;
     CT* const dst = static_cast<CT*>(p.c.cache) + (size_t)row * p.c.cache_stride + (size_t)item * p.c.group_stride + (size_t)pos * S.row;
     for (int d = lane; d < S.vp; d += 32) put(dst + d, d < S.vdim ? __ldcg(src + d) : 0.f);

@@ -27,9 +27,7 @@ struct HeadPrefillParams {
     int vn;           // vdim rounded up to 16
     int kstages;
     int paired;       // number of SMs when all blocks run at once, two per SM; else 0
-    const float* gate;  // gate of (row, head, v) at gate[row * ld + head * vdim + v]
-    int ld;
-    float* aside;     // [n][heads * vdim]: the first map's result
+    float* aside;     // [heads][128-query tiles][vdim][128]: the first map's result
     bf16* out;        // [n][ldo]
     int ldo;
     int* status;
@@ -49,10 +47,10 @@ __host__ __device__ inline HpSmem hp_smem_layout(int dim, int vn, int kstages) {
     return s;
 }
 
-__global__ void __launch_bounds__(HP_THREADS) head_prefill_kernel(const __grid_constant__ HeadPrefillParams p, const __grid_constant__ CUtensorMap map_q,
-                                                                  const __grid_constant__ CUtensorMap map_kv) {
+__global__ void __launch_bounds__(HP_THREADS, 2) head_prefill_kernel(const __grid_constant__ HeadPrefillParams p, const __grid_constant__ CUtensorMap map_q,
+                                                                  const __grid_constant__ CUtensorMap map_kv, const __grid_constant__ CUtensorMap map_g) {
     extern __shared__ __align__(1024) uint8_t hp_raw[];
-    __shared__ __align__(8) uint64_t s_q, s_qfree, s_k[2], s_kfree[2], s_v, s_s[2], s_sfree[2], s_p, s_o;
+    __shared__ __align__(8) uint64_t s_q, s_qfree, s_gate, s_k[2], s_kfree[2], s_v, s_s[2], s_sfree[2], s_p, s_o;
     __shared__ uint32_t s_tmem;
     __shared__ float s_row[2][2][HP_TILE];  // [tile parity][half][query]: the halves' maxima (at the ends: sums)
     __shared__ float s_ss[2][HP_TILE];
@@ -71,6 +69,7 @@ __global__ void __launch_bounds__(HP_THREADS) head_prefill_kernel(const __grid_c
     if (threadIdx.x == 0) {
         mbar_init(&s_q, 1);
         mbar_init(&s_qfree, 1);
+        mbar_init(&s_gate, 1);
         mbar_init(&s_v, 1);
         mbar_init(&s_p, HP_WARPS);
         mbar_init(&s_o, 1);
@@ -116,6 +115,12 @@ __global__ void __launch_bounds__(HP_THREADS) head_prefill_kernel(const __grid_c
                 mbar_arrive_expect_tx(&s_v, (uint32_t)L.vbytes);
                 for (int i = 0; i < nv; ++i) tma_load_3d(smem + L.v + i * HP_SUB, &map_kv, 64 * i, pos, g, &s_v);
             }
+            if (ok && mbar_wait_bounded(&s_o, (uint32_t)((nt2 - 1) & 1))) {  // all products are done: the gates take the operands' place
+                mbar_arrive_expect_tx(&s_gate, (uint32_t)L.vbytes);
+                for (int i = 0; i < nv; ++i) tma_load_2d(smem + L.q + i * HP_SUB, &map_g, h * p.s.vp + 64 * i, q0, &s_gate);
+            } else {
+                ok = false;
+            }
             if (!ok) {
                 atomicExch(p.status, DEV_ERR_TMA_TIMEOUT);
                 for (int i = 0; i < 2000; ++i) __nanosleep(1000);  // copies in flight land within microseconds
@@ -160,7 +165,7 @@ __global__ void __launch_bounds__(HP_THREADS) head_prefill_kernel(const __grid_c
         const int qd = warp & 3, half = (warp - 2) >> 2, r = 32 * qd + lane;
         const uint32_t lane_off = (uint32_t)(32 * qd) << 16;
         const int qi = q0 + r, qpos = p.pos0 + qi, qfirst = p.chunk ? qpos / p.chunk * p.chunk : 0;
-        float* const aside = p.aside + (size_t)min(qi, p.n - 1) * p.s.heads * p.s.vdim + (size_t)h * p.s.vdim;
+        float* const aside = p.aside + ((size_t)h * (blocks / p.s.heads) + q0 / HP_TILE) * p.s.vdim * HP_TILE + r;
         float m = 0.f, l = 0.f;
         bool ok = true;
         for (int t = 0; t < nt2; ++t) {
@@ -197,16 +202,9 @@ __global__ void __launch_bounds__(HP_THREADS) head_prefill_kernel(const __grid_c
                 for (int c = 32 * half; c < p.s.vdim; c += 64) {
                     float o[32];
                     tmem_ld32f(tmem_o + lane_off + (uint32_t)c, o);
-                    if (qi >= p.n) continue;
-                    if ((p.s.vdim & 3) == 0) {
 #pragma unroll
-                        for (int k = 0; k < 32; k += 4)
-                            if (c + k < p.s.vdim) *reinterpret_cast<float4*>(aside + c + k) = make_float4(o[k] * inv, o[k + 1] * inv, o[k + 2] * inv, o[k + 3] * inv);
-                    } else {
-#pragma unroll
-                        for (int k = 0; k < 32; ++k)
-                            if (c + k < p.s.vdim) aside[c + k] = o[k] * inv;
-                    }
+                    for (int k = 0; k < 32; ++k)
+                        if (c + k < p.s.vdim) aside[(c + k) * HP_TILE] = o[k] * inv;
                 }
             }
             if (j == 0) {
@@ -260,21 +258,9 @@ __global__ void __launch_bounds__(HP_THREADS) head_prefill_kernel(const __grid_c
         const float w2 = -p.s.lambda / (s_row[nt2 & 1][0][r] + s_row[nt2 & 1][1][r]);
         auto difference = [&](int c, float (&o)[32]) {  // (rows beyond n: any numbers, not stored)
             tmem_ld32f(tmem_o + lane_off + (uint32_t)c, o);
-            if ((p.s.vdim & 3) == 0) {
 #pragma unroll
-                for (int k = 0; k < 32; k += 4)
-                    if (c + k < p.s.vdim) {
-                        const float4 a = *reinterpret_cast<const float4*>(aside + c + k);
-                        o[k] = fmaf(w2, o[k], a.x);
-                        o[k + 1] = fmaf(w2, o[k + 1], a.y);
-                        o[k + 2] = fmaf(w2, o[k + 2], a.z);
-                        o[k + 3] = fmaf(w2, o[k + 3], a.w);
-                    }
-            } else {
-#pragma unroll
-                for (int k = 0; k < 32; ++k)
-                    if (c + k < p.s.vdim) o[k] = fmaf(w2, o[k], aside[c + k]);
-            }
+            for (int k = 0; k < 32; ++k)
+                if (c + k < p.s.vdim) o[k] = fmaf(w2, o[k], aside[(c + k) * HP_TILE]);
         };
         float ss = 0.f;
 #pragma unroll 1
@@ -286,40 +272,31 @@ __global__ void __launch_bounds__(HP_THREADS) head_prefill_kernel(const __grid_c
         }
         s_ss[half][r] = ss;
         partial_sync_2(HP_WARPS * 32);
+        if (ok && !__all_sync(0xffffffffu, mbar_wait_bounded(&s_gate, 0u))) ok = false;
         if (!ok) {
             if (lane == 0) atomicExch(p.status, DEV_ERR_TMA_TIMEOUT);
         } else {
             const float scale = p.s.out_scale / sqrtf((s_ss[0][r] + s_ss[1][r]) / (float)p.s.vdim + p.s.eps);
             bf16* out = p.out + (size_t)qi * p.ldo + (size_t)h * p.s.vdim;
             const bool wide = ((p.s.vdim | p.ldo) & 7) == 0;
-            // gates of this warp's 32 queries, 32 values at a time, through the shared memory that held Q, K and V (all products are done)
-            float* const sg = reinterpret_cast<float*>(smem + L.q) + (warp - 2) * (32 * 33);
 #pragma unroll 1
             for (int c = 32 * half; c < p.s.vdim; c += 64) {
                 float o[32];
-                __syncwarp();
-#pragma unroll
-                for (int i = 0; i < 32; ++i) {
-                    const int t = q0 + 32 * qd + i;
-                    o[i] = t < p.n && c + lane < p.s.vdim ? __ldg(p.gate + (size_t)t * p.ld + h * p.s.vdim + c + lane) : 0.f;
-                }
-#pragma unroll
-                for (int i = 0; i < 32; ++i) sg[i * 33 + lane] = fast_sigmoid(o[i]);
-                __syncwarp();
                 difference(c, o);
                 const int n = qi < p.n ? p.s.vdim - c : 0;  // values of this query to store
 #pragma unroll
-                for (int k = 0; k < 32; ++k) o[k] *= scale * sg[lane * 33 + k];
-                if (wide) {
+                for (int i = 0; i < 4; ++i) {
+                    const uint4 g8 = *reinterpret_cast<const uint4*>(smem + L.q + (c >> 6) * HP_SUB + sw128_chunk(r, 4 * half + i));
+                    const uint4 v = make_uint4(mul_pack_bf16(g8.x, o[8 * i] * scale, o[8 * i + 1] * scale), mul_pack_bf16(g8.y, o[8 * i + 2] * scale, o[8 * i + 3] * scale),
+                                               mul_pack_bf16(g8.z, o[8 * i + 4] * scale, o[8 * i + 5] * scale), mul_pack_bf16(g8.w, o[8 * i + 6] * scale, o[8 * i + 7] * scale));
+                    if (wide) {
+                        if (8 * i < n) *reinterpret_cast<uint4*>(out + c + 8 * i) = v;
+                    } else {
+                        const uint32_t w[4] = {v.x, v.y, v.z, v.w};
 #pragma unroll
-                    for (int i = 0; i < 4; ++i)
-                        if (8 * i < n)
-                            *reinterpret_cast<uint4*>(out + c + 8 * i) = make_uint4(pack_bf16(o[8 * i], o[8 * i + 1]), pack_bf16(o[8 * i + 2], o[8 * i + 3]),
-                                                                                    pack_bf16(o[8 * i + 4], o[8 * i + 5]), pack_bf16(o[8 * i + 6], o[8 * i + 7]));
-                } else {
-#pragma unroll
-                    for (int k = 0; k < 32; ++k)
-                        if (k < n) put(out + c + k, o[k]);
+                        for (int k = 0; k < 8; ++k)
+                            if (8 * i + k < n) out[c + 8 * i + k] = __ushort_as_bfloat16((unsigned short)(w[k >> 1] >> (16 * (k & 1))));
+                    }
                 }
             }
         }

@@ -2,7 +2,7 @@
 // forget gates within a chunk, a_s = i_s - F_s, and M_t = max(m_0, max_{s <= t} a_s) (so that the running maximum is m_t = F_t + M_t),
 //     S_t = exp(m_0 - M_t) S_0 + sum_{s <= t} exp(a_s - M_t) k_s v_s^T        (both sides scaled by exp(-m_t)),
 // every exponent at most zero.  So a chunk is two products with weights in between, and the state goes from chunk to chunk by one more:
-//   mlstm_operands_kernel  q (times dim^-1/2), k, v as bf16 operands;
+//   mlstm_operands_kernel  q (times dim^-1/2), k, v, and the output gate times the norm's weight, as bf16;
 //   mlstm_gates_kernel     a, M and the factors of every token and chunk, the running maximum after the portion;
 //   mlstm_state_kernel     a block has 128 x 64 values of a head's S in tensor memory, f32, and goes through the chunks: hands S out as
 //                          two bf16 terms (16 significant bits) for the kernel below, decays it, adds K^T (u V), where u V is split
@@ -24,7 +24,7 @@ struct MlstmPrefillParams {
     MlstmParams m;       // one sequence; out: bf16
     int n, nchunk;
     int dp, vp, vs;      // dim rounded up to 16; vdim rounded up to 8 (operands), and of the states' rows
-    bf16 *q, *k, *v;     // [n][heads * dp], [n][heads * dp], [n][heads * vp]
+    bf16 *q, *k, *v, *g;  // [n][heads * dp] twice, [n][heads * vp] twice
     float *a, *mx, *w, *floor, *u;  // [heads][nchunk * MP_L]: a_t, M_t, exp(m_0 - M_t), exp(-m_t), exp(a_t - M of the chunk's end)
     float* decay;        // [heads][nchunk]: exp(m_0 - M of the chunk's end)
     bf16 *sh, *sl;       // [nchunk][heads][dp][vs]: S before the chunk, high and low terms
@@ -38,17 +38,17 @@ __global__ void __launch_bounds__(256) mlstm_operands_kernel(const __grid_consta
     const MlstmShape& S = p.m.s;
     const int t = (int)blockIdx.x;
     const float* const in = p.m.in + (size_t)t * p.m.ld;
-    auto part = [&](bf16* out, const float* src, int dim, int pad, float mul) {
+    auto part = [&](bf16* out, int dim, int pad, auto value) {  // value(index among heads * dim)
         bf16* const dst = out + (size_t)t * S.heads * pad;
         for (int i = 2 * threadIdx.x; i < S.heads * pad; i += 512) {
             const int h = i / pad, d = i - h * pad;  // (pad is even)
-            const float x = d < dim ? src[(size_t)h * dim + d] * mul : 0.f, y = d + 1 < dim ? src[(size_t)h * dim + d + 1] * mul : 0.f;
-            *reinterpret_cast<uint32_t*>(dst + i) = pack_bf16(x, y);
+            *reinterpret_cast<uint32_t*>(dst + i) = pack_bf16(d < dim ? value(h * dim + d) : 0.f, d + 1 < dim ? value(h * dim + d + 1) : 0.f);
         }
     };
-    part(p.q, in, S.dim, p.dp, S.qscale);
-    part(p.k, in + p.m.off_k, S.dim, p.dp, 1.f);
-    part(p.v, in + p.m.off_v, S.vdim, p.vp, 1.f);
+    part(p.q, S.dim, p.dp, [&](int i) { return __ldcg(in + i) * S.qscale; });
+    part(p.k, S.dim, p.dp, [&](int i) { return __ldcg(in + p.m.off_k + i); });
+    part(p.v, S.vdim, p.vp, [&](int i) { return __ldcg(in + p.m.off_v + i); });
+    part(p.g, S.vdim, p.vp, [&](int i) { return __ldg(p.m.norm + i) * fast_sigmoid(__ldcg(in + p.m.off_g + i)); });
 }
 
 // Grid (heads), a warp per chunk, a lane four consecutive tokens.
@@ -128,7 +128,7 @@ __global__ void __launch_bounds__(MP_MAX_CHUNKS * 32) mlstm_gates_kernel(const _
 struct MsSmem {  // K [2 stages][2 pieces of 64 dims], u V [2 stages] high and low [2 pieces each: 64 columns; u]
     static constexpr int k = 0, w = 4 * MP_SUB, wbytes = 4 * MP_SUB, total = 12 * MP_SUB;
 };
-__global__ void __launch_bounds__(MP_THREADS) mlstm_state_kernel(const __grid_constant__ MlstmPrefillParams p, const __grid_constant__ CUtensorMap map_k) {
+__global__ void __launch_bounds__(MP_THREADS, 1) mlstm_state_kernel(const __grid_constant__ MlstmPrefillParams p, const __grid_constant__ CUtensorMap map_k) {
     extern __shared__ __align__(1024) uint8_t ms_raw[];
     __shared__ __align__(8) uint64_t s_k[2], s_kfree[2], s_w, s_mma;
     __shared__ uint32_t s_tmem;
@@ -284,7 +284,7 @@ __global__ void __launch_bounds__(MP_THREADS) mlstm_state_kernel(const __grid_co
 }
 
 // Grid (vt, chunks, heads), clusters of vt blocks.
-constexpr int MC_ROWS = 32, MC_BOX = MC_ROWS * 128, MC_SLOT = 4 * MC_BOX, MC_MAX_SLOTS = 4;  // a ring slot: 32 rows of S x 128 columns, both terms
+constexpr int MC_MAX_DP = 320, MC_ROWS = 32, MC_BOX = MC_ROWS * 128, MC_SLOT = 4 * MC_BOX, MC_MAX_SLOTS = 4;  // a ring slot: 32 rows of S x 128 columns, both terms
 struct McSmem {  // Q, K (later A high and low), V, ring of S
     int q, k, v, s, total, qbytes;
 };
@@ -300,11 +300,13 @@ __host__ __device__ inline McSmem mc_smem_layout(int dp, int sstages) {
 }
 __global__ void __launch_bounds__(MP_THREADS, 1) mlstm_chunk_kernel(const __grid_constant__ MlstmPrefillParams p, const __grid_constant__ CUtensorMap map_q,
                                                                  const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
-                                                                 const __grid_constant__ CUtensorMap map_sh, const __grid_constant__ CUtensorMap map_sl) {
+                                                                 const __grid_constant__ CUtensorMap map_sh, const __grid_constant__ CUtensorMap map_sl,
+                                                                 const __grid_constant__ CUtensorMap map_g) {
     extern __shared__ __align__(1024) uint8_t mc_raw[];
-    __shared__ __align__(8) uint64_t s_qk, s_v, s_s[MC_MAX_SLOTS], s_sfree[MC_MAX_SLOTS], s_a, s_p, s_o;
+    __shared__ __align__(8) uint64_t s_qk, s_v, s_s[MC_MAX_SLOTS], s_sfree[MC_MAX_SLOTS], s_a, s_p, s_o, s_gate;
     __shared__ uint32_t s_tmem;
     __shared__ float s_g[MP_L];                     // a of the chunk's tokens
+    __shared__ __align__(16) float s_n[MC_MAX_DP];  // n before the chunk
     __shared__ float s_den[2][MP_L];                // halves' shares of n . q
     __shared__ float s_part[2][MP_L];               // halves' sums of squares
     __shared__ float s_ss[ML_MAX_CLUSTER][MP_L];    // blocks' sums of squares
@@ -321,6 +323,7 @@ __global__ void __launch_bounds__(MP_THREADS, 1) mlstm_chunk_kernel(const __grid
         mbar_init(&s_a, 1);
         mbar_init(&s_p, MP_WARPS);
         mbar_init(&s_o, 1);
+        mbar_init(&s_gate, 1);
         for (int i = 0; i < p.sstages; ++i) {
             mbar_init(s_s + i, 1);
             mbar_init(s_sfree + i, 1);
@@ -359,6 +362,12 @@ __global__ void __launch_bounds__(MP_THREADS, 1) mlstm_chunk_kernel(const __grid
                     tma_load_2d(dst + i * MC_BOX, &map_sh, c0 + 64 * i, row, s_s + s);
                     tma_load_2d(dst + (2 + i) * MC_BOX, &map_sl, c0 + 64 * i, row, s_s + s);
                 }
+            }
+            if (ok && mbar_wait_bounded(&s_o, 0u)) {  // all products are done: the gates take the operands' place
+                mbar_arrive_expect_tx(&s_gate, 2 * MP_SUB);
+                for (int i = 0; i < 2; ++i) tma_load_2d(smem + L.q + i * MP_SUB, &map_g, h * p.vp + c0 + 64 * i, t0, &s_gate);
+            } else {
+                ok = false;
             }
             if (!ok) {
                 atomicExch(p.status, DEV_ERR_TMA_TIMEOUT);
@@ -408,18 +417,19 @@ __global__ void __launch_bounds__(MP_THREADS, 1) mlstm_chunk_kernel(const __grid
         const uint32_t lane_off = (uint32_t)(32 * qd) << 16;
         const size_t at = ((size_t)h * p.nchunk + c) * MP_L;
         if (tid < MP_L) s_g[tid] = __ldg(p.a + at + tid);
+        if (state)
+            for (int i = tid; i < p.dp; i += MP_WARPS * 32) s_n[i] = __ldg(p.sn + ((size_t)c * S.heads + h) * p.dp + i);
         const float M = __ldg(p.mx + at + r), w = __ldg(p.w + at + r), floor = __ldg(p.floor + at + r);
         bool ok = true;
         float den = 0.f;
         partial_sync_2(MP_WARPS * 32);
         if (!__all_sync(0xffffffffu, mbar_wait_bounded(&s_qk, 0u))) ok = false;
         if (state && ok) {  // n . q of this token: the halves take alternate 64-value pieces
-            const float* const n = p.sn + ((size_t)c * S.heads + h) * p.dp;
             for (int j = half; j < nd; j += 2)
-#pragma unroll 1
+#pragma unroll 2
                 for (int i = 0; i < 8 && 64 * j + 8 * i < p.dp; ++i) {
                     const uint4 x = *reinterpret_cast<const uint4*>(smem + L.q + j * MP_SUB + sw128_chunk(r, i));
-                    const float4 a = __ldg(reinterpret_cast<const float4*>(n + 64 * j + 8 * i)), b = __ldg(reinterpret_cast<const float4*>(n + 64 * j + 8 * i) + 1);
+                    const float4 a = *reinterpret_cast<const float4*>(s_n + 64 * j + 8 * i), b = *reinterpret_cast<const float4*>(s_n + 64 * j + 8 * i + 4);
                     den += __uint_as_float(x.x << 16) * a.x + __uint_as_float(x.x & 0xFFFF0000u) * a.y + __uint_as_float(x.y << 16) * a.z + __uint_as_float(x.y & 0xFFFF0000u) * a.w +
                            __uint_as_float(x.z << 16) * b.x + __uint_as_float(x.z & 0xFFFF0000u) * b.y + __uint_as_float(x.w << 16) * b.z + __uint_as_float(x.w & 0xFFFF0000u) * b.w;
                 }
@@ -476,6 +486,7 @@ __global__ void __launch_bounds__(MP_THREADS, 1) mlstm_chunk_kernel(const __grid
             }
         }
         s_part[half][r] = ss;
+        if (ok && !__all_sync(0xffffffffu, mbar_wait_bounded(&s_gate, 0u))) ok = false;
         if (!ok && lane == 0) atomicExch(p.status, DEV_ERR_TMA_TIMEOUT);
         partial_sync_2(MP_WARPS * 32);
     }
@@ -498,36 +509,25 @@ __global__ void __launch_bounds__(MP_THREADS, 1) mlstm_chunk_kernel(const __grid
         const float scale = 1.f / sqrtf(ss / (float)S.vdim + S.eps);
         bf16* const out = static_cast<bf16*>(p.m.out);
         const bool wide = ((S.vdim | p.m.ldo) & 7) == 0;
-        // gates of this warp's 32 tokens, 32 values at a time, through the shared memory that held Q (all products are done)
-        float* const sg = reinterpret_cast<float*>(smem + L.q) + (warp - 2) * (32 * 33);
-        const int tw = t0 + 32 * (warp & 3);
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
-            const int cc = c0 + 32 * half + 64 * i;  // first column within the head
-            if (cc >= S.vdim) continue;              // (uniform over the warp)
-            const bool col_in = cc + lane < S.vdim;
-            const float norm = col_in ? __ldg(p.m.norm + (size_t)h * S.vdim + cc + lane) : 0.f;
-            float x[32];
-            __syncwarp();
-#pragma unroll
-            for (int k = 0; k < 32; ++k) x[k] = tw + k < p.n && col_in ? __ldg(p.m.in + (size_t)(tw + k) * p.m.ld + p.m.off_g + (size_t)h * S.vdim + cc + lane) : 0.f;
-#pragma unroll
-            for (int k = 0; k < 32; ++k) sg[k * 33 + lane] = norm * fast_sigmoid(x[k]);
-            __syncwarp();
+            const int cc = c0 + 32 * half + 64 * i;           // first column within the head
             const int nv = t0 + row < p.n ? S.vdim - cc : 0;  // values of this token to store
             bf16* const dst = out + (size_t)(t0 + row) * p.m.ldo + (size_t)h * S.vdim + cc;
 #pragma unroll
-            for (int k = 0; k < 32; ++k) x[k] = o[i][k] * scale * sg[lane * 33 + k];
-            if (wide) {
+            for (int g = 0; g < 4; ++g) {
+                const uint4 g8 = *reinterpret_cast<const uint4*>(smem + L.q + i * MP_SUB + sw128_chunk(row, 4 * half + g));
+                const float* const x = o[i] + 8 * g;
+                const uint4 v = make_uint4(mul_pack_bf16(g8.x, x[0] * scale, x[1] * scale), mul_pack_bf16(g8.y, x[2] * scale, x[3] * scale),
+                                           mul_pack_bf16(g8.z, x[4] * scale, x[5] * scale), mul_pack_bf16(g8.w, x[6] * scale, x[7] * scale));
+                if (wide) {
+                    if (8 * g < nv) *reinterpret_cast<uint4*>(dst + 8 * g) = v;
+                } else {
+                    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
 #pragma unroll
-                for (int g = 0; g < 4; ++g)
-                    if (8 * g < nv)
-                        *reinterpret_cast<uint4*>(dst + 8 * g) = make_uint4(pack_bf16(x[8 * g], x[8 * g + 1]), pack_bf16(x[8 * g + 2], x[8 * g + 3]),
-                                                                            pack_bf16(x[8 * g + 4], x[8 * g + 5]), pack_bf16(x[8 * g + 6], x[8 * g + 7]));
-            } else {
-#pragma unroll
-                for (int k = 0; k < 32; ++k)
-                    if (k < nv) put(dst + k, x[k]);
+                    for (int k = 0; k < 8; ++k)
+                        if (8 * g + k < nv) dst[8 * g + k] = __ushort_as_bfloat16((unsigned short)(w[k >> 1] >> (16 * (k & 1))));
+                }
             }
         }
     }

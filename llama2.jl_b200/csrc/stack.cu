@@ -404,7 +404,8 @@ struct StackSession {
     // many positions
     float *xr = nullptr, *in = nullptr, *y = nullptr;
     void *act = nullptr, *act2 = nullptr;        // operands of the products, [max_rows][k rounded up to 8]
-    bf16 *pq = nullptr, *pk = nullptr, *pv = nullptr;  // prompt attention: queries; latent attention: expanded keys, transposed values
+    // prompt attention: queries; latent attention: expanded keys, transposed values; differential attention: gates
+    bf16 *pq = nullptr, *pk = nullptr, *pv = nullptr, *pg = nullptr;
     int pv_ld = 0;
     float* aside = nullptr;                      // differential attention: the first map's result
     MlstmPrefillParams mp = {};                  // mLSTM in chunks: buffers (q null: there are none)
@@ -450,7 +451,7 @@ static int head_prefill_kstages(const HeadShape& s, const DeviceInfo& di, bool* 
 // Ring slots of the chunk kernel (0: the heads do not fit the chunked form).
 static int mlstm_prefill_stages(const MlstmShape& s, const DeviceInfo& di) {
     for (int k = MC_MAX_SLOTS; k >= 1; --k)
-        if (mc_smem_layout(up(s.dim, 16), k).total + 1024 <= di.max_smem_optin - 8192) return k;
+        if (up(s.dim, 16) <= MC_MAX_DP && mc_smem_layout(up(s.dim, 16), k).total + 1024 <= di.max_smem_optin - 10 * 1024) return k;
     return 0;
 }
 
@@ -519,7 +520,7 @@ int32_t stack_session_create(const StackModel* m, const StackSessionInfo& info, 
     s->di = di;
     const StackConfig& c = m->cfg;
     int max_in = 1, max_k = c.width, max_k2 = 1;
-    size_t pq = 0, pk = 0, pv = 0, aside = 0, mh = 0, mk = 0, mv = 0, ms = 0;
+    size_t pq = 0, pk = 0, pv = 0, pg = 0, aside = 0, mh = 0, mk = 0, mv = 0, ms = 0;
     s->pv_ld = up(info.seq_len, 8);
     for (size_t i = 0; i < m->layers.size(); ++i) {
         const StackLayerW& w = m->layers[i];
@@ -528,6 +529,7 @@ int32_t stack_session_create(const StackModel* m, const StackSessionInfo& info, 
         if (w.head.heads && head_prefill_kstages(w.head, di)) {
             pq = std::max(pq, (size_t)2 * w.head.heads * up(w.head.dim, 16));
             aside = std::max(aside, (size_t)w.head.heads * w.head.vdim);
+            pg = std::max(pg, (size_t)w.head.heads * w.head.vp);
         }
         if (w.mlstm.heads && mlstm_prefill_stages(w.mlstm, di)) {
             const MlstmShape& sh = w.mlstm;
@@ -588,13 +590,14 @@ int32_t stack_session_create(const StackModel* m, const StackSessionInfo& info, 
         L2B_TRY(alloc(s->pq, T * pq * 2));
         if (pk) L2B_TRY(alloc(s->pk, (size_t)info.seq_len * pk * 2));
         if (pv) L2B_TRY(alloc(s->pv, pv * s->pv_ld * 2));
-        if (aside) L2B_TRY(alloc(s->aside, T * aside * 4));
+        if (aside) L2B_TRY(alloc(s->aside, (size_t)up((int)T, HP_TILE) * aside * 4));
+        if (pg) L2B_TRY(alloc(s->pg, T * pg * 2));
     }
     const size_t nchunk = (T + MP_L - 1) / MP_L;
     if (!m->f32 && info.n_seq == 1 && info.max_rows >= MLSTM_MIN_ROWS && mh && nchunk <= MP_MAX_CHUNKS) {
         MlstmPrefillParams& p = s->mp;
         for (bf16** b : {&p.q, &p.k}) L2B_TRY(alloc(*b, T * mk * 2));
-        L2B_TRY(alloc(p.v, T * mv * 2));
+        for (bf16** b : {&p.v, &p.g}) L2B_TRY(alloc(*b, T * mv * 2));
         for (float** f : {&p.a, &p.mx, &p.w, &p.floor, &p.u}) L2B_TRY(alloc(*f, mh * nchunk * MP_L * 4));
         L2B_TRY(alloc(p.decay, mh * nchunk * 4));
         for (bf16** b : {&p.sh, &p.sl}) L2B_TRY(alloc(*b, nchunk * ms * 2));
@@ -689,7 +692,7 @@ static HeadAttnParams head_params(const StackSession* s, int run, const float* i
 }
 template <typename CT>
 static cudaError_t launch_head_rows(const HeadAttnParams& a, int rows, bool chained, cudaStream_t st) {
-    const int items = 2 * a.s.heads + (a.own_kv ? 3 * a.s.kv_heads : 0);
+    const int items = 2 * a.s.heads + (a.own_kv ? 3 * a.s.kv_heads : 0) + (a.pq ? a.s.heads : 0);
     return launch_kernel(head_rows_kernel<CT>, dim3((items + HA_WARPS - 1) / HA_WARPS, rows), dim3(HA_WARPS * 32), 0, st, chained, a);
 }
 // Differential attention of `rows` rows: query vectors and new cache rows, scan, output.
@@ -754,6 +757,7 @@ static EmbedParams embed_params(const StackModel* m, const int* tokens, float* x
     e.x = x;
     return e;
 }
+static int embed_blocks(int width) { return std::max(1, std::min(16, width % 8 == 0 ? (width + 2047) / 2048 : width / 256)); }
 static int mlp_epilogue(MlpKind k) { return k == MlpKind::GatedSilu ? DE_SWIGLU : DE_GEGLU; }
 
 int32_t stack_enqueue_token(StackSession* s, const int* token, const int* pos, float* logits, float* amax_val, int* amax_idx, int* status, cudaStream_t st,
@@ -763,7 +767,7 @@ int32_t stack_enqueue_token(StackSession* s, const int* token, const int* pos, f
     int count = 0, cur = 0;
     EmbedParams ep = embed_params(m, token, s->x[0]);
     ep.pos = pos;
-    CU(launch_kernel(embed_positions_kernel, dim3(std::max(1, std::min(32, c.width / 256)), 1), dim3(256), 0, st, false, ep));
+    CU(launch_kernel(embed_positions_kernel, dim3(embed_blocks(c.width), 1), dim3(256), 0, st, false, ep));
     ++count;
     const float* add_w = nullptr;  // non-null: y1 awaits its norm (this is its weight) and its place in the residual stream
     const float* step = nullptr;
@@ -1024,6 +1028,7 @@ static int32_t enqueue_head_rows(StackSession* s, int run, int n, int pos0, cons
         });
     a.pq = s->pq;
     a.dq = up(sh.dim, 16);
+    a.pg = s->pg;
     const int lanes = sh.rdims / 8, vectors = 2 * sh.heads + (a.own_kv ? 2 * sh.kv_heads : 0), per = lanes ? HA_WARPS * 32 / lanes : 1;
     if (sh.rdims % 8 == 0 && lanes && (lanes & (lanes - 1)) == 0 && lanes <= 32 && sh.dim % 16 == 0 && sh.vdim % 8 == 0)
         head_rows_quads_kernel<<<dim3((vectors + per - 1) / per, n), HA_WARPS * 32, 0, st>>>(a, lanes);
@@ -1033,12 +1038,13 @@ static int32_t enqueue_head_rows(StackSession* s, int run, int n, int pos0, cons
     memset(&f, 0, sizeof(f));
     f.s = sh; f.n = n; f.pos0 = pos0; f.chunk = a.c.chunk; f.dq = a.dq; f.vn = up(sh.vdim, 16); f.kstages = kstages;
     f.paired = two && blocks > s->di.sms && blocks <= 2 * s->di.sms ? s->di.sms : 0;
-    f.gate = a.in + a.off_g; f.ld = a.ld; f.aside = s->aside; f.out = static_cast<bf16*>(s->act2); f.ldo = ldo; f.status = status;
-    CUtensorMap mq, mkv;
+    f.aside = s->aside; f.out = static_cast<bf16*>(s->act2); f.ldo = ldo; f.status = status;
+    CUtensorMap mq, mkv, mg;
     L2B_TRY(bf16_map(mq, s->pq, (int64_t)2 * sh.heads * a.dq, n, (int64_t)2 * sh.heads * a.dq, HP_TILE));
     L2B_TRY(bf16_map(mkv, static_cast<const bf16*>(a.c.cache), sh.row, pos0 + n, sh.row, HP_TILE, sh.kv_heads, (int64_t)a.c.group_stride));
+    L2B_TRY(bf16_map(mg, s->pg, (int64_t)sh.heads * sh.vp, n, (int64_t)sh.heads * sh.vp, HP_TILE));
     const size_t smem = (size_t)hp_smem_layout(sh.dim, f.vn, kstages).total + 1024;
-    CU(launch_kernel_args(head_prefill_kernel, dim3(blocks), dim3(HP_THREADS), smem, st, false, 1, f, mq, mkv));
+    CU(launch_kernel_args(head_prefill_kernel, dim3(blocks), dim3(HP_THREADS), smem, st, false, 1, f, mq, mkv, mg));
     *launches += 2;
     return L2B_OK;
 }
@@ -1066,11 +1072,12 @@ static int32_t enqueue_mlstm_rows(StackSession* s, int run, int n, int pos0, con
         p.sstages = stages;
         p.status = status;
         for (p.vt = 1; p.vt * MP_COLS < sh.vdim;) p.vt *= 2;
-        CUtensorMap mq, mk, mv, msh, msl;
+        CUtensorMap mq, mk, mv, msh, msl, mg;
         const int64_t nk = (int64_t)sh.heads * p.dp, nv = (int64_t)sh.heads * p.vp, rows = (int64_t)p.nchunk * sh.heads * p.dp;
         L2B_TRY(bf16_map(mq, p.q, nk, n, nk, MP_L));
         L2B_TRY(bf16_map(mk, p.k, nk, n, nk, MP_L));
         L2B_TRY(bf16_map(mv, p.v, nv, n, nv, MP_L));
+        L2B_TRY(bf16_map(mg, p.g, nv, n, nv, MP_L));
         L2B_TRY(bf16_map(msh, p.sh, p.vs, rows, p.vs, MC_ROWS));
         L2B_TRY(bf16_map(msl, p.sl, p.vs, rows, p.vs, MC_ROWS));
         mlstm_operands_kernel<<<n, 256, 0, st>>>(p);
@@ -1079,7 +1086,7 @@ static int32_t enqueue_mlstm_rows(StackSession* s, int run, int n, int pos0, con
         CU(cudaGetLastError());
         const dim3 sgrid((sh.vdim + MP_STATE_COLS - 1) / MP_STATE_COLS, (sh.dim + 127) / 128, sh.heads), cgrid(p.vt, p.nchunk, sh.heads);
         CU(launch_kernel_args(mlstm_state_kernel, sgrid, dim3(MP_THREADS), (size_t)MsSmem::total + 1024, st, false, 1, p, mk));
-        CU(launch_kernel_args(mlstm_chunk_kernel, cgrid, dim3(MP_THREADS), (size_t)mc_smem_layout(p.dp, stages).total + 1024, st, false, p.vt, p, mq, mk, mv, msh, msl));
+        CU(launch_kernel_args(mlstm_chunk_kernel, cgrid, dim3(MP_THREADS), (size_t)mc_smem_layout(p.dp, stages).total + 1024, st, false, p.vt, p, mq, mk, mv, msh, msl, mg));
         *launches += 4;
         return L2B_OK;
     }
@@ -1097,7 +1104,7 @@ int32_t stack_enqueue_rows(StackSession* s, const int* dev_tokens, int n, int po
     EmbedParams ep = embed_params(m, dev_tokens, s->xr);
     ep.pos0 = pos0;
     ep.pos_list = pos_list;
-    CU(launch_kernel(embed_positions_kernel, dim3(std::max(1, std::min(16, c.width / 256)), n), dim3(256), 0, st, false, ep));
+    CU(launch_kernel(embed_positions_kernel, dim3(embed_blocks(c.width), n), dim3(256), 0, st, false, ep));
     ++count;
     const int lda = up(c.width, 8);
     const float* add_w = nullptr;  // non-null: y awaits its norm (this is its weight) and its place in the residual stream

@@ -27,9 +27,28 @@ __global__ void embed_positions_kernel(const __grid_constant__ EmbedParams p) {
     const bool valid = tok >= 0 && tok < p.vocab;
     const int pos = p.pos ? __ldcg(p.pos) : p.pos_list ? __ldcg(p.pos_list + row) : p.pos0 + row;
     const bf16* const pv = p.pos_table && pos >= 0 && pos < p.max_positions ? p.pos_table + (size_t)pos * p.width : nullptr;
-    for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < p.width; i += gridDim.x * blockDim.x) {
-        const float e = valid ? p.scale * __bfloat162float(p.table[(size_t)tok * p.width + i]) : 0.f;
-        p.x[(size_t)row * p.width + i] = pv ? e + __bfloat162float(pv[i]) : e;
+    const int first = blockIdx.x * blockDim.x + threadIdx.x, step = gridDim.x * blockDim.x;
+    float* const x = p.x + (size_t)row * p.width;
+    const bf16* const tv = p.table + (size_t)(valid ? tok : 0) * p.width;
+    if ((p.width & 7) == 0) {  // eight values at a time
+        const float scale = valid ? p.scale : 0.f;
+        for (int i = first; i < p.width / 8; i += step) {
+            const uint4 a = __ldg(reinterpret_cast<const uint4*>(tv) + i), b = pv ? __ldg(reinterpret_cast<const uint4*>(pv) + i) : make_uint4(0u, 0u, 0u, 0u);
+            const uint32_t e[4] = {a.x, a.y, a.z, a.w}, q[4] = {b.x, b.y, b.z, b.w};
+            float v[8];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+                v[2 * k] = scale * __uint_as_float(e[k] << 16) + __uint_as_float(q[k] << 16);
+                v[2 * k + 1] = scale * __uint_as_float(e[k] & 0xFFFF0000u) + __uint_as_float(q[k] & 0xFFFF0000u);
+            }
+            reinterpret_cast<float4*>(x)[2 * i] = make_float4(v[0], v[1], v[2], v[3]);
+            reinterpret_cast<float4*>(x)[2 * i + 1] = make_float4(v[4], v[5], v[6], v[7]);
+        }
+        return;
+    }
+    for (int i = first; i < p.width; i += step) {
+        const float e = valid ? p.scale * __bfloat162float(tv[i]) : 0.f;
+        x[i] = pv ? e + __bfloat162float(pv[i]) : e;
     }
 }
 
