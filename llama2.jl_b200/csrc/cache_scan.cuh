@@ -60,7 +60,7 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], 
 __device__ __forceinline__ void ldmatrix4_trans(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
-// Grid (nsplit * blocks of 16 heads, rows).  N: K = 16 steps of a cache row, and pairs of 8-column tiles of the summed columns, per warp at most.
+// Grid (nsplit, blocks of 16 heads, rows).  N: K = 16 steps of a cache row, and pairs of 8-column tiles of the summed columns, per warp at most.
 template <int N>
 __global__ void __launch_bounds__(CS_SCAN_THREADS) cache_scan_mma_kernel(const __grid_constant__ CacheScan p) {
     extern __shared__ __align__(128) uint8_t cs_ring[];  // [stages][CS_STAGE_ROWS][pitch]
@@ -69,9 +69,9 @@ __global__ void __launch_bounds__(CS_SCAN_THREADS) cache_scan_mma_kernel(const _
     __shared__ __align__(16) uint32_t s_hi[CS_MMA_HEADS][12], s_lo[CS_MMA_HEADS][12];  // weights of a stage: 16 bf16 per head (rows padded)
     __shared__ float s_corr[CS_MMA_HEADS];
     constexpr int KS = N, NT = N;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, row = (int)blockIdx.y;
-    const int split = (int)blockIdx.x % p.nsplit, per = (p.per_group + CS_MMA_HEADS - 1) / CS_MMA_HEADS, gb = (int)blockIdx.x / p.nsplit;
-    const int group = gb / per, h0 = group * p.per_group + gb % per * CS_MMA_HEADS, h1 = (group + 1) * p.per_group;  // heads h0 .. of this group
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, row = (int)blockIdx.z;
+    const int split = (int)blockIdx.x, per = (p.per_group + CS_MMA_HEADS - 1) / CS_MMA_HEADS, group = per == 1 ? (int)blockIdx.y : (int)blockIdx.y / per;
+    const int h0 = group * p.per_group + ((int)blockIdx.y - group * per) * CS_MMA_HEADS, h1 = (group + 1) * p.per_group;  // heads h0 .. of this group
     const int pitch = cs_pitch(p.row), stage_bytes = cs_mma_stage_bytes(p.row);
     pdl_launch_dependents();
     if (tid == 0) {
@@ -216,15 +216,15 @@ __global__ void __launch_bounds__(CS_SCAN_THREADS) cache_scan_mma_kernel(const _
 }
 
 // ---- scan on the CUDA cores ---------------------------------------------------------------------------------------
-// Grid (nsplit * blocks of 8 heads, rows).  NI: 256-value pieces a cache row is spread over (32 lanes x 8 values each).
+// Grid (nsplit, blocks of 8 heads, rows).  NI: 256-value pieces a cache row is spread over (32 lanes x 8 values each).
 template <typename CT, int NI>
 __global__ void __launch_bounds__(CS_SCAN_THREADS) cache_scan_kernel(const __grid_constant__ CacheScan p) {
     extern __shared__ __align__(128) uint8_t cs_ring[];  // [stages][CS_STAGE_ROWS][row] of CT
     __shared__ __align__(8) uint64_t s_full[CS_MAX_STAGES], s_empty[CS_MAX_STAGES];
     constexpr int BATCH = NI <= 3 ? 4 : 2;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, row = (int)blockIdx.y;
-    const int split = (int)blockIdx.x % p.nsplit, per = (p.per_group + CS_WARPS - 1) / CS_WARPS, gb = (int)blockIdx.x / p.nsplit;
-    const int group = gb / per, hg = gb % per * CS_WARPS + warp, h = group * p.per_group + hg;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, row = (int)blockIdx.z;
+    const int split = (int)blockIdx.x, per = (p.per_group + CS_WARPS - 1) / CS_WARPS, group = per == 1 ? (int)blockIdx.y : (int)blockIdx.y / per;
+    const int hg = ((int)blockIdx.y - group * per) * CS_WARPS + warp, h = group * p.per_group + hg;
     pdl_launch_dependents();
     if (tid == 0) {
         for (int i = 0; i < p.stages; ++i) {

@@ -62,11 +62,12 @@ __device__ __forceinline__ void epilogue_tokens(const DenseEpilogue& e, int t0, 
             dst[k] = make_uint4(w[0], w[1], w[2], w[3]);
         }
     } else {
-        const float bias = KIND == DE_STORE && e.bias ? __ldg(e.bias + f) : 0.f;
+        const float bias = KIND == DE_AFFINE && e.bias ? __ldg(e.bias + f) : 0.f;
 #pragma unroll
         for (int k = 0; k < 32; ++k) {
             if (k >= n) continue;
-            if (KIND == DE_STORE) e.y[(size_t)(t0 + k) * e.ld + f] = fmaf(v[k], e.mul, bias);
+            if (KIND == DE_STORE) e.y[(size_t)(t0 + k) * e.ld + f] = v[k];
+            if (KIND == DE_AFFINE) e.y[(size_t)(t0 + k) * e.ld + f] = fmaf(v[k], e.mul, bias);
             if (KIND == DE_SWIGLU) put(act + (size_t)(t0 + k) * e.ld + f, silu(v[k]) * v2[k]);
             if (KIND == DE_GEGLU) put(act + (size_t)(t0 + k) * e.ld + f, gelu_tanh(v[k]) * v2[k]);
             if (KIND == DE_STORE_ACT) put(act + (size_t)(t0 + k) * e.ld + f, v[k]);
@@ -79,6 +80,7 @@ __device__ __forceinline__ void epilogue_tokens(const DenseEpilogue& e, int t0, 
         case DE_RESIDUAL: epilogue_tokens<DE_RESIDUAL>(e, t0, n, f, v, v2); break;
         case DE_GEGLU: epilogue_tokens<DE_GEGLU>(e, t0, n, f, v, v2); break;
         case DE_SWIGLU: epilogue_tokens<DE_SWIGLU>(e, t0, n, f, v, v2); break;
+        case DE_AFFINE: epilogue_tokens<DE_AFFINE>(e, t0, n, f, v, v2); break;
         case DE_SIDE: epilogue_tokens<DE_SIDE>(e, t0, n, f, v, v2); break;
         case DE_STORE_ACT: epilogue_tokens<DE_STORE_ACT>(e, t0, n, f, v, v2); break;
         case DE_STORE_T: epilogue_tokens<DE_STORE_T>(e, t0, n, f, v, v2); break;

@@ -39,7 +39,7 @@ struct DmvParams {
     float* x_out;           // block 0 writes the updated vector here (null: no update)
     NormParams norm;
     DenseEpilogue epi;      // t = 0
-    float* amax_val;        // DE_LOGITS: per block
+    float* amax_val;        // DE_LOGITS, DE_AFFINE_LOGITS: per block
     int* amax_idx;
     int* status;
 };
@@ -55,6 +55,8 @@ inline int dmv_choose_stages(const DmvParams& p, size_t max_smem) {
     return (int)std::min<long>(DMV_MAX_STAGES, std::min<long>(fit, std::max<long>(use, 2)));
 }
 
+// RMS: the norm in front is an rms norm (else none, or dynamic tanh).
+template <bool RMS>
 __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __grid_constant__ DmvParams p) {
     extern __shared__ __align__(128) uint8_t dmv_smem[];
     __shared__ __align__(8) uint64_t s_full[DMV_MAX_STAGES], s_empty[DMV_MAX_STAGES];
@@ -63,6 +65,7 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
     float* const xf = reinterpret_cast<float*>(dmv_smem + p.stages * DMV_STAGE);
     float* const part = xf + p.nchunk * 256;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const bool logits = p.epi.kind == DE_LOGITS || p.epi.kind == DE_AFFINE_LOGITS;
     pdl_launch_dependents();
     if (threadIdx.x == 0) {
         for (int i = 0; i < p.stages; ++i) {
@@ -117,7 +120,7 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
             for (int i = 0; i < 2000; ++i) __nanosleep(1000);  // copies in flight land within microseconds
         }
         __syncthreads();
-        if (p.epi.kind == DE_LOGITS) __syncthreads();
+        if (logits) __syncthreads();
         return;
     }
 
@@ -153,14 +156,14 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
                     if (p.upd.y) t = fmaf(xf[at] * scale, __ldg(p.upd.w + i), t);
                     if (p.upd.step) t += __ldg(p.upd.step + i);
                     if (p.x_out && b == 0) p.x_out[i] = t;
-                    xs = fmaf(t, t, xs);
-                    xf[at] = apply_norm(p.norm, t, i);
+                    if (RMS) xs = fmaf(t, t, xs);
+                    xf[at] = apply_norm<RMS>(p.norm, t, i);
                 } else if (i < kc) {
                     xf[at] = 0.f;
                 }
             }
         }
-        if (p.norm.kind == NORM_RMS) {
+        if (RMS) {
             xs = warp_sum(xs);
             if (lane == 0) s_ss[warp] = xs;  // (read after the last barrier)
         }
@@ -227,7 +230,7 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
     __syncthreads();
 
     float rms_scale = 1.f;
-    if (p.norm.kind == NORM_RMS) {
+    if (RMS) {
         float ss = 0.f;
 #pragma unroll
         for (int i = 0; i < DMV_WARPS; ++i) ss += s_ss[i];
@@ -241,16 +244,15 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
         for (int s = 0; s < p.cs; ++s) v += pr[s];
         if (p.unit == 2)
             for (int s = 0; s < p.cs; ++s) v2 += pr[p.cs + s];
-        v *= rms_scale;
-        v2 *= rms_scale;
+        if (RMS) v *= rms_scale, v2 *= rms_scale;
         dense_epilogue<float>(p.epi, 0, u0 + u, v, v2);
-        if (p.epi.kind == DE_LOGITS) v = scaled_biased(p.epi, u0 + u, v);
+        if (p.epi.kind == DE_AFFINE_LOGITS) v = affine(p.epi, u0 + u, v);
         if (v > best) {
             best = v;
             best_i = u0 + u;
         }
     }
-    if (p.epi.kind != DE_LOGITS) return;
+    if (!logits) return;
     auto better = [](float v, int i, float w, int j) { return v > w || (v == w && i < j); };
     for (int o = 16; o > 0; o >>= 1) {
         const float ov = __shfl_xor_sync(0xffffffffu, best, o);

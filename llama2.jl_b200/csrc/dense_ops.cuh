@@ -137,12 +137,14 @@ enum : int {
     DE_LOGITS = 4,    // as DE_STORE, and the block's first maximum
     DE_STORE_ACT = 5, // act[t][f]
     DE_STORE_T = 6,   // act[f][t] (transposed)
-    DE_SWIGLU = 7     // act[t][f] = silu(gate) * up (two weight rows per result)
+    DE_SWIGLU = 7,    // act[t][f] = silu(gate) * up (two weight rows per result)
+    DE_AFFINE = 8,    // y[t][f] = mul * v + bias[f]
+    DE_AFFINE_LOGITS = 9  // as DE_AFFINE, and the block's first maximum
 };
 struct DenseEpilogue {
     int kind;
-    float mul;            // DE_STORE, DE_LOGITS: factor of the product, and
-    const float* bias;    // what is added to it per result (null: nothing)
+    float mul;            // DE_AFFINE, DE_AFFINE_LOGITS
+    const float* bias;    // the same (null: nothing)
     float* y;
     void* act;
     int ld;               // elements between rows of y / act
@@ -154,13 +156,18 @@ struct DenseEpilogue {
 inline DenseEpilogue dense_epilogue_of(int kind, float* y, void* act, int ld) {
     DenseEpilogue e = {};
     e.kind = kind;
-    e.mul = 1.f;
     e.y = y;
     e.act = act;
     e.ld = ld;
     return e;
 }
-__device__ __forceinline__ float scaled_biased(const DenseEpilogue& e, int f, float v) { return e.bias ? fmaf(v, e.mul, __ldg(e.bias + f)) : v * e.mul; }
+inline DenseEpilogue affine_epilogue(int kind, float mul, const float* bias, float* y, int ld) {
+    DenseEpilogue e = dense_epilogue_of(kind, y, nullptr, ld);
+    e.mul = mul;
+    e.bias = bias;
+    return e;
+}
+__device__ __forceinline__ float affine(const DenseEpilogue& e, int f, float v) { return e.bias ? fmaf(v, e.mul, __ldg(e.bias + f)) : v * e.mul; }
 __device__ __forceinline__ float side_value(const DenseEpilogue& e, int t, int f) {
     const int tok = __ldg(e.tokens + t);
     const bool valid = tok >= 0 && tok < e.vocab;  // (the load does not depend on it: several are in flight together)
@@ -172,13 +179,14 @@ __device__ __forceinline__ void dense_epilogue(const DenseEpilogue& e, int t, in
     const size_t o = (size_t)t * e.ld + f;
     AT* act = static_cast<AT*>(e.act);
     switch (e.kind) {
-        case DE_STORE: case DE_LOGITS: e.y[o] = scaled_biased(e, f, v); break;
+        case DE_STORE: case DE_LOGITS: e.y[o] = v; break;
         case DE_RESIDUAL: e.y[o] += v; break;
         case DE_GEGLU: put(act + o, gelu_tanh(v) * v2); break;
         case DE_SIDE: put(act + o, gelu_tanh(v) * side_value(e, t, f)); break;
         case DE_STORE_ACT: put(act + o, v); break;
         case DE_STORE_T: put(act + (size_t)f * e.ld + t, v); break;
         case DE_SWIGLU: put(act + o, silu(v) * v2); break;
+        case DE_AFFINE: case DE_AFFINE_LOGITS: e.y[o] = affine(e, f, v); break;
     }
 }
 
@@ -199,8 +207,10 @@ struct NormParams {
     const float* b;       // dynamic tanh
 };
 // One value; rms: without the factor 1 / rms(x).
+template <bool RMS>
 __device__ __forceinline__ float apply_norm(const NormParams& n, float x, int i) {
-    return n.kind == NORM_DYNAMIC_TANH ? dynamic_tanh(x, n.alpha, __ldg(n.w + i), __ldg(n.b + i)) : n.kind == NORM_RMS ? x * __ldg(n.w + i) : x;
+    if (RMS) return x * __ldg(n.w + i);
+    return n.kind ? dynamic_tanh(x, n.alpha, __ldg(n.w + i), __ldg(n.b + i)) : x;
 }
 
 // Barrier over the first `threads` threads of the block.

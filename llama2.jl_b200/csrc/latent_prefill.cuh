@@ -254,7 +254,7 @@ __global__ void __launch_bounds__(LP_THREADS) latent_prefill_kernel(const __grid
                     o[i] = t < p.n && c + lane < p.vdim ? __ldg(p.gate + (size_t)t * p.ld + h * p.vdim + c + lane) : 0.f;
                 }
 #pragma unroll
-                for (int i = 0; i < 32; ++i) sg[i * 33 + lane] = fast_sigmoid(o[i]);
+                for (int i = 0; i < 32; ++i) sg[i * 33 + lane] = sigmoid(o[i]);
                 __syncwarp();
                 tmem_ld32f(tmem_o + lane_off + (uint32_t)c, o);
                 const int nv = qi < p.n ? p.vdim - c : 0;  // values of this query to store

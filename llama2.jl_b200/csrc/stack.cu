@@ -468,7 +468,8 @@ static int32_t set_stack_kernel_attrs() {
             if (e == cudaSuccess) e = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, optin - (int)fa.sharedSizeBytes);
             if (e != cudaSuccess) g_stack_attr_err = e;
         };
-        set((const void*)dense_matvec_kernel);
+        set((const void*)dense_matvec_kernel<false>);
+        set((const void*)dense_matvec_kernel<true>);
         set((const void*)latent_prefill_kernel);
         set((const void*)head_prefill_kernel);
         set((const void*)mlstm_state_kernel);
@@ -639,7 +640,7 @@ static void plan_scan(CacheScan& c, bool f32, int rows, const DeviceInfo& di) {
     c.stages = std::max(1, std::min(CS_MAX_STAGES, (di.max_smem_optin - 16 * 1024) / stage));
 }
 static cudaError_t launch_scan(const CacheScan& c, bool f32, int rows, cudaStream_t st) {
-    const dim3 grid(scan_blocks(c, f32) * c.nsplit, rows), block(CS_SCAN_THREADS);
+    const dim3 grid(c.nsplit, scan_blocks(c, f32), rows), block(CS_SCAN_THREADS);
     const size_t smem = (size_t)c.stages * (f32 ? CS_STAGE_ROWS * c.row * 4 : cs_mma_stage_bytes(c.row));
     auto go = [&](auto k) { return launch_kernel(k, grid, block, smem, st, true, c); };
     if (f32) {
@@ -744,7 +745,7 @@ static int32_t launch_dense_matvec(const StackSession* s, const StackMatrix& w, 
     p.stages = dmv_choose_stages(p, (size_t)s->di.max_smem_optin - 2048);
     if (p.stages < 2) return fail(L2B_ERR_BAD_ARG, "input vector too long for shared memory");
     const size_t smem = (size_t)p.stages * DMV_STAGE + dmv_fixed_bytes(p);
-    CU(launch_kernel(dense_matvec_kernel, dim3(grid), dim3(DMV_THREADS), smem, st, true, p));
+    CU(launch_kernel(p.norm.kind == NORM_RMS ? dense_matvec_kernel<true> : dense_matvec_kernel<false>, dim3(grid), dim3(DMV_THREADS), smem, st, true, p));
     if (nblocks) *nblocks = grid;
     return L2B_OK;
 }
@@ -810,9 +811,7 @@ int32_t stack_enqueue_token(StackSession* s, const int* token, const int* pos, f
         const StackLayerW& w = m->layers[l];
         if (m->runs[r].pass >= 0) step = m->loop_step + (size_t)m->runs[r].pass * c.width;
         from_residual(p, &w.norm1);
-        DenseEpilogue proj = dense_epilogue_of(DE_STORE, s->in1, nullptr, 0);
-        proj.bias = w.in_bias;
-        L2B_TRY(mv_epi(w.in, p, proj));
+        L2B_TRY(mv_epi(w.in, p, w.in_bias ? affine_epilogue(DE_AFFINE, 1.f, w.in_bias, s->in1, 0) : dense_epilogue_of(DE_STORE, s->in1, nullptr, 0)));
         switch (c.layers[l].mix.kind) {
             case MixerKind::LatentAttention: {
                 LatentAttnParams a = latent_params(s, (int)r, s->in1);
@@ -872,9 +871,7 @@ int32_t stack_enqueue_token(StackSession* s, const int* token, const int* pos, f
     s->x_last = cur;
     p.amax_val = amax_val;
     p.amax_idx = amax_idx;
-    DenseEpilogue e = dense_epilogue_of(DE_LOGITS, logits, nullptr, 0);
-    e.mul = c.logit_scale;
-    L2B_TRY(mv_epi(m->head, p, e, nparts));
+    L2B_TRY(mv_epi(m->head, p, c.logit_scale == 1.f ? dense_epilogue_of(DE_LOGITS, logits, nullptr, 0) : affine_epilogue(DE_AFFINE_LOGITS, c.logit_scale, nullptr, logits, 0), nparts));
     if (nlaunch) *nlaunch = count;
     return L2B_OK;
 }
@@ -1145,9 +1142,7 @@ int32_t stack_enqueue_rows(StackSession* s, const int* dev_tokens, int n, int po
         const StackLayerW& w = m->layers[l];
         if (m->runs[r].pass >= 0) step = m->loop_step + (size_t)m->runs[r].pass * c.width;
         L2B_TRY(from_residual(&w.norm1, true));
-        DenseEpilogue proj = dense_epilogue_of(DE_STORE, s->in, nullptr, w.in.rows);
-        proj.bias = w.in_bias;
-        L2B_TRY(gemm_epi(w.in, s->act, proj));
+        L2B_TRY(gemm_epi(w.in, s->act, w.in_bias ? affine_epilogue(DE_AFFINE, 1.f, w.in_bias, s->in, w.in.rows) : dense_epilogue_of(DE_STORE, s->in, nullptr, w.in.rows)));
         switch (c.layers[l].mix.kind) {
             case MixerKind::LatentAttention: L2B_TRY(enqueue_latent_rows(s, (int)r, n, pos0, pos_list, up(w.o.k, 8), status, st, &count)); break;
             case MixerKind::DifferentialAttention: L2B_TRY(enqueue_head_rows(s, (int)r, n, pos0, pos_list, up(w.o.k, 8), status, st, &count)); break;
@@ -1188,8 +1183,7 @@ int32_t stack_enqueue_logits(StackSession* s, const int* dev_index, int n, float
     r.act = s->act;
     r.lda = up(m->cfg.width, 8);
     L2B_TRY(launch_residual_rows(s, r, n, st));
-    DenseEpilogue e = dense_epilogue_of(DE_STORE, logits, nullptr, m->cfg.vocab);
-    e.mul = m->cfg.logit_scale;
+    const DenseEpilogue e = m->cfg.logit_scale == 1.f ? dense_epilogue_of(DE_STORE, logits, nullptr, m->cfg.vocab) : affine_epilogue(DE_AFFINE, m->cfg.logit_scale, nullptr, logits, m->cfg.vocab);
     L2B_TRY(launch_gemm(s, m->head, s->act, r.lda, n, e, status, st));
     if (launches) *launches += 2;
     return L2B_OK;

@@ -96,7 +96,8 @@ __global__ void __launch_bounds__(256) residual_rows_kernel(const __grid_constan
         return t;
     };
     float rms_scale = 1.f;
-    if (act && p.norm.kind == NORM_RMS) {  // (the second pass finds its inputs in the first-level cache)
+    const bool rms = p.norm.kind == NORM_RMS;
+    if (act && rms) {  // (the second pass finds its inputs in the first-level cache)
         float ss = 0.f;
         for (int i = threadIdx.x; i < n; i += 256) {
             const F t = updated(i);
@@ -111,7 +112,7 @@ __global__ void __launch_bounds__(256) residual_rows_kernel(const __grid_constan
         if (act) {
             A o;
 #pragma unroll
-            for (int k = 0; k < V; ++k) put(&o.v[k], apply_norm(p.norm, t.v[k], i * V + k) * rms_scale);
+            for (int k = 0; k < V; ++k) put(&o.v[k], rms ? apply_norm<true>(p.norm, t.v[k], i * V + k) * rms_scale : apply_norm<false>(p.norm, t.v[k], i * V + k));
             act[i] = o;
         }
     }
