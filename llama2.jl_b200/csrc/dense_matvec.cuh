@@ -55,8 +55,10 @@ inline int dmv_choose_stages(const DmvParams& p, size_t max_smem) {
     return (int)std::min<long>(DMV_MAX_STAGES, std::min<long>(fit, std::max<long>(use, 2)));
 }
 
-// RMS: the norm in front is an rms norm (else none, or dynamic tanh).
-template <bool RMS>
+// RMS: the norm in front is an rms norm (else none, or dynamic tanh).  KINDS: one of the sets of epilogues below.
+constexpr unsigned DMV_KINDS_GELU = 1u << DE_STORE | 1u << DE_RESIDUAL | 1u << DE_LOGITS | 1u << DE_GEGLU | 1u << DE_SIDE;
+constexpr unsigned DMV_KINDS_SILU = 1u << DE_STORE | 1u << DE_RESIDUAL | 1u << DE_LOGITS | 1u << DE_SWIGLU | 1u << DE_AFFINE | 1u << DE_AFFINE_LOGITS;
+template <bool RMS, unsigned KINDS>
 __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __grid_constant__ DmvParams p) {
     extern __shared__ __align__(128) uint8_t dmv_smem[];
     __shared__ __align__(8) uint64_t s_full[DMV_MAX_STAGES], s_empty[DMV_MAX_STAGES];
@@ -65,7 +67,7 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
     float* const xf = reinterpret_cast<float*>(dmv_smem + p.stages * DMV_STAGE);
     float* const part = xf + p.nchunk * 256;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const bool logits = p.epi.kind == DE_LOGITS || p.epi.kind == DE_AFFINE_LOGITS;
+    const bool logits = p.epi.kind == DE_LOGITS || ((KINDS >> DE_AFFINE_LOGITS & 1) && p.epi.kind == DE_AFFINE_LOGITS);
     pdl_launch_dependents();
     if (threadIdx.x == 0) {
         for (int i = 0; i < p.stages; ++i) {
@@ -245,8 +247,8 @@ __global__ void __launch_bounds__(DMV_THREADS, 2) dense_matvec_kernel(const __gr
         if (p.unit == 2)
             for (int s = 0; s < p.cs; ++s) v2 += pr[p.cs + s];
         if (RMS) v *= rms_scale, v2 *= rms_scale;
-        dense_epilogue<float>(p.epi, 0, u0 + u, v, v2);
-        if (p.epi.kind == DE_AFFINE_LOGITS) v = affine(p.epi, u0 + u, v);
+        dense_epilogue<float, KINDS>(p.epi, 0, u0 + u, v, v2);
+        if ((KINDS >> DE_AFFINE_LOGITS & 1) && p.epi.kind == DE_AFFINE_LOGITS) v = affine(p.epi, u0 + u, v);
         if (v > best) {
             best = v;
             best_i = u0 + u;

@@ -174,19 +174,21 @@ __device__ __forceinline__ float side_value(const DenseEpilogue& e, int t, int f
     const float v = __bfloat162float(e.etab[(size_t)(valid ? tok : 0) * e.e_ld + e.e_off + f]);
     return valid ? v : 0.f;
 }
-template <typename AT>
+// KINDS: bits of the kinds a kernel may meet (code for kinds that a short kernel never meets costs it time).
+constexpr unsigned DE_EVERY = ~0u;
+template <typename AT, unsigned KINDS = DE_EVERY>
 __device__ __forceinline__ void dense_epilogue(const DenseEpilogue& e, int t, int f, float v, float v2) {
     const size_t o = (size_t)t * e.ld + f;
     AT* act = static_cast<AT*>(e.act);
     switch (e.kind) {
         case DE_STORE: case DE_LOGITS: e.y[o] = v; break;
         case DE_RESIDUAL: e.y[o] += v; break;
-        case DE_GEGLU: put(act + o, gelu_tanh(v) * v2); break;
-        case DE_SIDE: put(act + o, gelu_tanh(v) * side_value(e, t, f)); break;
-        case DE_STORE_ACT: put(act + o, v); break;
-        case DE_STORE_T: put(act + (size_t)f * e.ld + t, v); break;
-        case DE_SWIGLU: put(act + o, silu(v) * v2); break;
-        case DE_AFFINE: case DE_AFFINE_LOGITS: e.y[o] = affine(e, f, v); break;
+        case DE_GEGLU: if (KINDS >> DE_GEGLU & 1) put(act + o, gelu_tanh(v) * v2); break;
+        case DE_SIDE: if (KINDS >> DE_SIDE & 1) put(act + o, gelu_tanh(v) * side_value(e, t, f)); break;
+        case DE_STORE_ACT: if (KINDS >> DE_STORE_ACT & 1) put(act + o, v); break;
+        case DE_STORE_T: if (KINDS >> DE_STORE_T & 1) put(act + (size_t)f * e.ld + t, v); break;
+        case DE_SWIGLU: if (KINDS >> DE_SWIGLU & 1) put(act + o, silu(v) * v2); break;
+        case DE_AFFINE: case DE_AFFINE_LOGITS: if (KINDS >> DE_AFFINE & 1) e.y[o] = affine(e, f, v); break;
     }
 }
 

@@ -468,8 +468,8 @@ static int32_t set_stack_kernel_attrs() {
             if (e == cudaSuccess) e = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, optin - (int)fa.sharedSizeBytes);
             if (e != cudaSuccess) g_stack_attr_err = e;
         };
-        set((const void*)dense_matvec_kernel<false>);
-        set((const void*)dense_matvec_kernel<true>);
+        set((const void*)dense_matvec_kernel<false, DMV_KINDS_GELU>); set((const void*)dense_matvec_kernel<true, DMV_KINDS_GELU>);
+        set((const void*)dense_matvec_kernel<false, DMV_KINDS_SILU>); set((const void*)dense_matvec_kernel<true, DMV_KINDS_SILU>);
         set((const void*)latent_prefill_kernel);
         set((const void*)head_prefill_kernel);
         set((const void*)mlstm_state_kernel);
@@ -745,7 +745,11 @@ static int32_t launch_dense_matvec(const StackSession* s, const StackMatrix& w, 
     p.stages = dmv_choose_stages(p, (size_t)s->di.max_smem_optin - 2048);
     if (p.stages < 2) return fail(L2B_ERR_BAD_ARG, "input vector too long for shared memory");
     const size_t smem = (size_t)p.stages * DMV_STAGE + dmv_fixed_bytes(p);
-    CU(launch_kernel(p.norm.kind == NORM_RMS ? dense_matvec_kernel<true> : dense_matvec_kernel<false>, dim3(grid), dim3(DMV_THREADS), smem, st, true, p));
+    const bool rms = p.norm.kind == NORM_RMS;
+    if (!(DMV_KINDS_GELU >> p.epi.kind & 1) && !(DMV_KINDS_SILU >> p.epi.kind & 1)) return fail(L2B_ERR_BAD_ARG, "the matrix-vector kernel has no such epilogue");
+    CU(launch_kernel(DMV_KINDS_GELU >> p.epi.kind & 1 ? (rms ? dense_matvec_kernel<true, DMV_KINDS_GELU> : dense_matvec_kernel<false, DMV_KINDS_GELU>)
+                                                      : (rms ? dense_matvec_kernel<true, DMV_KINDS_SILU> : dense_matvec_kernel<false, DMV_KINDS_SILU>),
+                     dim3(grid), dim3(DMV_THREADS), smem, st, true, p));
     if (nblocks) *nblocks = grid;
     return L2B_OK;
 }
@@ -768,7 +772,7 @@ int32_t stack_enqueue_token(StackSession* s, const int* token, const int* pos, f
     int count = 0, cur = 0;
     EmbedParams ep = embed_params(m, token, s->x[0]);
     ep.pos = pos;
-    CU(launch_kernel(embed_positions_kernel, dim3(embed_blocks(c.width), 1), dim3(256), 0, st, false, ep));
+    CU(launch_kernel(embed_positions_kernel, dim3(std::max(1, std::min(32, c.width / 256)), 1), dim3(32), 0, st, false, ep));
     ++count;
     const float* add_w = nullptr;  // non-null: y1 awaits its norm (this is its weight) and its place in the residual stream
     const float* step = nullptr;
